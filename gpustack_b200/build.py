@@ -41,6 +41,7 @@ SOURCES = [
     "sandwich.cu",
     "gated_recurrence.cu",
     "gated_linear_attn.cu",
+    "conv_attn_prep.cu",
 ]
 # What a layer-list decoder (attention with a softmax sink / matrix-memory recurrence, norm after the
 # sum) launches: a fresh checkout that only serves such a model compiles these and nothing else.
@@ -101,8 +102,27 @@ SANDWICH_SOURCES = [
 ]
 
 
+# What a decoder with a norm on every sublayer's output, attention over convolved q, k and v with capped scores and routed
+# feed-forwards launches
+OUTPUT_NORM_SOURCES = [
+    "runtime.cu",
+    "elementwise.cu",
+    "gemm_tcgen05.cu",
+    "gemm_simt.cu",
+    "gemm_simt_grouped.cu",
+    "postnorm.cu",
+    "conv_attn_prep.cu",
+    "attention_sink.cu",
+]
+
+
 def layer_list_sources(mcfg):
     """(tag, sources) of the library a process serving this layer-list model needs."""
+    if getattr(mcfg, "residual", "post_ln") == "output_norm":
+        routed = any(l.mlp is not None for l in mcfg.layers)
+        tc = any(l.mixer.tile_sized for l in mcfg.layers)
+        tag = "output_norm" + ("_routed" if routed else "") + ("_tc" if tc else "")
+        return tag, OUTPUT_NORM_SOURCES + (ROUTED_SOURCES if routed else []) + (ATTENTION_TC_SOURCES if tc else [])
     if getattr(mcfg, "residual", "post_ln") == "sandwich":
         attn = [l.mixer if l.mixer.kind == "attention" else l.mixer.left for l in mcfg.layers
                 if l.mixer.kind in ("attention", "side_by_side")]

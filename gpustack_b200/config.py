@@ -15,7 +15,7 @@ from typing import Optional
 
 SUPPORTED_ARCHS = ("LlamaForCausalLM", "MistralForCausalLM", "Qwen2ForCausalLM", "MixtralForCausalLM")
 # designs whose config.json lists their layers one by one (LayerListConfig below)
-LAYER_LIST_ARCHS = ("Vodavik", "Danipel", "Resevik", "Dotorax")
+LAYER_LIST_ARCHS = ("Vodavik", "Danipel", "Resevik", "Dotorax", "Kerarax")
 
 
 @dataclass
@@ -238,12 +238,31 @@ class AttentionSpec:
     # pool > 0 (with a window): beside the window's tokens, position i sees one (mean key, mean value) per block
     # [b pool, (b + 1) pool) that lies wholly before the window, (b + 1) pool - 1 <= i - window, in the same softmax
     pool: int = 0
+    softcap: float = 0.0           # > 0: score <- softcap * tanh(score / softcap) before the softmax
+    plus_one: bool = False         # the softmax denominator is 1 + sum exp(score): a sink of score 0 without a parameter
+    # > 0: a short causal convolution over time (this many taps, no bias) on every channel of q, k and v right after
+    # the projection, before the q / k norm; the last taps - 1 projected rows of a sequence are part of its state
+    conv_taps: int = 0
 
     kind = "attention"
 
     @property
     def q_width(self) -> int:
         return self.heads * self.dim
+
+    @property
+    def qkv_width(self) -> int:
+        """Channels of the fused [q | k | v] projection."""
+        return self.q_width + self.kv_heads * (self.dim + self.vdim)
+
+    def cache_widths(self, bf16: bool = True) -> tuple:
+        """(key, value) width of a cached row.  A mixer whose prepared rows go through a kernel of their own (conv_taps)
+        is laid out at one tensor-core tile width when served in bf16, keys and values padded with zeros to 64 or 128:
+        zero columns change neither a score nor an output, and the tensor-core kernels can serve any pair of widths."""
+        w = max(self.dim, self.vdim)
+        if not bf16 or not self.conv_taps or self.pool or w > 128 or self.heads // self.kv_heads > 16:
+            return self.dim, self.vdim
+        return (64, 64) if w <= 64 else (128, 128)
 
     @property
     def tile_sized(self) -> bool:
@@ -255,7 +274,8 @@ class AttentionSpec:
     def tokens_tile_sized(self) -> bool:
         """tile_sized without regard to pooled blocks: the tensor-core kernels can attend this mixer's TOKENS and hand
         over every row's log-sum-exp; the pooled blocks then continue that softmax in the generic kernel."""
-        return self.dim == self.vdim and self.dim in (64, 128) and self.heads // self.kv_heads <= 16
+        wk, wv = self.cache_widths()
+        return wk == wv and wk in (64, 128) and self.heads // self.kv_heads <= 16
 
     @property
     def gate_width(self) -> int:
@@ -465,7 +485,7 @@ class LatentAttentionSpec:
 
 @dataclass
 class MoESpec:
-    """Routed feed-forward: softmax over experts + identity router outputs; the `top` largest of score +
+    """Routed feed-forward.  The default form: softmax over experts + identity router outputs; the `top` largest of score +
     correction are chosen, weighted by score / (sum of the chosen scores + 1e-20) * scale.  The last `identity`
     router outputs return the input itself.  An expert is  down(g sigmoid(1.702 g) (u + 1))  with
     g = min(gate x, limit), u = clamp(up x, -limit, limit); a shared expert of the same form (shared_ff > 0)
@@ -480,11 +500,21 @@ class MoESpec:
     shared_limit: float = 0.0
     # other routed designs: score "sigmoid" = sigmoid(z) per output instead of the softmax; renormalize False = the
     # chosen scores are the weights as they are; weight_on "input" = an expert runs on weight * x (its output is not
-    # scaled again); act = the experts' gate activation ("clamped_swish" above | "silu": down(silu(gate x) * up x))
+    # scaled again); act = the experts' gate activation ("clamped_swish" above | "silu": down(silu(gate x) * up x) |
+    # "relu2", no gate: down(relu(up x)^2)); score "chosen_softmax" = the outputs with the largest logits (with their
+    # learned bias, router_bias) are chosen and the weights are the softmax over the chosen logits alone; shared_gate =
+    # the shared expert's output is multiplied by sigmoid(w . x), one number per token
     score: str = "softmax"
     renormalize: bool = True
     weight_on: str = "output"
     act: str = "clamped_swish"
+    router_bias: bool = False
+    shared_gate: bool = False
+
+    @property
+    def gated(self) -> bool:
+        """Experts with a gate and an up matrix (interleaved rows); otherwise one matrix in front of the activation."""
+        return self.act != "relu2"
 
 
 @dataclass
@@ -522,14 +552,20 @@ class LayerListConfig:
     # "parallel": pre-norm with ONE norm per layer whose output feeds the mixer and the feed-forward side by side,
     # x <- x + mixer(norm(x)) + ff(norm(x))
     # "sandwich": a norm before and after every sublayer, x <- x + residual_mult * norm_b(f(norm_a(x)))
+    # "output_norm": a norm on what a sublayer puts out and nothing else, x <- x + norm(f(x))
     residual: str = "post_ln"
-    # "layernorm" (bias-free) | "tanh": tanh(alpha x) w + b, no statistics | "rms" | "rms_zero_centred": an RMS norm
+    # "layernorm" (bias-free) | "layernorm_bias" | "tanh": tanh(alpha x) w + b, no statistics | "rms" | "rms_zero_centred": an RMS norm
     # whose stored weight is the deviation from one, x / rms(x) * (1 + w)
     norm: str = "layernorm"
     # input convolution: every sublayer reads h + conv(h) instead of its normed input h -- a causal convolution over
     # time with canon_taps taps per channel (the last tap multiplies the current token); 0 = none.  The last
     # canon_taps - 1 inputs of every sublayer are part of a sequence's state.
     canon_taps: int = 0
+    # a fixed vector added to the embedding: entries 2i / 2i + 1 = sin / cos of p * 10000^(-2i / width); embed_norm: the
+    # sum goes through the model's norm (tensor embed.norm) before the first layer
+    sinusoidal_positions: bool = False
+    embed_norm: bool = False
+    logit_softcap: float = 0.0                 # > 0: logits <- cap * tanh(logits / cap)
     learned_positions: bool = False            # x_0 = embed[token] + pos[position] (table of max_position_embeddings rows)
     # layers loop_start .. loop_stop-1 run loop_times times in a row with the same weights (every pass with its own
     # cache / state); before each pass but the first the embedding output is added to the residual
@@ -570,7 +606,8 @@ class LayerListConfig:
     def has_state(self) -> bool:
         """True when some mixer carries a recurrent state per sequence (needs a state slot; no prefix reuse)."""
         return self.canon_taps > 1 or any(l.mixer.kind in ("mlstm", "linear_attention", "side_by_side",
-                                                           "gated_linear_attention") for l in self.layers)
+                                                           "gated_linear_attention")
+                                           or (l.mixer.kind == "attention" and l.mixer.conv_taps > 1) for l in self.layers)
 
     def kv_owner(self, l: int) -> Optional[int]:
         """Layer whose K/V cache layer l's attention reads (itself unless kv_from), None for other mixers."""
@@ -589,7 +626,8 @@ class LayerListConfig:
     def kv_bytes_per_token(self, tp: int = 1, elem_bytes: int = 2) -> int:
         mixers = [self.layers[l].mixer for l, _ in self.runs()]
         mixers = [m.left if m.kind == "side_by_side" else m for m in mixers]
-        n = sum(m.kv_heads * (m.dim + m.vdim) * elem_bytes for m in mixers if m.kind == "attention" and m.kv_from is None)
+        n = sum(m.kv_heads * sum(m.cache_widths(elem_bytes == 2)) * elem_bytes for m in mixers
+                if m.kind == "attention" and m.kv_from is None)
         # pooled block means (fp32): ceil(16 / pool) entries per 16-token page
         n += sum(m.kv_heads * (m.dim + m.vdim) * 4 * m.pool_per_page(16) // 16 for m in mixers
                  if m.kind == "attention" and m.pool)
@@ -603,6 +641,8 @@ class LayerListConfig:
                 n += 4 * m.heads * (m.dim * m.vdim + z * m.dim + z)
             elif m.kind in ("linear_attention", "gated_linear_attention"):
                 n += 4 * m.heads * m.dim * m.vdim
+            elif m.kind == "attention" and m.conv_taps > 1:
+                n += 4 * m.qkv_width * (m.conv_taps - 1)
             elif m.kind == "side_by_side":
                 n += 4 * m.right.width * m.right.conv          # the recurrence and its convolution's last inputs
         if self.canon_taps > 1:
@@ -631,7 +671,7 @@ class LayerListConfig:
                 n += D * (2 * m.heads * m.dim + 2 * m.out_width + 2 * m.heads) + m.out_width * D
             if l.mlp is not None and l.mlp.kind == "moe":
                 e = l.mlp.moe
-                n += 3 * D * (e.experts * e.ff + e.shared_ff) + (e.experts + e.identity) * D
+                n += (3 if e.gated else 2) * D * (e.experts * e.ff + e.shared_ff) + (e.experts + e.identity) * D
             elif l.mlp is not None:
                 n += (2 if l.mlp.act == "relu2" else 3) * D * l.mlp.ff
         return 2 * (n + self.vocab_size * D)
@@ -647,6 +687,8 @@ class LayerListConfig:
             return _resevik_from_dict(d)
         if arch == "Dotorax":
             return _dotorax_from_dict(d)
+        if arch == "Kerarax":
+            return _kerarax_from_dict(d)
         layers = []
         for i, e in enumerate(d["layers"]):
             mx = e["mixer"]
@@ -689,6 +731,8 @@ class LayerListConfig:
             return _resevik_to_dict(self)
         if self.architecture == "Dotorax":
             return _dotorax_to_dict(self)
+        if self.architecture == "Kerarax":
+            return _kerarax_to_dict(self)
         out = []
         for l in self.layers:
             m = l.mixer
@@ -963,6 +1007,65 @@ def _dotorax_to_dict(c: "LayerListConfig") -> dict:
     return {"architecture": "Dotorax", "vocab": c.vocab_size, "width": c.hidden_size, "layers": out,
             "norm": {"eps": c.norm_eps}, "residual_mult": c.residual_mult, "canon": {"taps": c.canon_taps},
             "max_positions": c.max_position_embeddings}
+
+
+def _kerarax_from_dict(d: dict) -> "LayerListConfig":
+    """Kerarax: sinusoidal positions and a norm on the embedding; layer norms with weight and bias on every sublayer's
+    output, x <- x + LN(f(x)); grouped attention whose q, k and v pass a short causal convolution per channel, weighted
+    RMS norm of q and k per head, capped scores, a softmax with one more in its denominator; routed relu^2 experts
+    weighted by a softmax over the chosen logits, with a shared expert under a gate of one number per token; capped
+    logits."""
+    layers = []
+    for i, e in enumerate(d["layers"]):
+        mx, kind = e["mixer"], e["type"]
+        if kind != "attention":
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        spec = AttentionSpec(heads=int(mx["heads"]), kv_heads=int(mx.get("kv_heads", mx["heads"])), dim=int(mx["dim"]),
+                             vdim=int(mx.get("vdim", mx["dim"])), scale=float(mx["scale"]), qk_norm=True, qkv_bias=False,
+                             sink=False, gate=False, softcap=float(mx["softcap"]), plus_one=True, conv_taps=int(mx["conv"]))
+        if spec.heads < 1 or spec.kv_heads < 1 or spec.heads % spec.kv_heads:
+            raise ValueError(f"layer {i}: heads {spec.heads} not a multiple of kv_heads {spec.kv_heads}")
+        if spec.softcap <= 0.0:
+            raise ValueError(f"layer {i}: softcap {spec.softcap} must be positive")
+        if not 1 <= spec.conv_taps <= 8:
+            raise ValueError(f"layer {i}: conv {spec.conv_taps} taps (1 .. 8)")
+        mlp = e.get("mlp")
+        if mlp is not None:
+            if mlp.get("kind") != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+            ro, ex, sh = mlp["router"], mlp["expert"], mlp.get("shared") or None
+            moe = MoESpec(experts=int(ro["experts"]), top=int(ro["top"]), ff=int(ex["ff"]), limit=0.0,
+                          shared_ff=int(sh["ff"]) if sh else 0, score="chosen_softmax", act="relu2", router_bias=True,
+                          shared_gate=sh is not None)
+            if not 1 <= moe.top <= moe.experts:
+                raise ValueError(f"layer {i}: top {moe.top} of {moe.experts} experts")
+            mlp = MLPSpec(kind="moe", ff=max(moe.ff, moe.shared_ff), act="relu2", moe=moe)
+        layers.append(LayerSpec(mixer=spec, mlp=mlp))
+    cap = float(d.get("logit_softcap") or 0.0)
+    if cap < 0.0:
+        raise ValueError(f"logit_softcap {cap} must not be negative")
+    eos_all = _eos_of(d)
+    return LayerListConfig(architecture="Kerarax", vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers,
+                           norm_eps=float(d["norm"]["eps"]), residual="output_norm", norm="layernorm_bias",
+                           sinusoidal_positions=True, embed_norm=True, logit_softcap=cap, eos_token_ids=eos_all,
+                           eos_token_id=eos_all[0] if eos_all else None, bos_token_id=d.get("bos_token_id"))
+
+
+def _kerarax_to_dict(c: "LayerListConfig") -> dict:
+    out = []
+    for l in c.layers:
+        m = l.mixer
+        mx = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale, "softcap": m.softcap,
+              "conv": m.conv_taps}
+        mlp = None
+        if l.mlp is not None:
+            e = l.mlp.moe
+            mlp = {"kind": "moe", "expert": {"ff": e.ff}, "router": {"experts": e.experts, "top": e.top}}
+            if e.shared_ff:
+                mlp["shared"] = {"ff": e.shared_ff}
+        out.append({"type": "attention", "mixer": mx, "mlp": mlp})
+    return {"architecture": "Kerarax", "vocab": c.vocab_size, "width": c.hidden_size, "layers": out,
+            "norm": {"eps": c.norm_eps}, "logit_softcap": c.logit_softcap}
 
 
 # Named shapes used by tests and bench (random-init; there are no checkpoints offline).

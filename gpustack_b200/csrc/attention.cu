@@ -72,7 +72,9 @@ __device__ __forceinline__ bf16 finish_row(float num, float den, float mm, const
   return __float2bfloat16_rn(o);
 }
 
-template <int D>
+// CAP: the scaled score passes cap * tanh(score / cap) before the mask; scale_log2 then holds 2 log2e scale / cap and
+// cap_log2 the cap in base-2 units.
+template <int D, bool CAP>
 __global__ void __launch_bounds__(kDecWarps * 32, 2)
 paged_attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride,
                          const bf16* __restrict__ k_cache, const bf16* __restrict__ v_cache,
@@ -81,7 +83,7 @@ paged_attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride,
                          float* __restrict__ ws_o, float* __restrict__ ws_ml, int num_splits,
                          int Hq, int Hkv, float scale_log2, uint32_t* __restrict__ split_ctr,
                          const float* __restrict__ sink, const bf16* __restrict__ gate, int64_t gate_stride,
-                         int window, int gate_per_head, float* __restrict__ lse_out) {
+                         int window, int gate_per_head, float* __restrict__ lse_out, float cap_log2) {
   pdl_launch_dependents();
   pdl_wait();
   using Cfg = DecCfg<D>;
@@ -179,7 +181,9 @@ paged_attn_decode_kernel(const bf16* __restrict__ q, int64_t q_stride,
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int tok = tok0 + t * 8 + (e & 1);
-        const float v = (tok < seq_len && tok >= first_key) ? s[t][e] * scale_log2 : -INFINITY;
+        float x = s[t][e] * scale_log2;
+        if constexpr (CAP) x = fmaf(-2.f * cap_log2, rcp_approx(ex2_approx(x) + 1.f), cap_log2);
+        const float v = (tok < seq_len && tok >= first_key) ? x : -INFINITY;
         s[t][e] = v;
         if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
       }
@@ -760,6 +764,24 @@ extern "C" int b200_paged_attn_decode_hg(const void* q, int64_t q_stride, const 
                                     stream);
 }
 
+template <int D, bool CAP>
+static int launch_decode(dim3 grid, cudaStream_t s, const void* q, int64_t q_stride, const void* k_cache, const void* v_cache,
+                         const int32_t* block_table, int max_blocks, const int32_t* seq_lens, void* out, float* ws_o, float* ws_ml,
+                         int num_splits, int Hq, int Hkv, float scale_log2, uint32_t* split_ctr, const float* sink,
+                         const void* gate, int64_t gate_stride, int window, int gate_per_head, float* lse_out, float cap_log2) {
+  static bool once = false;
+  if (!once) {
+    const int rc = set_smem_attr(paged_attn_decode_kernel<D, CAP>, DecCfg<D>::kSmemBytes, "attn_decode");
+    if (rc) return rc;
+    once = true;
+  }
+  (void)launch_pdl(paged_attn_decode_kernel<D, CAP>, grid, dim3(kDecWarps * 32), DecCfg<D>::kSmemBytes, s, 1, (const bf16*)q,
+                   q_stride, (const bf16*)k_cache, (const bf16*)v_cache, block_table, max_blocks, seq_lens, (bf16*)out, ws_o,
+                   ws_ml, num_splits, Hq, Hkv, scale_log2, split_ctr, sink, (const bf16*)gate, gate_stride, window,
+                   gate_per_head, lse_out, cap_log2);
+  return b200_check_launch("b200_paged_attn_decode");
+}
+
 extern "C" int b200_paged_attn_decode_lse(const void* q, int64_t q_stride, const void* k_cache,
                                           const void* v_cache, const int32_t* block_table,
                                           int max_blocks, const int32_t* seq_lens, void* out,
@@ -767,7 +789,20 @@ extern "C" int b200_paged_attn_decode_lse(const void* q, int64_t q_stride, const
                                           int D, int block_size, float scale, const float* sink,
                                           const void* gate, int64_t gate_stride, int window, int gate_per_head,
                                           float* lse_out, void* stream) {
+  return b200_paged_attn_decode_cap(q, q_stride, k_cache, v_cache, block_table, max_blocks, seq_lens, out, workspace, num_splits,
+                                    B, Hq, Hkv, D, block_size, scale, sink, gate, gate_stride, window, gate_per_head, lse_out,
+                                    0.f, stream);
+}
+
+extern "C" int b200_paged_attn_decode_cap(const void* q, int64_t q_stride, const void* k_cache,
+                                          const void* v_cache, const int32_t* block_table,
+                                          int max_blocks, const int32_t* seq_lens, void* out,
+                                          void* workspace, int num_splits, int B, int Hq, int Hkv,
+                                          int D, int block_size, float scale, const float* sink,
+                                          const void* gate, int64_t gate_stride, int window, int gate_per_head,
+                                          float* lse_out, float softcap, void* stream) {
   B200_REQUIRE(window >= 0, "attn_decode: window %d", window);
+  B200_REQUIRE(softcap >= 0.f, "attn_decode: softcap %g is negative", (double)softcap);
   B200_REQUIRE(B >= 0 && Hq > 0 && Hkv > 0 && Hq % Hkv == 0, "attn_decode: bad head counts");
   B200_REQUIRE(Hq / Hkv <= 16, "attn_decode: group size %d > 16 unsupported", Hq / Hkv);
   B200_REQUIRE(block_size == kPage, "attn_decode: block_size must be %d", kPage);
@@ -776,7 +811,8 @@ extern "C" int b200_paged_attn_decode_lse(const void* q, int64_t q_stride, const
   B200_REQUIRE(q_stride % 8 == 0, "attn_decode: q_stride must be a multiple of 8");
   if (B == 0) return B200_OK;
   cudaStream_t s = (cudaStream_t)stream;
-  const float scale_log2 = scale * 1.4426950408889634f;
+  const float cap_log2 = softcap * 1.4426950408889634f;
+  const float scale_log2 = (softcap > 0.f ? 2.f * scale / softcap : scale) * 1.4426950408889634f;
   // counters live in the first bytes of the workspace, sized for THIS call's B (<= the B the buffer was
   // sized and zeroed for: a prefix of a zeroed, self-resetting array is itself zeroed)
   uint32_t* split_ctr = reinterpret_cast<uint32_t*>(workspace);
@@ -784,33 +820,13 @@ extern "C" int b200_paged_attn_decode_lse(const void* q, int64_t q_stride, const
                           : nullptr;
   float* ws_ml = ws_o ? ws_o + (size_t)B * Hq * num_splits * D : nullptr;
   dim3 grid(Hkv, num_splits, B);
-  int rc;
-  if (D == 128) {
-    static bool once = false;
-    if (!once) {
-      rc = set_smem_attr(paged_attn_decode_kernel<128>, DecCfg<128>::kSmemBytes, "attn_decode");
-      if (rc) return rc;
-      once = true;
-    }
-    (void)launch_pdl(paged_attn_decode_kernel<128>, dim3(grid), dim3(kDecWarps * 32), DecCfg<128>::kSmemBytes, s, 1, 
-        (const bf16*)q, q_stride, (const bf16*)k_cache, (const bf16*)v_cache, block_table,
-        max_blocks, seq_lens, (bf16*)out, ws_o, ws_ml, num_splits, Hq, Hkv, scale_log2, split_ctr, sink,
-        (const bf16*)gate, gate_stride, window, gate_per_head, lse_out);
-    rc = b200_check_launch("b200_paged_attn_decode");
-  } else {
-    static bool once = false;
-    if (!once) {
-      rc = set_smem_attr(paged_attn_decode_kernel<64>, DecCfg<64>::kSmemBytes, "attn_decode");
-      if (rc) return rc;
-      once = true;
-    }
-    (void)launch_pdl(paged_attn_decode_kernel<64>, dim3(grid), dim3(kDecWarps * 32), DecCfg<64>::kSmemBytes, s, 1, 
-        (const bf16*)q, q_stride, (const bf16*)k_cache, (const bf16*)v_cache, block_table,
-        max_blocks, seq_lens, (bf16*)out, ws_o, ws_ml, num_splits, Hq, Hkv, scale_log2, split_ctr, sink,
-        (const bf16*)gate, gate_stride, window, gate_per_head, lse_out);
-    rc = b200_check_launch("b200_paged_attn_decode");
-  }
-  return rc;
+#define B200_DECODE(DD, CAP)                                                                                              \
+  launch_decode<DD, CAP>(grid, s, q, q_stride, k_cache, v_cache, block_table, max_blocks, seq_lens, out, ws_o, ws_ml,    \
+                         num_splits, Hq, Hkv, scale_log2, split_ctr, sink, gate, gate_stride, window, gate_per_head,     \
+                         lse_out, cap_log2)
+  if (softcap > 0.f) return D == 128 ? B200_DECODE(128, true) : B200_DECODE(64, true);
+  return D == 128 ? B200_DECODE(128, false) : B200_DECODE(64, false);
+#undef B200_DECODE
 }
 
 extern "C" int b200_attn_prefill_tile(int Hq, int Hkv) {
@@ -828,7 +844,7 @@ int paged_attn_prefill_tc(const void* q, int64_t q_stride, int num_tokens, const
                           const int32_t* ctx_lens, const int32_t* tile_seq, const int32_t* tile_q0, int num_tiles,
                           void* out, int Hq, int Hkv, int D, float scale, cudaStream_t stream,
                           const float* sink = nullptr, const void* gate = nullptr, int64_t gate_stride = 0,
-                          int window = 0, int gate_per_head = 0, float* lse_out = nullptr);
+                          int window = 0, int gate_per_head = 0, float* lse_out = nullptr, float softcap = 0.f);
 }  // namespace b200
 
 extern "C" int b200_attn_prefill_tc_covers(int Hq, int Hkv, int D) {
@@ -878,13 +894,26 @@ extern "C" int b200_paged_attn_prefill_lse(const void* q, int64_t q_stride, int 
                                            int Hq, int Hkv, int D, int block_size, float scale, const float* sink,
                                            const void* gate, int64_t gate_stride, int window, int gate_per_head,
                                            float* lse_out, void* stream) {
+  return b200_paged_attn_prefill_cap(q, q_stride, num_tokens, k_cache, v_cache, num_blocks, block_table, max_blocks, cu_q,
+                                     ctx_lens, tile_seq, tile_q0, num_tiles, out, Hq, Hkv, D, block_size, scale, sink, gate,
+                                     gate_stride, window, gate_per_head, lse_out, 0.f, stream);
+}
+
+extern "C" int b200_paged_attn_prefill_cap(const void* q, int64_t q_stride, int num_tokens, const void* k_cache,
+                                           const void* v_cache, int num_blocks, const int32_t* block_table,
+                                           int max_blocks, const int32_t* cu_q, const int32_t* ctx_lens,
+                                           const int32_t* tile_seq, const int32_t* tile_q0, int num_tiles, void* out,
+                                           int Hq, int Hkv, int D, int block_size, float scale, const float* sink,
+                                           const void* gate, int64_t gate_stride, int window, int gate_per_head,
+                                           float* lse_out, float softcap, void* stream) {
+  B200_REQUIRE(softcap >= 0.f, "attn_prefill_ex: softcap %g is negative", (double)softcap);
   B200_REQUIRE(window >= 0, "attn_prefill_ex: window %d", window);
   B200_REQUIRE(b200_attn_prefill_tc_covers(Hq, Hkv, D), "attn_prefill_ex: heads %d / %d x %d not covered", Hq, Hkv, D);
   B200_REQUIRE(block_size == kPage, "attn_prefill_ex: block_size must be %d", kPage);
   if (num_tiles <= 0) return B200_OK;
   const int rc = paged_attn_prefill_tc(q, q_stride, num_tokens, k_cache, v_cache, num_blocks, block_table, max_blocks,
                                        cu_q, ctx_lens, tile_seq, tile_q0, num_tiles, out, Hq, Hkv, D, scale,
-                                       (cudaStream_t)stream, sink, gate, gate_stride, window, gate_per_head, lse_out);
+                                       (cudaStream_t)stream, sink, gate, gate_stride, window, gate_per_head, lse_out, softcap);
   if (rc > 0) {
     b200_set_error("attn_prefill_ex: the tensor-core kernel does not take this call (alignment or device)");
     return B200_ERR_UNSUPPORTED;

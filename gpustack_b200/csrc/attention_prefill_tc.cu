@@ -60,13 +60,20 @@ constexpr int kFaSmemBytes = 115712;                   // (228 KB - 2 x 1 KB res
 constexpr int kFaMaxSlack = kFaSmemBytes - kFaOffBar - 256;
 constexpr int kFaTmemCols = 256;                       // S0 [0,64)  S1 [64,128)  O [128,256)
 constexpr float kFaRescaleThreshold = 8.f;             // log2 units
+// a capped softmax whose scores stay within +-80 (base 2) runs against the reference 0: up to 2^80 per key, 2^24 keys and
+// values of 2^20 stay inside fp32, and 2^-80 is a normal number
+constexpr float kFaBoundedCap = 80.f;
 
 // P_TMEM: P_j is written back into the first 32 columns of the TMEM buffer S_j came from (bf16 pairs
 // per 32-bit column, tcgen05.st) and the PV MMA reads its A operand from tensor memory: no shared-
 // memory round trip, no proxy fence, and the softmax of block j+1 no longer waits for PV_j to retire
 // (it only ever waits for p_empty when the O accumulator has to be rescaled).  P_TMEM = false keeps
 // P in swizzled shared memory (B200_ATTN_P_TMEM=0, A/B runs).
-template <int G, bool P_TMEM>
+// CAP: the scaled score passes cap * tanh(score / cap) before the mask (scale_log2 then holds 2 log2e scale / cap, cap_log2
+// the cap in base-2 units).  A capped score is bounded, so when 2^cap_log2 cannot leave the fp32 range (`bounded`: the
+// probabilities, their sum and the accumulator included) the softmax needs no running maximum at all: its reference is 0,
+// no row is searched for its maximum and O is never rescaled.
+template <int G, bool P_TMEM, bool CAP>
 __global__ void __launch_bounds__(kFaThreads, 2)
 paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
                              const __grid_constant__ CUtensorMap tmap_k,
@@ -76,7 +83,7 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
                              const int32_t* __restrict__ tile_seq, const int32_t* __restrict__ tile_q0,
                              int num_tiles, bf16* __restrict__ out, int Hq, int Hkv, float scale_log2,
                              const float* __restrict__ sink, const bf16* __restrict__ gate, int64_t gate_stride,
-                             int window, int gate_per_head, float* __restrict__ lse_out) {
+                             int window, int gate_per_head, float* __restrict__ lse_out, float cap_log2, int bounded) {
   constexpr int TPT = 128 / G;   // query tokens per tile
   extern __shared__ uint8_t fa_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(fa_raw) + 1023) &
@@ -302,7 +309,8 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
       const bool valid = qi < m.q_len;
       const int qpos = m.ctx + qi;
       const int total_len = m.total_len;
-      float m_used = -INFINITY, l = 0.f;
+      float m_used = (CAP && bounded) ? 0.f : -INFINITY, l = 0.f;
+      const float sl = CAP ? 1.f : scale_log2;    // what a (masked) score is multiplied by on its way into the exponent
 
       const int row_lo = window > 0 ? qpos - window + 1 : 0;   // first key this row sees
       for (int j = m.j0; j < m.n_blocks; ++j, ++gb) {
@@ -314,6 +322,14 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
         tmem_ld_32x32(t_lane + s_col + 32, s1);
         tmem_ld_wait();
         const int kv0 = j * kFaKv;
+        if constexpr (CAP) {
+          // cap tanh(x / cap) = cap - 2 cap / (exp(2 x / cap) + 1): exact to fp32 rounding of the cap, +-cap in the limits
+#pragma unroll
+          for (int c = 0; c < 32; ++c) {
+            s0[c] = __float_as_uint(fmaf(-2.f * cap_log2, rcp_approx(ex2_approx(__uint_as_float(s0[c]) * scale_log2) + 1.f), cap_log2));
+            s1[c] = __float_as_uint(fmaf(-2.f * cap_log2, rcp_approx(ex2_approx(__uint_as_float(s1[c]) * scale_log2) + 1.f), cap_log2));
+          }
+        }
         // block-uniform: does any row of the tile see a masked column in this block?
         const bool need_mask = (kv0 + kFaKv - 1 > m.ctx + m.q0) || (kv0 + kFaKv - 1 >= total_len) ||
                                (window > 0 && kv0 < m.ctx + m.q0 + TPT - window);
@@ -328,9 +344,11 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
         // row maximum on the raw scores (scale > 0 commutes with max); the scale itself is folded
         // into the exponent's FFMA below
         float mx = -INFINITY;
+        if (!(CAP && bounded)) {
 #pragma unroll
-        for (int c = 0; c < 32; ++c) mx = fmaxf(mx, fmaxf(__uint_as_float(s0[c]), __uint_as_float(s1[c])));
-        mx *= scale_log2;
+          for (int c = 0; c < 32; ++c) mx = fmaxf(mx, fmaxf(__uint_as_float(s0[c]), __uint_as_float(s1[c])));
+          mx *= sl;
+        }
         // lazy rescale: move the reference maximum only when the row maximum outgrew it by > 2^8
         // (always on the first block, where m_used = -inf and the factor is exp2(-inf) = 0)
         float alpha = 1.f;
@@ -347,10 +365,10 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
         const float neg_m = m_used == -INFINITY ? 0.f : -m_used;
 #pragma unroll
         for (int c = 0; c < 32; c += 2) {
-          const float p0 = ex2_approx(fmaf(__uint_as_float(s0[c]), scale_log2, neg_m));
-          const float p1 = ex2_approx(fmaf(__uint_as_float(s0[c + 1]), scale_log2, neg_m));
-          const float p2 = ex2_approx(fmaf(__uint_as_float(s1[c]), scale_log2, neg_m));
-          const float p3 = ex2_approx(fmaf(__uint_as_float(s1[c + 1]), scale_log2, neg_m));
+          const float p0 = ex2_approx(fmaf(__uint_as_float(s0[c]), sl, neg_m));
+          const float p1 = ex2_approx(fmaf(__uint_as_float(s0[c + 1]), sl, neg_m));
+          const float p2 = ex2_approx(fmaf(__uint_as_float(s1[c]), sl, neg_m));
+          const float p3 = ex2_approx(fmaf(__uint_as_float(s1[c + 1]), sl, neg_m));
           sum += (p0 + p1) + (p2 + p3);
           pk[c >> 1] = pack_bf16(p0, p1);
           pk[16 + (c >> 1)] = pack_bf16(p2, p3);
@@ -481,14 +499,14 @@ paged_attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q,
   }
 }
 
-template <int G, bool P_TMEM>
+template <int G, bool P_TMEM, bool CAP = false>
 static int launch_prefill_tc(const void* q, int64_t q_stride, int num_tokens, const void* k_cache,
                              const void* v_cache, int num_blocks, const int32_t* block_table, int max_blocks,
                              const int32_t* cu_q, const int32_t* ctx_lens, const int32_t* tile_seq,
                              const int32_t* tile_q0, int num_tiles, void* out, int Hq, int Hkv, float scale,
                              const float* sink, const void* gate, int64_t gate_stride, int window, int gate_per_head,
-                             float* lse_out, cudaStream_t stream) {
-  auto kernel = paged_attn_prefill_tc_kernel<G, P_TMEM>;
+                             float* lse_out, float softcap, cudaStream_t stream) {
+  auto kernel = paged_attn_prefill_tc_kernel<G, P_TMEM, CAP>;
   static bool attr_set = false;
   if (!attr_set) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kFaSmemBytes);
@@ -508,7 +526,8 @@ static int launch_prefill_tc(const void* q, int64_t q_stride, int num_tokens, co
   if (rc) return rc;
   rc = make_tmap_bf16_2d(&tv, v_cache, kv_rows, kFaD, kFaD, kFaPage, 64);
   if (rc) return rc;
-  const float scale_log2 = scale * 1.4426950408889634f;
+  const float cap_log2 = softcap * 1.4426950408889634f;
+  const float scale_log2 = (CAP ? 2.f * scale / softcap : scale) * 1.4426950408889634f;
   static int persist = -1;
   if (persist < 0) {
     const char* pe = getenv("B200_ATTN_PERSIST");   // =0: one CTA per (tile, kv-head) instead of the persistent loop
@@ -519,7 +538,8 @@ static int launch_prefill_tc(const void* q, int64_t q_stride, int num_tokens, co
   const int grid = (int)(persist ? (total_work < 2LL * sms ? total_work : 2LL * sms) : total_work);
   cudaError_t e = launch_pdl(kernel, dim3(grid), dim3(kFaThreads), (size_t)kFaSmemBytes, stream, 1, tq, tk, tv,
                              block_table, max_blocks, cu_q, ctx_lens, tile_seq, tile_q0, num_tiles, (bf16*)out, Hq,
-                             Hkv, scale_log2, sink, (const bf16*)gate, gate_stride, window, gate_per_head, lse_out);
+                             Hkv, scale_log2, sink, (const bf16*)gate, gate_stride, window, gate_per_head, lse_out, cap_log2,
+                             cap_log2 <= kFaBoundedCap ? 1 : 0);
   if (e != cudaSuccess) {
     b200_set_error("b200_paged_attn_prefill(tc): launch failed: %s", cudaGetErrorString(e));
     (void)cudaGetLastError();
@@ -534,7 +554,7 @@ int paged_attn_prefill_tc(const void* q, int64_t q_stride, int num_tokens, const
                           int num_blocks, const int32_t* block_table, int max_blocks, const int32_t* cu_q,
                           const int32_t* ctx_lens, const int32_t* tile_seq, const int32_t* tile_q0, int num_tiles,
                           void* out, int Hq, int Hkv, int D, float scale, cudaStream_t stream, const float* sink,
-                          const void* gate, int64_t gate_stride, int window, int gate_per_head, float* lse_out) {
+                          const void* gate, int64_t gate_stride, int window, int gate_per_head, float* lse_out, float softcap) {
   static int enabled = -1;
   if (enabled < 0) {
     const char* e = getenv("B200_ATTN_PREFILL_TC");   // =0: keep the mma.sync kernels (A/B runs)
@@ -550,9 +570,10 @@ int paged_attn_prefill_tc(const void* q, int64_t q_stride, int num_tokens, const
     const char* e = getenv("B200_ATTN_P_TMEM");   // =0: P through shared memory (A/B runs)
     p_tmem = (e && e[0] == '0') ? 0 : 1;
   }
-#define B200_FA_LAUNCH(GG, PT)                                                                                       \
-  launch_prefill_tc<GG, PT>(q, q_stride, num_tokens, k_cache, v_cache, num_blocks, block_table, max_blocks, cu_q,    \
-                            ctx_lens, tile_seq, tile_q0, num_tiles, out, Hq, Hkv, scale, sink, gate, gate_stride, window, gate_per_head, lse_out, stream)
+#define B200_FA_LAUNCH(GG, ...)                                                                                      \
+  launch_prefill_tc<GG, __VA_ARGS__>(q, q_stride, num_tokens, k_cache, v_cache, num_blocks, block_table, max_blocks, cu_q,    \
+                            ctx_lens, tile_seq, tile_q0, num_tiles, out, Hq, Hkv, scale, sink, gate, gate_stride, window, gate_per_head, lse_out, softcap, stream)
+  if (softcap > 0.f) return G == 4 ? B200_FA_LAUNCH(4, true, true) : B200_FA_LAUNCH(8, true, true);
   if (G == 4) return p_tmem ? B200_FA_LAUNCH(4, true) : B200_FA_LAUNCH(4, false);
   return p_tmem ? B200_FA_LAUNCH(8, true) : B200_FA_LAUNCH(8, false);
 #undef B200_FA_LAUNCH

@@ -12,7 +12,8 @@
 //     the window -- block b is seen by position i when (b + 1) pool - 1 <= i - window -- in the same softmax as the
 //     window's tokens; the means are fp32 entries of a second cache addressed through the same block table
 //     (sandwich.cu: kv_pool_update),
-//   * an output gate with ONE number per head, and a learned factor per head on the score.
+//   * an output gate with ONE number per head, and a learned factor per head on the score,
+//   * a soft cap on the scaled score: cap * tanh(score / cap), before the mask and the softmax.
 // Three kernels: `attn_prep` (bias + norms + temperature, in place for q, scatter of k and v into
 // the pages), `prefill` (a tile of 16 query rows of one sequence per CTA, keys staged in shared
 // memory 32 at a time, online softmax) and `decode` (one query row per CTA, the four warps take
@@ -33,6 +34,9 @@ __device__ __forceinline__ float as_f32(float v) { return v; }
 __device__ __forceinline__ float as_f32(bf16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ void as_store(float* p, float v) { *p = v; }
 __device__ __forceinline__ void as_store(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+// a score already multiplied by scale / cap (cap > 0), or by scale alone
+__device__ __forceinline__ float capped(float s, float cap) { return cap > 0.f ? cap * tanhf(s) : s; }
 
 constexpr int kMaxDvLanes = 16;    // value width <= 512: kernels are built for 8 (<= 256) and 16 columns per lane
 
@@ -199,7 +203,7 @@ attn_sink_prefill_kernel(const TA* __restrict__ proj, int64_t ld, int gate_col, 
                          const float* __restrict__ sink, TA* out, int64_t ldo, int H, int G, int dk, int dv, int page,
                          float scale, int64_t v_ld, int window, int gate_per_head, const float* __restrict__ head_scale,
                          const float* __restrict__ pool_k, const float* __restrict__ pool_v, int pool, int per_page,
-                         const float* __restrict__ init_lse) {
+                         const float* __restrict__ init_lse, float softcap) {
   extern __shared__ float smem[];
   float* Qs = smem;                                   // [16][dk]
   float* Ks = Qs + kPfRows * dk;                      // [32][dk + 1]
@@ -215,6 +219,7 @@ attn_sink_prefill_kernel(const TA* __restrict__ proj, int64_t ld, int gate_col, 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int32_t* bt = block_table + (size_t)s * max_blocks;
   if (head_scale != nullptr) scale *= head_scale[h];
+  if (softcap > 0.f) scale /= softcap;
 
   for (int i = threadIdx.x; i < kPfRows * dk; i += blockDim.x) {
     const int r = i / dk, d = i - r * dk;
@@ -303,7 +308,7 @@ attn_sink_prefill_kernel(const TA* __restrict__ proj, int64_t ld, int gate_col, 
       const int qpos = ctx + q0 + warp * kPfRowsPerWarp + r;
       const bool seen = pooled ? (k0 + lane) < (qpos - window + 1) / pool      // (negative numerators: nothing seen)
                                : ((k0 + lane) <= qpos && (k0 + lane) < kv_end && (window <= 0 || qpos - (k0 + lane) < window));
-      const float sv = seen ? sc[r] * scale : -CUDART_INF_F;
+      const float sv = seen ? capped(sc[r] * scale, softcap) : -CUDART_INF_F;
       const float mn = fmaxf(m[r], warp_max(sv));
       float p = 0.f, corr = 1.f;
       if (mn > -CUDART_INF_F) {
@@ -368,7 +373,8 @@ attn_sink_decode_kernel(const TA* __restrict__ proj, int64_t ld, int gate_col, c
                         const int32_t* __restrict__ seq_lens, const float* __restrict__ sink, TA* out, int64_t ldo,
                         int H, int G, int dk, int dv, int page, float scale, int64_t v_ld, int window, int gate_per_head,
                         const float* __restrict__ head_scale, const float* __restrict__ pool_k,
-                        const float* __restrict__ pool_v, int pool, int per_page, const float* __restrict__ init_lse) {
+                        const float* __restrict__ pool_v, int pool, int per_page, const float* __restrict__ init_lse,
+                        float softcap) {
   __shared__ float sm_m[kDecWarps], sm_l[kDecWarps];
   extern __shared__ __align__(16) float sm_dyn[];      // [dk (padded to 8)] query, then [warps][dv] partial outputs
   constexpr int E = 16 / (int)sizeof(TA);               // elements per 16-byte load
@@ -380,6 +386,7 @@ attn_sink_decode_kernel(const TA* __restrict__ proj, int64_t ld, int gate_col, c
   const int n = seq_lens[b];
   const int32_t* bt = block_table + (size_t)b * max_blocks;
   if (head_scale != nullptr) scale *= head_scale[h];
+  if (softcap > 0.f) scale /= softcap;
   for (int d = threadIdx.x; d < dkp; d += blockDim.x)
     qsm[d] = d < dk ? as_f32(proj[(size_t)b * ld + h * dk + d]) * scale : 0.f;
   __syncthreads();
@@ -422,7 +429,7 @@ attn_sink_decode_kernel(const TA* __restrict__ proj, int64_t ld, int gate_col, c
       } else {
         for (int d = 0; d < dk; ++d) a = fmaf(qsm[d], kp[d], a);
       }
-      sc = a;
+      sc = capped(a, softcap);
     }
     const float mn = fmaxf(m, warp_max(sc));
     const float corr = expf(m - mn), p = live ? expf(sc - mn) : 0.f;
@@ -464,7 +471,7 @@ attn_sink_decode_kernel(const TA* __restrict__ proj, int64_t ld, int gate_col, c
       } else {
         for (int d = 0; d < dk; ++d) a = fmaf(qsm[d], as_f32(kp[d]), a);
       }
-      sc = a;
+      sc = capped(a, softcap);
     }
     const float mn = fmaxf(m, warp_max(sc));            // finite: some key of this block is live
     const float corr = expf(m - mn), p = live ? expf(sc - mn) : 0.f;
@@ -572,10 +579,12 @@ static int attn_sink_prefill_launch(const void* proj, int f32, int64_t ld, int g
                                     const int32_t* tile_q0, int n_tiles, int tile_rows, const float* sink, void* out,
                                     int64_t ldo, int H, int G, int dk, int dv, int page, float scale, int64_t v_ld,
                                     int window, int gate_per_head, const float* head_scale, const float* pool_k,
-                                    const float* pool_v, int pool, int per_page, const float* init_lse, void* stream) {
+                                    const float* pool_v, int pool, int per_page, const float* init_lse,
+                                    float softcap, void* stream) {
   if (v_ld <= 0) v_ld = dv;
   B200_REQUIRE(pool_k == nullptr || (pool_v != nullptr && window > 0 && pool > 0 && per_page == (page + pool - 1) / pool),
                "attn_sink_prefill: pooled blocks need a window, both caches and ceil(page / pool) entries per page");
+  B200_REQUIRE(softcap >= 0.f, "attn_sink_prefill: softcap %g is negative", (double)softcap);
   B200_REQUIRE(v_ld >= dv, "attn_sink_prefill: value row pitch %lld < dv=%d", (long long)v_ld, dv);
   B200_REQUIRE(tile_rows > 0 && tile_rows % kPfRows == 0, "attn_sink_prefill: tiles of %d rows (multiples of %d)",
                tile_rows, kPfRows);
@@ -594,13 +603,25 @@ static int attn_sink_prefill_launch(const void* proj, int f32, int64_t ld, int g
     attn_sink_prefill_kernel<TA, L><<<grid, kPfWarps * 32, smem, s>>>(                                             \
         (const TA*)proj, ld, gate_col, (const TA*)k_cache, (const TA*)v_cache, block_table, max_blocks, cu_q,       \
         ctx_lens, tile_seq, tile_q0, sink, (TA*)out, ldo, H, G, dk, dv, page, scale, v_ld, window, gate_per_head,   \
-        head_scale, pool_k, pool_v, pool, per_page, init_lse);                                                     \
+        head_scale, pool_k, pool_v, pool, per_page, init_lse, softcap);                                            \
   } while (0)
   const bool wide = dv > 256;
   if (f32) { if (wide) B200_PF(float, 16); else B200_PF(float, 8); }
   else { if (wide) B200_PF(bf16, 16); else B200_PF(bf16, 8); }
 #undef B200_PF
   return b200_check_launch("b200_attn_sink_prefill");
+}
+
+extern "C" int b200_attn_sink_prefill_cap(const void* proj, int f32, int64_t ld, int gate_col, const void* k_cache,
+                                           const void* v_cache, const int32_t* block_table, int max_blocks,
+                                           const int32_t* cu_q, const int32_t* ctx_lens, const int32_t* tile_seq,
+                                           const int32_t* tile_q0, int n_tiles, int tile_rows, const float* sink, void* out,
+                                           int64_t ldo, int H, int G, int dk, int dv, int page, float scale, int64_t v_ld,
+                                           int window, int gate_per_head, const float* head_scale, const float* pool_k,
+                                           const float* pool_v, int pool, int per_page, float softcap, void* stream) {
+  return attn_sink_prefill_launch(proj, f32, ld, gate_col, k_cache, v_cache, block_table, max_blocks, cu_q, ctx_lens, tile_seq,
+                                  tile_q0, n_tiles, tile_rows, sink, out, ldo, H, G, dk, dv, page, scale, v_ld, window,
+                                  gate_per_head, head_scale, pool_k, pool_v, pool, per_page, nullptr, softcap, stream);
 }
 
 extern "C" int b200_attn_sink_prefill_pool(const void* proj, int f32, int64_t ld, int gate_col, const void* k_cache,
@@ -612,7 +633,7 @@ extern "C" int b200_attn_sink_prefill_pool(const void* proj, int f32, int64_t ld
                                            const float* pool_v, int pool, int per_page, void* stream) {
   return attn_sink_prefill_launch(proj, f32, ld, gate_col, k_cache, v_cache, block_table, max_blocks, cu_q, ctx_lens, tile_seq,
                                   tile_q0, n_tiles, tile_rows, sink, out, ldo, H, G, dk, dv, page, scale, v_ld, window,
-                                  gate_per_head, head_scale, pool_k, pool_v, pool, per_page, nullptr, stream);
+                                  gate_per_head, head_scale, pool_k, pool_v, pool, per_page, nullptr, 0.f, stream);
 }
 
 extern "C" int b200_attn_sink_prefill_more(const void* proj, int f32, int64_t ld, const void* k_cache,
@@ -624,7 +645,7 @@ extern "C" int b200_attn_sink_prefill_more(const void* proj, int f32, int64_t ld
   B200_REQUIRE(init_lse != nullptr && pool_k != nullptr, "attn_sink_prefill_more: needs the first part's log-sum-exp and pooled blocks");
   return attn_sink_prefill_launch(proj, f32, ld, -1, k_cache, k_cache, block_table, max_blocks, cu_q, ctx_lens, tile_seq,
                                   tile_q0, n_tiles, tile_rows, nullptr, out, ldo, H, G, dk, dv, page, scale, 0, window, 0,
-                                  head_scale, pool_k, pool_v, pool, per_page, init_lse, stream);
+                                  head_scale, pool_k, pool_v, pool, per_page, init_lse, 0.f, stream);
 }
 
 extern "C" int b200_attn_sink_prefill_ex(const void* proj, int f32, int64_t ld, int gate_col, const void* k_cache,
@@ -654,10 +675,12 @@ static int attn_sink_decode_launch(const void* proj, int f32, int64_t ld, int ga
                                    const int32_t* seq_lens, int B, const float* sink, void* out, int64_t ldo, int H,
                                    int G, int dk, int dv, int page, float scale, int64_t v_ld, int window,
                                    int gate_per_head, const float* head_scale, const float* pool_k,
-                                   const float* pool_v, int pool, int per_page, const float* init_lse, void* stream) {
+                                   const float* pool_v, int pool, int per_page, const float* init_lse,
+                                    float softcap, void* stream) {
   if (v_ld <= 0) v_ld = dv;
   B200_REQUIRE(pool_k == nullptr || (pool_v != nullptr && window > 0 && pool > 0 && per_page == (page + pool - 1) / pool),
                "attn_sink_decode: pooled blocks need a window, both caches and ceil(page / pool) entries per page");
+  B200_REQUIRE(softcap >= 0.f, "attn_sink_decode: softcap %g is negative", (double)softcap);
   B200_REQUIRE(v_ld >= dv, "attn_sink_decode: value row pitch %lld < dv=%d", (long long)v_ld, dv);
   B200_REQUIRE(H > 0 && G > 0 && H % G == 0 && dk > 0 && dv > 0 && dv <= 32 * kMaxDvLanes && page > 0,
                "attn_sink_decode: bad shape H=%d G=%d dk=%d dv=%d", H, G, dk, dv);
@@ -673,16 +696,27 @@ static int attn_sink_decode_launch(const void* proj, int f32, int64_t ld, int ga
     attn_sink_decode_kernel<TA, V, 16><<<grid, kDecWarps * 32, smem, s>>>(                                       \
         (const TA*)proj, ld, gate_col, (const TA*)k_cache, (const TA*)v_cache, block_table, max_blocks, seq_lens, \
         sink, (TA*)out, ldo, H, G, dk, dv, page, scale, v_ld, window, gate_per_head, head_scale, pool_k, pool_v,  \
-        pool, per_page, init_lse);                                                                               \
+        pool, per_page, init_lse, softcap);                                                                      \
   else                                                                                                           \
     attn_sink_decode_kernel<TA, V, 8><<<grid, kDecWarps * 32, smem, s>>>(                                        \
       (const TA*)proj, ld, gate_col, (const TA*)k_cache, (const TA*)v_cache, block_table, max_blocks, seq_lens,   \
       sink, (TA*)out, ldo, H, G, dk, dv, page, scale, v_ld, window, gate_per_head, head_scale, pool_k, pool_v,    \
-      pool, per_page, init_lse)
+      pool, per_page, init_lse, softcap)
   if (f32) { if (vec) B200_DEC(float, true); else B200_DEC(float, false); }
   else { if (vec) B200_DEC(bf16, true); else B200_DEC(bf16, false); }
 #undef B200_DEC
   return b200_check_launch("b200_attn_sink_decode");
+}
+
+extern "C" int b200_attn_sink_decode_cap(const void* proj, int f32, int64_t ld, int gate_col, const void* k_cache,
+                                          const void* v_cache, const int32_t* block_table, int max_blocks,
+                                          const int32_t* seq_lens, int B, const float* sink, void* out, int64_t ldo, int H,
+                                          int G, int dk, int dv, int page, float scale, int64_t v_ld, int window,
+                                          int gate_per_head, const float* head_scale, const float* pool_k,
+                                          const float* pool_v, int pool, int per_page, float softcap, void* stream) {
+  return attn_sink_decode_launch(proj, f32, ld, gate_col, k_cache, v_cache, block_table, max_blocks, seq_lens, B, sink, out, ldo,
+                                 H, G, dk, dv, page, scale, v_ld, window, gate_per_head, head_scale, pool_k, pool_v, pool,
+                                 per_page, nullptr, softcap, stream);
 }
 
 extern "C" int b200_attn_sink_decode_pool(const void* proj, int f32, int64_t ld, int gate_col, const void* k_cache,
@@ -693,7 +727,7 @@ extern "C" int b200_attn_sink_decode_pool(const void* proj, int f32, int64_t ld,
                                           const float* pool_v, int pool, int per_page, void* stream) {
   return attn_sink_decode_launch(proj, f32, ld, gate_col, k_cache, v_cache, block_table, max_blocks, seq_lens, B, sink, out, ldo,
                                  H, G, dk, dv, page, scale, v_ld, window, gate_per_head, head_scale, pool_k, pool_v, pool,
-                                 per_page, nullptr, stream);
+                                 per_page, nullptr, 0.f, stream);
 }
 
 extern "C" int b200_attn_sink_decode_more(const void* proj, int f32, int64_t ld, const int32_t* block_table, int max_blocks,
@@ -703,7 +737,7 @@ extern "C" int b200_attn_sink_decode_more(const void* proj, int f32, int64_t ld,
   B200_REQUIRE(init_lse != nullptr && pool_k != nullptr, "attn_sink_decode_more: needs the first part's log-sum-exp and pooled blocks");
   // no token is read: the caches' pointers only pass the alignment test of the vector path
   return attn_sink_decode_launch(proj, f32, ld, -1, pool_k, pool_k, block_table, max_blocks, seq_lens, B, nullptr, out, ldo, H, G,
-                                 dk, dv, page, scale, 0, window, 0, head_scale, pool_k, pool_v, pool, per_page, init_lse, stream);
+                                 dk, dv, page, scale, 0, window, 0, head_scale, pool_k, pool_v, pool, per_page, init_lse, 0.f, stream);
 }
 
 extern "C" int b200_attn_sink_decode_ex(const void* proj, int f32, int64_t ld, int gate_col, const void* k_cache,

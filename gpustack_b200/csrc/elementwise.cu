@@ -111,6 +111,7 @@ splitk_reduce_kernel(const float* __restrict__ P, int S, bf16* __restrict__ Y, i
 //     the cross-rank (max, argmax) exchange that serves greedy picks the sampled token.
 //     (Reference: $VLLM/v1/sample/sampler.py draws from softmax(logits / T); nucleus (top_p < 1) rows are
 //     re-sampled by the host path.)  The row seed changes every step (request seed x position).
+//   softcap > 0: every logit first becomes softcap * tanh(logit / softcap) and is written back, in the same pass.
 __device__ __forceinline__ uint32_t fmix32(uint32_t h) {
   h ^= h >> 16; h *= 0x85ebca6bu; h ^= h >> 13; h *= 0xc2b2ae35u; h ^= h >> 16;
   return h;
@@ -122,14 +123,14 @@ __device__ __forceinline__ float gumbel_key(float logit, float inv_t, uint32_t s
 }
 
 __global__ void __launch_bounds__(1024)
-argmax_f32_kernel(const float* __restrict__ logits, int64_t ld, int32_t* __restrict__ out_idx,
+argmax_f32_kernel(float* __restrict__ logits, int64_t ld, int32_t* __restrict__ out_idx,
                   float* __restrict__ out_val, int V, const float* __restrict__ temps,
-                  const uint32_t* __restrict__ seeds, int vocab_offset) {
+                  const uint32_t* __restrict__ seeds, int vocab_offset, float softcap) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float s_val[32];
   __shared__ int s_idx[32];
-  const float* row = logits + (size_t)blockIdx.x * ld;
+  float* row = logits + (size_t)blockIdx.x * ld;
   const float temp = temps ? temps[blockIdx.x] : 0.f;
   const bool sample = temp > 0.f;
   const float inv_t = sample ? 1.f / temp : 1.f;
@@ -140,6 +141,11 @@ argmax_f32_kernel(const float* __restrict__ logits, int64_t ld, int32_t* __restr
   for (int vi = threadIdx.x; vi < nvec; vi += blockDim.x) {
     const float4 v = ld_cg_f4(reinterpret_cast<const float4*>(row) + vi);
     float f[4] = {v.x, v.y, v.z, v.w};
+    if (softcap > 0.f) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) f[j] = softcap * tanhf(f[j] / softcap);
+      reinterpret_cast<float4*>(row)[vi] = make_float4(f[0], f[1], f[2], f[3]);
+    }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int i = vi * 4 + j;
@@ -149,6 +155,7 @@ argmax_f32_kernel(const float* __restrict__ logits, int64_t ld, int32_t* __restr
   }
   for (int i = nvec * 4 + threadIdx.x; i < V; i += blockDim.x) {
     float f = row[i];
+    if (softcap > 0.f) row[i] = f = softcap * tanhf(f / softcap);
     if (sample) f = gumbel_key(f, inv_t, seed, (uint32_t)(vocab_offset + i));
     if (f > best || (f == best && i < best_i)) { best = f; best_i = i; }
   }
@@ -234,18 +241,23 @@ extern "C" int b200_argmax_f32(const float* logits, int64_t ld, int32_t* out_idx
                                int B, int V, void* stream) {
   B200_REQUIRE(B >= 0 && V > 0, "argmax: bad shape");
   if (B == 0) return B200_OK;
-  (void)launch_pdl_cls(kPdlSampler, argmax_f32_kernel, dim3(B), dim3(1024), 0, (cudaStream_t)stream, 1, logits, ld, out_idx,
-                       out_val, V, (const float*)nullptr, (const uint32_t*)nullptr, 0);
+  (void)launch_pdl_cls(kPdlSampler, argmax_f32_kernel, dim3(B), dim3(1024), 0, (cudaStream_t)stream, 1, (float*)logits, ld, out_idx,
+                       out_val, V, (const float*)nullptr, (const uint32_t*)nullptr, 0, 0.f);
   return b200_check_launch("b200_argmax_f32");
 }
 
 // Greedy (temps[b] == 0) or Gumbel-max temperature sampling (temps[b] > 0, seed seeds[b]) of row b in one
 // pass; vocab_offset = global index of column 0 (vocabulary-parallel shards); out_val = the winning key.
-extern "C" int b200_sample_f32(const float* logits, int64_t ld, const float* temps, const uint32_t* seeds,
-                               int vocab_offset, int32_t* out_idx, float* out_val, int B, int V, void* stream) {
-  B200_REQUIRE(B >= 0 && V > 0 && vocab_offset >= 0, "sample: bad shape");
+extern "C" int b200_sample_softcap_f32(float* logits, int64_t ld, float softcap, const float* temps, const uint32_t* seeds,
+                                       int vocab_offset, int32_t* out_idx, float* out_val, int B, int V, void* stream) {
+  B200_REQUIRE(B >= 0 && V > 0 && vocab_offset >= 0 && softcap >= 0.f, "sample: bad shape");
   if (B == 0) return B200_OK;
   (void)launch_pdl_cls(kPdlSampler, argmax_f32_kernel, dim3(B), dim3(1024), 0, (cudaStream_t)stream, 1, logits, ld, out_idx,
-                       out_val, V, temps, seeds, vocab_offset);
+                       out_val, V, temps, seeds, vocab_offset, softcap);
   return b200_check_launch("b200_sample_f32");
+}
+
+extern "C" int b200_sample_f32(const float* logits, int64_t ld, const float* temps, const uint32_t* seeds,
+                               int vocab_offset, int32_t* out_idx, float* out_val, int B, int V, void* stream) {
+  return b200_sample_softcap_f32((float*)logits, ld, 0.f, temps, seeds, vocab_offset, out_idx, out_val, B, V, stream);
 }

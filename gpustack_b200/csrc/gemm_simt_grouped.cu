@@ -13,6 +13,7 @@
 //                 act 1  gelu_tanh(g) * u        gelu_tanh(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
 //                 act 2  g' sigmoid(1.702 g') (u' + 1),  g' = min(g, limit), u' = clamp(u, -limit, limit)
 //                 act 3  silu(g) * u
+//   * act 4 without a gate (W rows as they are): relu(v)^2 of every output, before row_scale;
 //   * any combination (a routed gated expert layer is grouped + gated + gathered).
 // A result element never depends on M, on the row's place in the batch or on the other rows of its tile.
 #include "common.cuh"
@@ -55,7 +56,7 @@ struct GsArgs {
   int n_real;
   int64_t w_expert;                  // elements between the experts' matrices
   const float* row_scale;            // NULL: none
-  int act;                           // 0 = plain linear
+  int act;                           // 0 = plain linear, 1 .. 3 gated, 4 = relu^2 without a gate
   float limit;
   int scale_in;                      // 1: row_scale multiplies the row's INPUT (the accumulators before the activation)
 };
@@ -155,8 +156,10 @@ gemm_simt_grouped_kernel(GsArgs a) {
       if (a.scale_in) {              // W (rs x) = rs (W x): the product is linear in the row
         v *= rs;
         if (GATED) v = gated_act(v, accu[i][j] * rs, a.act, a.limit);
+        else if (a.act == 4) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
       } else {
         if (GATED) v = gated_act(v, accu[i][j], a.act, a.limit);
+        else if (a.act == 4) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
         v *= rs;
       }
       gs_out(Y + (int64_t)m * a.ldy + n, v);
@@ -167,7 +170,7 @@ gemm_simt_grouped_kernel(GsArgs a) {
 template <typename TX, typename TY>
 static int launch_gs(const GsArgs& a, int batch, cudaStream_t s) {
   dim3 grid((a.N + kGsBN - 1) / kGsBN, (a.M + kGsBM - 1) / kGsBM, batch);
-  if (a.act) gemm_simt_grouped_kernel<TX, TY, true><<<grid, 256, 0, s>>>(a);
+  if (a.act >= 1 && a.act <= 3) gemm_simt_grouped_kernel<TX, TY, true><<<grid, 256, 0, s>>>(a);
   else gemm_simt_grouped_kernel<TX, TY, false><<<grid, 256, 0, s>>>(a);
   return b200_check_launch("b200_linear_simt_grouped");
 }
@@ -183,7 +186,7 @@ extern "C" int b200_linear_simt_grouped_ex(const void* X, int x_f32, const void*
                                            int act, float limit, int scale_in, void* stream) {
   B200_REQUIRE(M >= 0 && N > 0 && K > 0 && batch >= 1, "linear_simt_grouped: bad shape M=%d N=%d K=%d batch=%d", M, N, K, batch);
   B200_REQUIRE(ldx >= K && ldw >= K && ldy >= N, "linear_simt_grouped: leading dimensions too small");
-  B200_REQUIRE(act >= 0 && act <= 3, "linear_simt_grouped: unknown activation %d", act);
+  B200_REQUIRE(act >= 0 && act <= 4, "linear_simt_grouped: unknown activation %d", act);
   B200_REQUIRE(tile_expert == nullptr || (num_tiles != nullptr && M % kGsBM == 0), "linear_simt_grouped: grouped rows come in tiles of %d", kGsBM);
   B200_REQUIRE(row_pair == nullptr || top_k >= 1, "linear_simt_grouped: top_k");
   if (M == 0) return B200_OK;

@@ -1113,6 +1113,7 @@ extern "C" int b200_moe_grouped_gemm(const void* X, const void* W, void* Y, int 
 
 // The same with the options of the other routed designs: gated != 0 applies gated_pair(act, limit) over interleaved
 // gate / up rows (Y [capacity_rows, N/2] bf16); otherwise Y is bf16 or, out_f32 != 0, fp32, times row_scale if given.
+// act 4 without a gate: relu(v)^2 of every output (bf16 out, no row_scale).
 // Tiles whose expert index is >= num_experts read weight rows beyond the stack (zeros): their output is not used.
 extern "C" int b200_moe_grouped_gemm_ex(const void* X, const void* W, void* Y, int capacity_rows, int N, int K,
                                         int num_experts, int64_t ldx, int64_t ldw, int64_t ldy, const float* row_scale,
@@ -1131,7 +1132,8 @@ extern "C" int b200_moe_grouped_gemm_ex(const void* X, const void* W, void* Y, i
     return B200_ERR_UNSUPPORTED;
   }
   cudaStream_t s = (cudaStream_t)stream;
-  const int fl = gated ? gated_flags(act, limit) : (out_f32 ? 1 : 0);
+  B200_REQUIRE(gated || act != 4 || (row_scale == nullptr && !out_f32), "moe_grouped_gemm: relu^2 output is bf16 without row_scale");
+  const int fl = gated ? gated_flags(act, limit) : ((out_f32 ? 1 : 0) | (act == 4 ? 2 : 0));
 #define B200_GRPX_CASE(BX)                                                                                        \
   case BX:                                                                                                        \
     return gated ? launch_gemm_grouped<BX, 1>(X, W, Y, capacity_rows, N, K, num_experts, ldx, ldw, ldy, nullptr,   \

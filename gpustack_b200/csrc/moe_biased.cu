@@ -5,6 +5,8 @@
 //                      s / (sum of the chosen s + 1e-20) * scale -- the correction steers the choice only.
 //   moe_route_scored:  the same with two options: s = sigmoid(z) per output instead of the softmax, and weights that
 //                      are the chosen scores as they are (times scale), not renormalised.
+//                      A third form chooses by z + correction (here the router's learned bias, part of the logit) and
+//                      weights with the softmax over the chosen logits alone.
 //   moe_combine_mixed: out[t] = sum_j ( id_j < n_real ? yp[pair_row[t K + j]] : w_j * x[t] ) (+ shared[t]).
 //                      Routed rows arrive already multiplied by their weight (the down projection's row
 //                      scale); an identity expert returns the layer input itself times the weight.  fp32 sum in a
@@ -29,7 +31,7 @@ __device__ __forceinline__ float rb_f32(bf16 v) { return __bfloat162float(v); }
 __global__ void __launch_bounds__(128)
 moe_route_biased_kernel(const float* __restrict__ logits, int64_t ld, const float* __restrict__ correction,
                         int32_t* __restrict__ topk_ids, float* __restrict__ topk_w, int T, int E, int K, float scale,
-                        int sigmoid_scores, int renormalize) {
+                        int score_mode, int renormalize) {
   const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (t >= T) return;
   float s[kRbPerLane], c[kRbPerLane];
@@ -41,7 +43,15 @@ moe_route_biased_kernel(const float* __restrict__ logits, int64_t ld, const floa
     mx = fmaxf(mx, s[i]);
   }
   mx = warp_max(mx);
-  if (sigmoid_scores) {
+  if (score_mode == 2) {
+    // the biased logits themselves are chosen from and go into the softmax over the chosen (below)
+#pragma unroll
+    for (int i = 0; i < kRbPerLane; ++i) {
+      const int e = lane + 32 * i;
+      if (e < E && correction != nullptr) s[i] += correction[e];
+      c[i] = e < E ? s[i] : -CUDART_INF_F;
+    }
+  } else if (score_mode == 1) {
     // every output scored on its own; without a correction the choice is made on the logits themselves (the
     // sigmoid is monotone, and two large logits must not tie where it saturates)
 #pragma unroll
@@ -67,7 +77,7 @@ moe_route_biased_kernel(const float* __restrict__ logits, int64_t ld, const floa
       c[i] = e < E ? s[i] + (correction != nullptr ? correction[e] : 0.f) : -CUDART_INF_F;
     }
   }
-  float wsum = 0.f, mine_w = 0.f;
+  float wsum = 0.f, mine_w = 0.f, top_z = 0.f;
   int mine_id = 0;
   for (int j = 0; j < K; ++j) {
     float bv = -CUDART_INF_F, bs = 0.f;
@@ -87,6 +97,10 @@ moe_route_biased_kernel(const float* __restrict__ logits, int64_t ld, const floa
 #pragma unroll
     for (int i = 0; i < kRbPerLane; ++i)
       if (lane + 32 * i == be) c[i] = -CUDART_INF_F;                   // taken
+    if (score_mode == 2) {                                             // the first choice is the largest logit
+      if (j == 0) top_z = bs;
+      bs = expf(bs - top_z);
+    }
     wsum += bs;
     if (lane == j) { mine_id = be; mine_w = bs; }
   }
@@ -121,14 +135,15 @@ moe_combine_mixed_kernel(const TP* __restrict__ yp, int64_t ldp, const int32_t* 
 using namespace b200;
 
 extern "C" int b200_moe_route_scored(const float* logits, int64_t ld, const float* correction, int32_t* topk_ids,
-                                     float* topk_w, int T, int E, int K, float scale, int sigmoid_scores,
+                                     float* topk_w, int T, int E, int K, float scale, int score_mode,
                                      int renormalize, void* stream) {
   B200_REQUIRE(ld >= E, "moe_route_biased: row stride %lld < E=%d", (long long)ld, E);
   B200_REQUIRE(T >= 0 && E >= 1 && E <= 32 * kRbPerLane && K >= 1 && K <= kRbMaxTop && K <= E,
                "moe_route_biased: unsupported E=%d K=%d (E <= %d, K <= %d)", E, K, 32 * kRbPerLane, kRbMaxTop);
+  B200_REQUIRE(score_mode >= 0 && score_mode <= 2, "moe_route_biased: unknown score form %d", score_mode);
   if (T == 0) return B200_OK;
   moe_route_biased_kernel<<<(T + 3) / 4, 128, 0, (cudaStream_t)stream>>>(logits, ld, correction, topk_ids, topk_w, T, E, K,
-                                                                       scale, sigmoid_scores, renormalize);
+                                                                       scale, score_mode, renormalize);
   return b200_check_launch("b200_moe_route_biased");
 }
 

@@ -1,4 +1,5 @@
-"""Model runner of the layer-list decoders (config.LayerListConfig: Vodavik, Danipel, Resevik, Dotorax).
+"""Model runner of the layer-list decoders (config.LayerListConfig: Vodavik, Danipel, Resevik, Dotorax,
+Kerarax).
 
 Same step interface as runner.ModelRunner -- the engine, the scheduler's plans, the staging buffer, CUDA-graph
 decode steps and the sampler are shared -- with this family's layer sequence:
@@ -26,6 +27,11 @@ decode steps and the sampler are shared -- with this family's layer sequence:
   attention mixer with rotation: rot_prep (rotation, weightless q / k norm, keys to their pages, values = the keys
                    as projected) -> the same attention kernels, with a sliding window.
 
+  attention mixer with convolved q, k, v:  ONE conv_attn_prep launch -- causal convolution of the projected rows (ring of the
+                   last projected rows per sequence), head norms, keys and values to their pages -- then the same attention
+                   kernels with capped scores and one more in the softmax denominator.  In bf16 the heads are laid out at a
+                   tensor-core tile width (zero columns behind dim / vdim), whatever dim and vdim are.
+
 Residual schemes (config.residual): "post_ln" as drawn above; "parallel": pre-norm with ONE RMS norm per layer,
 
     embed * scale -> per layer run [ x += branches of the layer before (+ embedding before a repeated pass) ; h = RMSnorm(x)
@@ -47,7 +53,13 @@ where ONE sandwich_join launch does the sum (with the post-norm of the output) a
 convolution with its per-sequence ring follows.  Its mixers: rotary attention with one gate per head; a side-by-side
 pair of [sliding-window attention that also sees the pooled blocks before the window | gated diagonal recurrence behind a
 short convolution], whose two output projections meet in the join with their factors; gated linear attention with a
-decay per key channel and token.
+decay per key channel and token.  "output_norm": a norm on every sublayer's output and none in front,
+
+    LN(embed + sinusoid) -> per sublayer [ x += LN(output of the sublayer before) ; xb = x rounded -> sublayer ]
+          -> x += LN(last output) -> LN of the wanted rows -> lm_head -> capped logits (in the sampler's pass)
+
+where ONE output_norm_join launch does the norm, the sum and the rounding -- for a routed feed-forward also the sum over
+the chosen experts and the gated shared expert.
 
 Feed-forwards:
 relu^2 (ungated), gated GELU, a clamped gated unit, or a routed mixture of clamped gated experts with identity experts
@@ -66,6 +78,7 @@ import torch
 from . import ops
 from .lib import B200Error
 from .runner import BF16, ModelRunner
+from .weights import pad_head_columns
 
 
 class LayerListRunner(ModelRunner):
@@ -84,7 +97,8 @@ class LayerListRunner(ModelRunner):
         attn = [(l, x.mixer.left if x.mixer.kind == "side_by_side" else x.mixer) for l, x in enumerate(cfg.layers)
                 if x.mixer.kind in ("attention", "side_by_side")]
         self.fast_decode = {l: bf and m.tile_sized for l, m in attn}
-        self.fast_prefill = {l: bf and m.tile_sized and ops.attn_prefill_tc_covers(m.heads, m.kv_heads, m.dim) for l, m in attn}
+        self.fast_prefill = {l: bf and m.tile_sized and ops.attn_prefill_tc_covers(m.heads, m.kv_heads, m.cache_widths(bf)[0])
+                             for l, m in attn}
         base = ops.attn_sink_prefill_tile()
         # ONE tile list serves every layer of a step: the tile size most tensor-core layers want (ties: the larger)
         tiles = [ops.attn_prefill_tile(m.heads, m.kv_heads) for l, m in attn
@@ -105,6 +119,7 @@ class LayerListRunner(ModelRunner):
         self.streams = cfg.residual == "streams"
         self.parallel = cfg.residual == "parallel"
         self.sandwich = cfg.residual == "sandwich"
+        self.output_norm = cfg.residual == "output_norm"
         self.canon_taps = getattr(cfg, "canon_taps", 0)
         self.runs = cfg.runs()                 # [(layer, embedding added before it)]: caches and state belong to a run
         self.looped = any(again for _, again in self.runs)
@@ -112,6 +127,12 @@ class LayerListRunner(ModelRunner):
         self.S = cfg.n_streams if self.streams else 1
         self.proj_width = max(lw.proj.shape[0] for lw in self.w.layers)
         self.mix_width = max(l.mixer.out_width for l in cfg.layers)
+        # attention over convolved q, k, v: prepared queries in rows of their own, heads at the cache's widths
+        conv = [(l, x.mixer) for l, x in enumerate(cfg.layers) if x.mixer.kind == "attention" and x.mixer.conv_taps]
+        self.q_rows_width = max([m.heads * m.cache_widths(bf)[0] for _, m in conv] or [0])
+        self.mix_width = max([self.mix_width] + [m.heads * m.cache_widths(bf)[1] for _, m in conv])
+        self.o_padded = {l: pad_head_columns(self.w.layers[l].o, m.heads, m.vdim, m.cache_widths(bf)[1]) for l, m in conv
+                         if m.cache_widths(bf)[1] != m.vdim}
         self.ff_width = max([(l.mlp.moe.shared_ff if l.mlp.kind == "moe" else l.mlp.ff) for l in cfg.layers
                              if l.mlp is not None] or [0])
         lat = [l.mixer for l in cfg.layers if l.mixer.kind == "latent_attention"]
@@ -144,6 +165,7 @@ class LayerListRunner(ModelRunner):
         self.y = e(T, D, dt=torch.float32)                # a sublayer's output: fp32 into the residual sum
         self.proj = e(T * self.proj_width, dt=a)          # flat; viewed [T, rows of this layer's fused projection]
         self.mix_out = e(T * self.mix_width, dt=a)
+        self.q_rows = e(T * max(1, self.q_rows_width), dt=a)
         self.act = e(T * max(1, self.ff_width), dt=a)
         self.gates = e(T * max(1, self.gate_width), dt=torch.float32)
         self.o_raw = e(T * max(1, self.rec_width), dt=torch.float32)
@@ -164,7 +186,7 @@ class LayerListRunner(ModelRunner):
         self.routed_ws = None
         if self.routed:
             self.routed_ws = ops.RoutedWorkspace(T, max(r.top for r in self.routed),
-                                                 max(r.experts + r.identity for r in self.routed), D,
+                                                 max(r.experts + r.identity + r.shared_gate for r in self.routed), D,
                                                  max(r.ff for r in self.routed), a, dev)
 
     def _alloc_step_io(self):
@@ -189,9 +211,10 @@ class LayerListRunner(ModelRunner):
                 self.pool_k[l] = torch.zeros(num_blocks, m.kv_heads, per_page, m.dim, dtype=torch.float32, device=self.device)
                 self.pool_v[l] = torch.zeros(num_blocks, m.kv_heads, per_page, m.vdim, dtype=torch.float32, device=self.device)
             if m.kind == "attention" and m.kv_from is None:
-                self.k_cache[l] = torch.zeros(num_blocks, m.kv_heads, self.block_size, m.dim, dtype=self.act_dtype,
+                wk, wv = m.cache_widths(self.act_dtype == BF16)
+                self.k_cache[l] = torch.zeros(num_blocks, m.kv_heads, self.block_size, wk, dtype=self.act_dtype,
                                               device=self.device)
-                self.v_cache[l] = torch.zeros(num_blocks, m.kv_heads, self.block_size, m.vdim, dtype=self.act_dtype,
+                self.v_cache[l] = torch.zeros(num_blocks, m.kv_heads, self.block_size, wv, dtype=self.act_dtype,
                                               device=self.device)
             elif m.kind == "latent_attention":
                 # ONE row per token for all heads: [latent: kv_rank | rotated key part: rot_dim]; the values are its head
@@ -214,6 +237,8 @@ class LayerListRunner(ModelRunner):
             m = self.mcfg.layers[li].mixer
             if R > 0:        # the last inputs of the mixer's and the feed-forward's convolution, by position mod R
                 self.canon_ring[l] = (f(num_slots, R, D), f(num_slots, R, D) if self.mcfg.layers[li].mlp is not None else None)
+            if m.kind == "attention" and m.conv_taps > 1:    # ring of the last projected rows, by position mod (taps - 1)
+                self.state[l] = (f(num_slots, m.conv_taps - 1, m.qkv_width),)
             if m.kind == "side_by_side":             # S [slots, W], and the ring of its convolution's last inputs
                 r = m.right
                 self.state[l] = (f(num_slots, r.width), f(num_slots, r.conv - 1, r.width) if r.conv > 1 else None)
@@ -244,6 +269,12 @@ class LayerListRunner(ModelRunner):
                 ops.embed_pos(ids, self._pos[:T], self.w.embed, self.w.pos, self.resid32[:T])
             else:
                 ops.embed_streams(ids, self.w.embed, self.resid32[:T], 1, self.mcfg.embed_scale)
+            self._pending = None
+            self.stats["kernel_launches"] += 1
+            return
+        if self.output_norm:
+            ops.embed_sinusoid(ids, self._pos[:T], self.w.embed, self.w.pos_freq, self.resid32[:T],
+                               norm=(self.w.embed_norm, self.w.embed_norm_b), eps=self.mcfg.norm_eps, xb_out=self.xb[:T])
             self._pending = None
             self.stats["kernel_launches"] += 1
             return
@@ -302,6 +333,14 @@ class LayerListRunner(ModelRunner):
         self._pending = None
         self.layer_trace.append(self.resid32[:T].clone())
 
+    def _take_output(self, T: int) -> None:
+        """Output-norm residual: the output of the sublayer before (self._pending = the join's arguments) enters the fp32
+        stream through its norm, and the stream's rounded copy is the next sublayer's input."""
+        if self._pending is not None:
+            ops.output_norm_join(self.resid32[:T], self.mcfg.norm_eps, x_out=self.resid32[:T], h_out=self.xb[:T], **self._pending)
+            self._pending = None
+            self.stats["kernel_launches"] += 1
+
     def _join(self, T: int, l: int, q: int) -> None:
         """The branch output self.y of sublayer q (1 mixer, 2 feed-forward) of layer l enters the residual, and the
         next sublayer's input is prepared in self.xb."""
@@ -331,12 +370,13 @@ class LayerListRunner(ModelRunner):
         self-resetting workspace per head shape, sized for the largest batch."""
         span = min(self.max_model_len, m.window) if m.window else self.max_model_len    # keys a row can see
         splits = ops.attn_decode_splits(B, m.kv_heads, span)
-        key = (m.heads, m.kv_heads, m.dim, span)
+        width = m.cache_widths(True)[0]
+        key = (m.heads, m.kv_heads, width, span)
         if key not in self._dec_ws:
             from .lib import load
 
             L = load()
-            need = max(L.b200_attn_decode_workspace_bytes(b, m.heads, m.dim, ops.attn_decode_splits(b, m.kv_heads, span))
+            need = max(L.b200_attn_decode_workspace_bytes(b, m.heads, width, ops.attn_decode_splits(b, m.kv_heads, span))
                        for b in range(1, self.max_seqs + 1))
             self._dec_ws[key] = torch.zeros((need + 3) // 4, dtype=torch.float32, device=self.device)
         return splits, self._dec_ws[key]
@@ -365,6 +405,8 @@ class LayerListRunner(ModelRunner):
             out = self._view(self.mix_out, T, m.out_width)
             if self.parallel:
                 self._open_layer(T, l, lw, again)
+            if self.output_norm:
+                self._take_output(T)
             if self.sandwich:
                 ring = self.canon_ring[l] or (None, None)
                 self._sandwich_open(T, lw.norm1, lw.canon1, ring[0], cu_all, ctx_all, slots_all)
@@ -399,7 +441,16 @@ class LayerListRunner(ModelRunner):
             elif m.kind == "attention":
                 own = m.kv_from is None
                 H, G, dk, dv = m.heads, m.kv_heads, m.dim, m.vdim
-                if m.rot is not None or m.values_are_keys or m.qk_unit_norm:
+                q, wo = proj, lw.o                # rows that start with the queries; the output projection
+                if m.conv_taps:
+                    wk, wv = self.k_cache[l].shape[3], self.v_cache[l].shape[3]
+                    q, out = self._view(self.q_rows, T, H * wk), self._view(self.mix_out, T, H * wv)
+                    wo = self.o_padded.get(li, wo)
+                    ops.conv_attn_prep(proj, lw.conv_w, lw.q_norm, lw.k_norm, self.state[l][0] if self.state[l] else None, cu_all,
+                                       ctx_all, slots_all, ts, tq, self.prefill_tile, cu_p.shape[0] - 1 if nt else 0, Bd, slots, q,
+                                       self.k_cache[l], self.v_cache[l], H, G, dk, dv, eps)
+                    dk, dv = wk, wv
+                elif m.rot is not None or m.values_are_keys or m.qk_unit_norm:
                     # rotation, then the weightless q / k norm; keys to their pages, values = the keys as projected
                     # (a layer that reads another layer's cache prepares its queries only)
                     ops.rot_prep(proj, 0, H * dk, -1 if m.values_are_keys else (H + G) * dk, pos, slots, proj,
@@ -414,22 +465,23 @@ class LayerListRunner(ModelRunner):
                 gate_col = (H * dk + kv_cols) if m.gate else -1
                 kc, vc = self.k_cache[l], self.v_cache[l]
                 if nt and self.fast_prefill[li]:
-                    ops.paged_attn_prefill_ex(proj[:Tp], proj.stride(0), kc, vc, bt_p, cu_p, ctx_p, ts, tq, out[:Tp], H, G, dk,
+                    ops.paged_attn_prefill_ex(q[:Tp], q.stride(0), kc, vc, bt_p, cu_p, ctx_p, ts, tq, out[:Tp], H, G, dk,
                                               m.scale, sink=lw.sink, gate=proj[:Tp, gate_col:] if m.gate else None,
-                                              window=m.window, gate_per_head=m.gate_per_head)
+                                              window=m.window, gate_per_head=m.gate_per_head, softcap=m.softcap)
                 elif nt:
-                    ops.attn_sink_prefill(proj[:Tp], gate_col, kc, vc, bt_p, cu_p, ctx_p, ts, tq, lw.sink, out[:Tp],
+                    ops.attn_sink_prefill(q[:Tp], gate_col, kc, vc, bt_p, cu_p, ctx_p, ts, tq, lw.sink, out[:Tp],
                                           H, G, dk, dv, m.scale, tile_rows=self.prefill_tile, window=m.window,
-                                          gate_per_head=m.gate_per_head, head_scale=lw.head_scale)
+                                          gate_per_head=m.gate_per_head, head_scale=lw.head_scale, softcap=m.softcap)
                 if Bd and self.fast_decode[li]:
                     splits, ws = self._decode_plan(Bd, m)
-                    ops.paged_attn_decode(proj[Tp:T], proj.stride(0), kc, vc, bt_d, lens_d, out[Tp:T], H, G, dk, m.scale,
+                    ops.paged_attn_decode(q[Tp:T], q.stride(0), kc, vc, bt_d, lens_d, out[Tp:T], H, G, dk, m.scale,
                                           num_splits=splits, workspace=ws, sink=lw.sink,
                                           gate=proj[Tp:T, gate_col:] if m.gate else None, window=m.window,
-                                          gate_per_head=m.gate_per_head)
+                                          gate_per_head=m.gate_per_head, softcap=m.softcap)
                 elif Bd:
-                    ops.attn_sink_decode(proj[Tp:T], gate_col, kc, vc, bt_d, lens_d, lw.sink, out[Tp:T], H, G, dk, dv,
-                                         m.scale, window=m.window, gate_per_head=m.gate_per_head, head_scale=lw.head_scale)
+                    ops.attn_sink_decode(q[Tp:T], gate_col, kc, vc, bt_d, lens_d, lw.sink, out[Tp:T], H, G, dk, dv,
+                                         m.scale, window=m.window, gate_per_head=m.gate_per_head, head_scale=lw.head_scale,
+                                         softcap=m.softcap)
                 self.stats["kernel_launches"] += 2 + (1 if nt else 0) + (1 if Bd else 0)
             elif m.kind == "linear_attention":
                 H, dk, dv = m.heads, m.dim, m.vdim
@@ -454,8 +506,17 @@ class LayerListRunner(ModelRunner):
                                o_raw, H, dk, dv, m.gate_cap, max_len=Tp if Tp else 1)
                 ops.mlstm_out(o_raw, proj, 2 * H * dk + H * dv, lw.out_norm, out, H, dv, eps)
                 self.stats["kernel_launches"] += 4
-            ops.linear(out, lw.o, self.y[:T])
+            ops.linear(out, wo if m.kind == "attention" else lw.o, self.y[:T])
             self.stats["kernel_launches"] += 1
+            if self.output_norm:
+                self._pending = {"y": self.y[:T], "post": (lw.norm1, lw.norm1_b)}
+                if layer.mlp is not None:
+                    self._take_output(T)
+                    self._pending = {"routed": self._routed_rows(T, layer.mlp.moe, lw), "post": (lw.norm2, lw.norm2_b)}
+                if self.layer_trace is not None:       # (the serving path leaves the last output to the final norm)
+                    self._take_output(T)
+                    self.layer_trace.append(self.resid32[:T].clone())
+                continue
             if self.sandwich:
                 self._pending = (self.y[:T], None, 1.0, 1.0, lw.norm1b)
                 if layer.mlp is not None:
@@ -575,6 +636,22 @@ class LayerListRunner(ModelRunner):
         ops.head_linear(o_lat, lw.uv, out, H, n=dv, k=R, x_head=R, out_head=dv)
         self.stats["kernel_launches"] += 3 + (1 if nt else 0) + (1 if Bd else 0)
 
+    def _routed_rows(self, T: int, e, lw) -> tuple:
+        """Routed feed-forward of self.xb[:T] up to, but without, the sum over a token's rows: (expert rows, row of each
+        (token, choice), choices, shared expert's rows, its gate's logits), the `routed` argument of output_norm_join."""
+        x, ws = self.xb[:T], self.routed_ws
+        shared = gate = None
+        if e.shared_ff:
+            act, shared = self._view(self.act, T, e.shared_ff), ws.shared[:T]
+            ops.linear(x, lw.shared13, act, relu2=True)
+            ops.linear(act, lw.shared2, shared)
+            gate = ws.logits[:T, e.experts] if e.shared_gate else None     # the router product's row behind the outputs
+            self.stats["kernel_launches"] += 2
+        ops.routed_experts(x, lw.router, lw.correction, lw.w13, lw.w2, ws, None, e.experts, 0, e.top, e.scale, e.ff, e.limit,
+                           renormalize=e.renormalize, act=e.act, score=e.score, combine=False)
+        self.stats["kernel_launches"] += ops.ROUTED_LAUNCHES - 1
+        return ws.yp, ws.pair_row, e.top, shared, gate
+
     def _feed_forward(self, T: int, mlp, lw, y=None) -> None:
         """self.xb[:T] -> y (fp32; self.y[:T] unless given)."""
         y = self.y[:T] if y is None else y
@@ -629,6 +706,9 @@ class LayerListRunner(ModelRunner):
             y, y2, ya, yb, post_w = self._pending if self._pending is not None else (None, None, 1.0, 1.0, None)
             ops.sandwich_join(self.resid32, cfg.norm_eps, y=y, y2=y2, ya=ya, yb=yb, post_w=post_w, mult=cfg.residual_mult,
                               pre_w=self.w.final_norm, rows=rows, h_out=self.x_last[:n])
+        elif self.output_norm:   # likewise: the last output's norm, the sum and the final norm in one pass
+            ops.output_norm_join(self.resid32, cfg.norm_eps, rows=rows, final=(self.w.final_norm, self.w.final_norm_b),
+                                 h_out=self.x_last[:n], **(self._pending or {}))
         elif self.parallel:      # the last layer's branch outputs enter the sum here, for the wanted rows only
             a, b = self._pending
             ops.add_rms_norm(self.resid32, self.w.final_norm, cfg.norm_eps, a=a, b=b, rows=rows, xb_out=self.x_last[:n])
@@ -640,7 +720,7 @@ class LayerListRunner(ModelRunner):
                                out_scale=cfg.logit_scale)
         lg = self.logits[:n]
         ops.linear(self.x_last[:n], self.w.lm_head, lg)
-        ops.sample(lg, temps, seeds, out_idx=self.out_ids[:n])
+        ops.sample(lg, temps, seeds, out_idx=self.out_ids[:n], softcap=cfg.logit_softcap)
         self.stats["kernel_launches"] += 3
 
 

@@ -164,6 +164,20 @@ SIGNATURES = {
                                                   _i32, _i32, _f32, _i32, _i32, _vp, _i64, _vp]),
     "b200_gla_scan": (_i32, [_vp, _i64, _i32, _i32, _i32, _vp, _i64, _f32, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32,
                              _vp]),
+    "b200_attn_sink_prefill_cap": (_i32, [_vp, _i32, _i64, _i32, _vp, _vp, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _i32, _vp, _vp, _i64,
+                   _i32, _i32, _i32, _i32, _i32, _f32, _i64, _i32, _i32, _vp, _vp, _vp, _i32, _i32, _f32, _vp]),
+    "b200_attn_sink_decode_cap": (_i32, [_vp, _i32, _i64, _i32, _vp, _vp, _vp, _i32, _vp, _i32, _vp, _vp, _i64, _i32, _i32, _i32, _i32,
+                   _i32, _f32, _i64, _i32, _i32, _vp, _vp, _vp, _i32, _i32, _f32, _vp]),
+    "b200_paged_attn_prefill_cap": (_i32, [_vp, _i64, _i32, _vp, _vp, _i32, _vp, _i32, _vp, _vp, _vp, _vp, _i32, _vp, _i32, _i32, _i32,
+                   _i32, _f32, _vp, _vp, _i64, _i32, _i32, _vp, _f32, _vp]),
+    "b200_paged_attn_decode_cap": (_i32, [_vp, _i64, _vp, _vp, _vp, _i32, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _vp,
+                   _vp, _i64, _i32, _i32, _vp, _f32, _vp]),
+    "b200_output_norm_join": (_i32, [_vp, _vp, _vp, _vp, _i32, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32,
+                                     _f32, _vp]),
+    "b200_embed_sinusoid": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _f32, _vp]),
+    "b200_conv_attn_prep": (_i32, [_vp, _i32, _i64, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _vp,
+                                   _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _vp]),
+    "b200_sample_softcap_f32": (_i32, [_vp, _i64, _f32, _vp, _vp, _i32, _vp, _vp, _i32, _i32, _vp]),
     "b200_gla_scan_rows": (_i32, [_vp, _i64, _i32, _i32, _i32, _vp, _i64, _f32, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32,
                              _i32, _vp]),
 }

@@ -143,14 +143,15 @@ def argmax(logits, out_idx=None, out_val=None):
     return idx
 
 
-def sample(logits, temps, seeds, out_idx=None, out_val=None, vocab_offset: int = 0):
+def sample(logits, temps, seeds, out_idx=None, out_val=None, vocab_offset: int = 0, softcap: float = 0.0):
     """Greedy (temps == 0) or Gumbel-max temperature sampling per row in ONE pass over the logits.
+    softcap > 0: the logits become softcap * tanh(logit / softcap) first, in place, in the same pass.
     temps: fp32 [B]; seeds: int32/uint32 [B] (bit patterns); returns int32 token ids (shard-local)."""
     _req(logits, torch.float32, "logits"); _req(temps, torch.float32, "temps"); _req(seeds, torch.int32, "seeds")
     B, V = logits.shape
     idx = torch.empty((B,), dtype=torch.int32, device=logits.device) if out_idx is None else out_idx
-    check(load().b200_sample_f32(_p(logits), logits.stride(0), _p(temps), _p(seeds), vocab_offset, _p(idx), _p(out_val),
-                                 B, V, _stream()), "sample")
+    check(load().b200_sample_softcap_f32(_p(logits), logits.stride(0), softcap, _p(temps), _p(seeds), vocab_offset, _p(idx),
+                                         _p(out_val), B, V, _stream()), "sample")
     return idx
 
 
@@ -368,19 +369,20 @@ def attn_decode_workspace(B, Hq, D, num_splits, device) -> torch.Tensor:
 
 def paged_attn_decode(q, q_stride, k_cache, v_cache, block_table, seq_lens, out, Hq, Hkv, D, scale,
                       num_splits=1, workspace=None, sink=None, gate=None, window: int = 0, gate_per_head: bool = False,
-                      lse_out=None):
+                      lse_out=None, softcap: float = 0.0):
     """q: [B, >=Hq*D] view into the qkv buffer (row stride q_stride elements).  sink [Hq] fp32: softmax sink;
     gate [B, >=Hq*D] bf16 view (same row stride rule): the output is multiplied by sigmoid(gate) -- with gate_per_head
-    the view holds ONE number per head, [B, >=Hq]; window > 0: the row at position n - 1 sees keys [n - window, n)."""
+    the view holds ONE number per head, [B, >=Hq]; window > 0: the row at position n - 1 sees keys [n - window, n);
+    softcap > 0: the scaled score passes softcap * tanh(score / softcap)."""
     B = seq_lens.shape[0]
     _req(block_table, torch.int32, "block_table"); _req(seq_lens, torch.int32, "seq_lens")
     if lse_out is not None:       # fp32 [B, Hq]: every row's log-sum-exp, for attn_sink_decode_more
         _req(lse_out, torch.float32, "lse_out")
-    check(load().b200_paged_attn_decode_lse(_p(q), q_stride, _p(k_cache), _p(v_cache), _p(block_table),
+    check(load().b200_paged_attn_decode_cap(_p(q), q_stride, _p(k_cache), _p(v_cache), _p(block_table),
                                             block_table.shape[1], _p(seq_lens), _p(out), _p(workspace),
                                             num_splits, B, Hq, Hkv, D, k_cache.shape[2], scale, _p(sink), _p(gate),
                                             0 if gate is None else gate.stride(0), int(window), 1 if gate_per_head else 0,
-                                            _p(lse_out), _stream()), "paged_attn_decode")
+                                            _p(lse_out), softcap, _stream()), "paged_attn_decode")
     return out
 
 
@@ -409,17 +411,19 @@ def attn_prefill_tc_covers(Hq, Hkv, D) -> bool:
 
 
 def paged_attn_prefill_ex(q, q_stride, k_cache, v_cache, block_table, cu_q, ctx_lens, tile_seq, tile_q0, out, Hq, Hkv, D,
-                          scale, sink=None, gate=None, window: int = 0, gate_per_head: bool = False, lse_out=None):
+                          scale, sink=None, gate=None, window: int = 0, gate_per_head: bool = False, lse_out=None,
+                          softcap: float = 0.0):
     """The tcgen05 prefill kernel with a softmax sink ([Hq] fp32), a sigmoid output gate (bf16 view [T, >=Hq*D], or
     [T, >=Hq] with gate_per_head: one number per head) and / or a sliding window (position i sees j with
-    0 <= i - j < window); only for shapes attn_prefill_tc_covers() accepts, tiles of attn_prefill_tile(Hq, Hkv) rows."""
+    0 <= i - j < window) and / or a soft cap on the scaled score; only for shapes attn_prefill_tc_covers() accepts, tiles of attn_prefill_tile(Hq, Hkv) rows."""
     if lse_out is not None:       # fp32 [T, Hq]: every row's log-sum-exp, for attn_sink_prefill_more
         _req(lse_out, torch.float32, "lse_out")
-    check(load().b200_paged_attn_prefill_lse(_p(q), q_stride, q.shape[0], _p(k_cache), _p(v_cache), k_cache.shape[0],
+    check(load().b200_paged_attn_prefill_cap(_p(q), q_stride, q.shape[0], _p(k_cache), _p(v_cache), k_cache.shape[0],
                                              _p(block_table), block_table.shape[1], _p(cu_q), _p(ctx_lens), _p(tile_seq),
                                              _p(tile_q0), tile_seq.shape[0], _p(out), Hq, Hkv, D, k_cache.shape[2], scale,
                                              _p(sink), _p(gate), 0 if gate is None else gate.stride(0), int(window),
-                                             1 if gate_per_head else 0, _p(lse_out), _stream()), "paged_attn_prefill_ex")
+                                             1 if gate_per_head else 0, _p(lse_out), softcap, _stream()),
+          "paged_attn_prefill_ex")
     return out
 
 
@@ -548,7 +552,7 @@ def _pool_args(pool, k_cache, dk, dv):
 
 def attn_sink_prefill(proj, gate_col, k_cache, v_cache, block_table, cu_q, ctx_lens, tile_seq, tile_q0, sink, out,
                       H, G, dk, dv, scale, tile_rows: int = 0, v_ld: int = 0, window: int = 0, gate_per_head: bool = False,
-                      head_scale=None, pool=None):
+                      head_scale=None, pool=None, softcap: float = 0.0):
     """v_ld: elements between value rows (0 = dv); v_cache is k_cache and v_ld == dk when the values are the
     first dv entries of the key rows (a latent cache).  window > 0: position i sees j with 0 <= i - j < window.
     gate_per_head: the gate is ONE column per head at gate_col; head_scale: fp32 [H] factors on the score;
@@ -558,11 +562,11 @@ def attn_sink_prefill(proj, gate_col, k_cache, v_cache, block_table, cu_q, ctx_l
     if k_cache.dtype != proj.dtype or out.dtype != proj.dtype:
         raise B200Error("attn_sink_prefill: projection, cache and output must share one element type")
     pk, pv, pn, ppp = _pool_args(pool, k_cache, dk, dv)
-    check(load().b200_attn_sink_prefill_pool(_p(proj), _is_f32(proj), proj.stride(0), gate_col, _p(k_cache), _p(v_cache),
+    check(load().b200_attn_sink_prefill_cap(_p(proj), _is_f32(proj), proj.stride(0), gate_col, _p(k_cache), _p(v_cache),
                                              _p(block_table), block_table.shape[1], _p(cu_q), _p(ctx_lens), _p(tile_seq),
                                              _p(tile_q0), tile_seq.shape[0], tile_rows or attn_sink_prefill_tile(), _p(sink),
                                              _p(out), out.stride(0), H, G, dk, dv, k_cache.shape[2], scale, v_ld, int(window),
-                                             1 if gate_per_head else 0, _p(head_scale), pk, pv, pn, ppp, _stream()),
+                                             1 if gate_per_head else 0, _p(head_scale), pk, pv, pn, ppp, softcap, _stream()),
           "attn_sink_prefill")
     return out
 
@@ -598,15 +602,16 @@ def attn_sink_decode_more(proj, k_cache, block_table, seq_lens, out, init_lse, H
 
 
 def attn_sink_decode(proj, gate_col, k_cache, v_cache, block_table, seq_lens, sink, out, H, G, dk, dv, scale,
-                     v_ld: int = 0, window: int = 0, gate_per_head: bool = False, head_scale=None, pool=None):
+                     v_ld: int = 0, window: int = 0, gate_per_head: bool = False, head_scale=None, pool=None,
+                     softcap: float = 0.0):
     _cuda(proj, k_cache, v_cache, block_table, seq_lens, sink, out, head_scale)
     if k_cache.dtype != proj.dtype or out.dtype != proj.dtype:
         raise B200Error("attn_sink_decode: projection, cache and output must share one element type")
     pk, pv, pn, ppp = _pool_args(pool, k_cache, dk, dv)
-    check(load().b200_attn_sink_decode_pool(_p(proj), _is_f32(proj), proj.stride(0), gate_col, _p(k_cache), _p(v_cache),
+    check(load().b200_attn_sink_decode_cap(_p(proj), _is_f32(proj), proj.stride(0), gate_col, _p(k_cache), _p(v_cache),
                                             _p(block_table), block_table.shape[1], _p(seq_lens), seq_lens.shape[0], _p(sink),
                                             _p(out), out.stride(0), H, G, dk, dv, k_cache.shape[2], scale, v_ld, int(window),
-                                            1 if gate_per_head else 0, _p(head_scale), pk, pv, pn, ppp, _stream()),
+                                            1 if gate_per_head else 0, _p(head_scale), pk, pv, pn, ppp, softcap, _stream()),
           "attn_sink_decode")
     return out
 
@@ -787,8 +792,74 @@ def gla_scan(x, q_col: int, k_col: int, v_col: int, z, inv_tau: float, cu_seq, c
           "gla_scan")
 
 
+# ------------------------------------------- a norm on every sublayer's output, convolved q / k / v
+def embed_sinusoid(ids, positions, table, freq, x_out, norm=None, eps: float = 0.0, xb_out=None):
+    """x_out[t] (fp32) = table[ids[t]] + (sin, cos)(positions[t] * freq[i]) in entries (2i, 2i + 1), through the layer norm
+    norm = (weight, bias) if given; xb_out: the same row rounded once."""
+    _cuda(ids, positions, table, freq, x_out, xb_out)
+    _req(ids, torch.int32, "ids"); _req(positions, torch.int32, "positions"); _req(table, torch.bfloat16, "table")
+    _req(freq, torch.float64, "freq"); _req(x_out, torch.float32, "x_out")
+    D = table.shape[1]
+    if freq.shape[0] < (D + 1) // 2:
+        raise B200Error("embed_sinusoid: one frequency per pair of entries")
+    w, b = norm if norm is not None else (None, None)
+    _cuda(w, b)
+    check(load().b200_embed_sinusoid(_p(ids), _p(positions), _p(table), _p(freq), _p(w), _p(b), _p(x_out), _p(xb_out),
+                                     0 if xb_out is None else _is_f32(xb_out), ids.shape[0], D, table.shape[0], eps, _stream()),
+          "embed_sinusoid")
+
+
+def output_norm_join(x_in, eps: float, y=None, routed=None, post=None, final=None, x_out=None, h_out=None, rows=None):
+    """z = x_in + LN(v; post) with a layer norm that has weight and bias; v is y [T, D] fp32, or with routed = (yp,
+    pair_row, top_k, shared or None, gate logits [T] view or None) the sum of a token's expert rows plus sigmoid(gate) *
+    shared (the combine of routed_experts(..., combine=False)); neither: z = x_in.  x_out = z (fp32); h_out (fp32 or
+    bf16) = z, or LN(z; final).  rows: gather, h_out only."""
+    yp, pair_row, top_k, shared, gate = routed if routed is not None else (None, None, 0, None, None)
+    pw, pb = post if post is not None else (None, None)
+    fw, fb = final if final is not None else (None, None)
+    _cuda(x_in, y, yp, pair_row, shared, gate, pw, pb, fw, fb, x_out, h_out, rows)
+    for t_, n_ in ((x_in, "x_in"), (y, "y"), (yp, "yp"), (shared, "shared"), (x_out, "x_out")):
+        if t_ is not None:
+            _req(t_, torch.float32, n_)
+    if gate is not None and gate.dtype != torch.float32:
+        raise B200Error("output_norm_join: fp32 gate logits")
+    D = x_in.shape[1]
+    T = rows.shape[0] if rows is not None else (h_out if h_out is not None else x_out).shape[0]
+    check(load().b200_output_norm_join(_p(x_in), _p(y), _p(yp), _p(pair_row), top_k, _p(shared), _p(gate),
+                                       0 if gate is None else gate.stride(0), _p(pw), _p(pb), _p(rows), _p(fw), _p(fb), _p(x_out),
+                                       _p(h_out), 0 if h_out is None else _is_f32(h_out), T, D, eps, _stream()),
+          "output_norm_join")
+
+
+def conv_attn_prep(proj, conv_w, q_norm, k_norm, ring, cu_seq, ctx_lens, state_slots, tile_seq, tile_q0, tile_rows: int,
+                   n_prompt: int, n_single: int, slots, q_out, k_cache, v_cache, H, G, dk, dv, eps: float):
+    """Short causal convolution of the projected rows [q | k | v] with per-sequence rings of earlier inputs, per-head norms,
+    queries to q_out [T, H * wk], keys and values to their pages (csrc/conv_attn_prep.cu).  conv_w fp32 [C, taps];
+    ring fp32 [slots, taps - 1, C] (None with one tap); the sequences are n_prompt prompt portions (covered by the row
+    tiles) and then n_single single rows; page widths wk >= dk and wv >= dv come from the caches."""
+    _cuda(proj, conv_w, q_norm, k_norm, ring, cu_seq, ctx_lens, state_slots, tile_seq, tile_q0, slots, q_out, k_cache, v_cache)
+    _req(conv_w, torch.float32, "conv_w")
+    C_, taps = conv_w.shape
+    wk, wv = k_cache.shape[3], v_cache.shape[3]
+    if C_ != (H + G) * dk + G * dv or proj.shape[1] < C_ or proj.stride(1) != 1:
+        raise B200Error("conv_attn_prep: projection rows of [q | k | v] channels expected")
+    if not (proj.dtype == q_out.dtype == k_cache.dtype == v_cache.dtype) or not q_out.is_contiguous() or q_out.shape[1] != H * wk:
+        raise B200Error("conv_attn_prep: projection, queries [T, H * key width] and pages share one element type")
+    if taps > 1:
+        _req(ring, torch.float32, "ring")
+        if tuple(ring.shape[1:]) != (taps - 1, C_):
+            raise B200Error("conv_attn_prep: a ring of [slots, taps - 1, channels]")
+    n_tiles = 0 if tile_seq is None else tile_seq.shape[0]
+    check(load().b200_conv_attn_prep(_p(proj), _is_f32(proj), proj.stride(0), _p(conv_w), taps, _p(q_norm), _p(k_norm), _p(ring),
+                                     _p(cu_seq), _p(ctx_lens), _p(state_slots), _p(tile_seq), _p(tile_q0), n_tiles, tile_rows,
+                                     n_prompt, n_single, _p(slots), _p(q_out), _p(k_cache), _p(v_cache), H, G, dk, dv, wk, wv,
+                                     k_cache.shape[2], eps, _stream()), "conv_attn_prep")
+
+
 # ------------------------------------------- residual streams, latent attention, gated / routed feed-forward
 GATED_ACTS = {"gelu_tanh": 1, "clamped_swish": 2, "silu": 3}
+UNGATED_ACTS = {"relu2": 4}
+SCORE_MODES = {"softmax": 0, "sigmoid": 1, "chosen_softmax": 2}
 
 
 def embed_streams(ids, table, X, S: int, scale: float = 1.0):
@@ -980,19 +1051,24 @@ TC_GROUPED_ACTS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}
 
 def routed_experts(x, router, correction, w13, w2, ws: RoutedWorkspace, out, n_real: int, n_identity: int, top_k: int,
                    scale: float, ff: int, limit: float, shared=None, sigmoid: bool = False, renormalize: bool = True,
-                   weight_on: str = "output", act: str = "clamped_swish"):
+                   weight_on: str = "output", act: str = "clamped_swish", score: Optional[str] = None, combine: bool = True):
     """out[t] (fp32) = sum over the top_k chosen router outputs of weight * expert(x[t]) (identity experts return
     x[t]) + shared[t].  router [n_real + n_identity, D]; w13 [n_real * 2 ff, D] interleaved; w2 [n_real * D, ff];
     shared: the shared expert's output rows (fp32) or None.  Six launches, no host synchronisation.
     sigmoid / renormalize: how the router scores and weights are formed (moe_biased.cu); weight_on "input": the sum
     is over expert(weight * x[t]) -- the weight scales the gathered input row (tensor cores) or the accumulators before
-    the activation (CUDA cores) and the output rows are not scaled; act: the experts' gate activation."""
+    the activation (CUDA cores) and the output rows are not scaled; act: the experts' gate activation, or "relu2": experts
+    without a gate, w13 [n_real * ff, D] as stored.  score "chosen_softmax": the largest logits + correction are chosen and
+    weighted by the softmax over the chosen.  combine False: the weighted expert rows stay in ws.yp (ws.pair_row names
+    them) for output_norm_join, `out` is not written."""
     T, D = x.shape
     E = n_real + n_identity
     n_pairs = T * top_k
-    act_name = act
+    act_name, gated = act, act not in UNGATED_ACTS
+    wide = 2 * ff if gated else ff                  # rows of an expert's first matrix
     # tensor cores when both expert products fit the grouped tcgen05 GEMM (bf16, K multiples of 64, 256-row weight pairs)
-    tc = (LAYER_LIST_TC and x.dtype == torch.bfloat16 and n_real > 0 and D % 256 == 0 and ff % 128 == 0 and x.is_contiguous()
+    tc = (LAYER_LIST_TC and x.dtype == torch.bfloat16 and n_real > 0 and D % 256 == 0 and wide % 256 == 0 and ff % 64 == 0
+          and x.is_contiguous()
           and w13.stride(0) == D and w2.stride(0) == ff)
     bx = moe_block_x(n_pairs, E) if tc else ws.bx
     cap = moe_capacity_rows(n_pairs, E, bx)
@@ -1006,7 +1082,8 @@ def routed_experts(x, router, correction, w13, w2, ws: RoutedWorkspace, out, n_r
     if w_in and n_identity:
         raise B200Error("routed_experts: identity experts with input weights are not defined")
     check(L.b200_moe_route_scored(_p(lg), lg.stride(0), _p(correction), _p(ws.topk_ids), _p(ws.topk_w), T, E, top_k, scale,
-                                  1 if sigmoid else 0, 1 if renormalize else 0, st), "moe_route_scored")
+                                  SCORE_MODES[score] if score else (1 if sigmoid else 0), 1 if renormalize else 0, st),
+          "moe_route_scored")
     check(L.b200_moe_align(_p(ws.topk_ids), _p(ws.topk_w), n_pairs, E, bx, cap, _p(ws.pair_row), _p(ws.row_pair),
                            _p(ws.row_weight), _p(ws.tile_expert), _p(ws.num_tiles), st), "moe_align")
     act = ws.act[:cap * ff].view(cap, ff)
@@ -1015,21 +1092,27 @@ def routed_experts(x, router, correction, w13, w2, ws: RoutedWorkspace, out, n_r
             ws.xp = torch.empty(ws.capacity, D, dtype=torch.bfloat16, device=x.device)
         check(L.b200_moe_gather_scaled(_p(x), _p(ws.row_pair), _p(ws.num_tiles), _p(ws.xp), D, top_k, cap,
                                        _p(ws.row_weight) if w_in else None, st), "moe_gather")
-        check(L.b200_moe_grouped_gemm_ex(_p(ws.xp), _p(w13), _p(act), cap, 2 * ff, D, n_real, D, D, ff, None,
-                                         _p(ws.tile_expert), _p(ws.num_tiles), bx, 1, TC_GROUPED_ACTS[act_name], limit, 0,
-                                         st), "moe_grouped_gemm(gate_up)")
+        check(L.b200_moe_grouped_gemm_ex(_p(ws.xp), _p(w13), _p(act), cap, wide, D, n_real, D, D, ff, None,
+                                         _p(ws.tile_expert), _p(ws.num_tiles), bx, 1 if gated else 0,
+                                         TC_GROUPED_ACTS[act_name] if gated else UNGATED_ACTS[act_name], limit, 0, st),
+              "moe_grouped_gemm(up)")
         check(L.b200_moe_grouped_gemm_ex(_p(act), _p(w2), _p(ws.yp), cap, D, ff, n_real, ff, ff, D,
                                          None if w_in else _p(ws.row_weight),
                                          _p(ws.tile_expert), _p(ws.num_tiles), bx, 0, 0, 0.0, 1, st), "moe_grouped_gemm(down)")
     elif n_real:
         check(L.b200_linear_simt_grouped_ex(_p(x), _is_f32(x), _p(w13), _p(act), _is_f32(act), cap, ff, D, x.stride(0),
                                             w13.stride(0), ff, 1, 0, 0, 0, _p(ws.row_pair), top_k, _p(ws.tile_expert),
-                                            _p(ws.num_tiles), n_real, 2 * ff * w13.stride(0),
-                                            _p(ws.row_weight) if w_in else None, GATED_ACTS[act_name], limit, 1 if w_in else 0,
-                                            st), "linear_simt_grouped(gate_up)")
+                                            _p(ws.num_tiles), n_real, wide * w13.stride(0),
+                                            _p(ws.row_weight) if w_in else None,
+                                            GATED_ACTS[act_name] if gated else UNGATED_ACTS[act_name], limit, 1 if w_in else 0,
+                                            st), "linear_simt_grouped(up)")
         linear_simt_grouped(act, w2, ws.yp, cap, D, ff, ff, w2.stride(0), D, tile_expert=ws.tile_expert,
                             num_tiles=ws.num_tiles, n_real=n_real, w_expert=D * w2.stride(0),
                             row_scale=None if w_in else ws.row_weight)
+    if not combine:
+        if n_identity:
+            raise B200Error("routed_experts: identity experts need the combine")
+        return out
     check(L.b200_moe_combine_mixed(_p(ws.yp), 1, D, _p(ws.pair_row), _p(ws.topk_ids), _p(ws.topk_w), _p(x), _is_f32(x),
                                    x.stride(0), _p(shared), 0 if shared is None else shared.stride(0), _p(out), out.stride(0),
                                    T, D, top_k, n_real, st), "moe_combine_mixed")

@@ -57,6 +57,9 @@ def _layer_list_workspace(m, e: EngineConfig) -> int:
         if x.kind == "attention":
             kv = 0 if x.kv_from is not None else x.kv_heads * (x.dim + (0 if x.values_are_keys else x.vdim))
             proj = max(proj, x.q_width + kv + x.gate_width + 7)
+            if x.conv_taps:
+                wk, wv = x.cache_widths(a == 2)
+                lat, mix = max(lat, x.heads * wk), max(mix, x.heads * wv)      # prepared query rows, padded head outputs
         elif x.kind == "side_by_side":
             y, r = x.left, x.right
             proj = max(proj, y.q_width + y.kv_heads * (y.dim + y.vdim) + r.proj_rows + 7)
@@ -78,7 +81,7 @@ def _layer_list_workspace(m, e: EngineConfig) -> int:
             r = l.mlp.moe
             ff = max(ff, r.shared_ff)
             cap = T * r.top + (r.experts + r.identity) * 64          # permuted (token, expert) rows in 64-row tiles
-            routed = max(routed, cap * (r.ff * a + D * 4 + 12) + T * (D * 4 + (r.experts + r.identity) * 4 + r.top * 12))
+            routed = max(routed, cap * (r.ff * a + D * 4 + 12) + T * (D * 4 + (r.experts + r.identity + r.shared_gate) * 4 + r.top * 12))
         elif l.mlp is not None:
             ff = max(ff, l.mlp.ff)
     S_smp = min(T, max(S, e.max_logit_rows or 0))

@@ -338,7 +338,7 @@ class LayerListLayer:
     mlstm      rows = [q: H*dk | k: H*dk | v: H*dv | gate: H*dv];  its two per-head gate projections are a
     second, fp32-output projection `gates` = [input: H | forget: H],
     linear attention  rows = [q: H*dk | k: H*dk | v: H*dv | gate: H*dv]; an attention mixer whose values are its
-    keys has no v rows."""
+    keys has no v rows.  Routed experts without a gate keep their up matrices in w13 / shared13 as stored."""
     norm1: torch.Tensor
     proj: torch.Tensor
     o: torch.Tensor
@@ -352,7 +352,7 @@ class LayerListLayer:
     norm2: Optional[torch.Tensor] = None
     up: Optional[torch.Tensor] = None
     down: Optional[torch.Tensor] = None
-    # tanh norm: bias vector and the scalar alpha (fp32 [1]) of norm1 / norm2
+    # tanh norm and layer norm with bias: bias vector and the scalar alpha (fp32 [1]) of norm1 / norm2
     norm1_b: Optional[torch.Tensor] = None
     norm1_alpha: Optional[torch.Tensor] = None
     norm2_b: Optional[torch.Tensor] = None
@@ -397,6 +397,7 @@ class LayerListLayer:
     # gated linear attention: proj rows = [q | k | v | gate | decay latent]; the decay's second projection and bias
     decay_up: Optional[torch.Tensor] = None      # bf16 [H*dk, rank]
     decay_bias: Optional[torch.Tensor] = None    # bf16 [H*dk]
+    conv_w: Optional[torch.Tensor] = None        # attention: fp32 [channels of q | k | v, taps], the convolutions after the projection
 
 
 @dataclass
@@ -409,6 +410,9 @@ class LayerListWeights:
     vocab_end: int = 0
     final_norm_b: Optional[torch.Tensor] = None
     final_norm_alpha: Optional[torch.Tensor] = None
+    embed_norm: Optional[torch.Tensor] = None    # norm of the embedding output
+    embed_norm_b: Optional[torch.Tensor] = None
+    pos_freq: Optional[torch.Tensor] = None      # fp64 [ceil(D / 2)]: frequencies of the sinusoidal positions
     pos: Optional[torch.Tensor] = None           # learned positions [max_position_embeddings, D]
 
 
@@ -420,14 +424,19 @@ def layer_list_tensor_shapes(cfg) -> Dict[str, tuple]:
     S = getattr(cfg, "streams", 0)
     parallel = getattr(cfg, "residual", "post_ln") == "parallel"     # one norm per layer feeds both sublayers
 
+    biased = tanh or getattr(cfg, "norm", "layernorm") == "layernorm_bias"
+
     def norm_shapes(name):
         shapes[name] = (D,)
-        if tanh:
+        if biased:
             shapes[name + ".b"] = (D,)
+        if tanh:
             shapes[name + ".alpha"] = ()
 
-    if tanh:
+    if biased:
         norm_shapes("final.norm")
+    if getattr(cfg, "embed_norm", False):
+        norm_shapes("embed.norm")
     sandwich = getattr(cfg, "residual", "post_ln") == "sandwich"
     taps = getattr(cfg, "canon_taps", 0)
     if getattr(cfg, "learned_positions", False):
@@ -505,6 +514,9 @@ def layer_list_tensor_shapes(cfg) -> Dict[str, tuple]:
                     shapes[p + "mix.v.b"] = (m.kv_heads * m.vdim,)
                 if m.qk_norm:
                     shapes[p + "mix.k.norm"] = (m.dim,)
+            if m.conv_taps:
+                for n in ("q", "k", "v"):
+                    shapes[p + f"mix.{n}.conv"] = (shapes[p + "mix." + n][0], m.conv_taps)
             if m.sink:
                 shapes[p + "mix.sink"] = (m.heads,)
             if m.gate:
@@ -530,14 +542,22 @@ def layer_list_tensor_shapes(cfg) -> Dict[str, tuple]:
             if layer.mlp.kind == "moe":
                 e = layer.mlp.moe
                 for i in range(e.experts):
-                    shapes[p + f"mlp.e{i}.gate"] = shapes[p + f"mlp.e{i}.up"] = (e.ff, D)
+                    if e.gated:
+                        shapes[p + f"mlp.e{i}.gate"] = (e.ff, D)
+                    shapes[p + f"mlp.e{i}.up"] = (e.ff, D)
                     shapes[p + f"mlp.e{i}.down"] = (D, e.ff)
                 shapes[p + "mlp.router"] = (e.experts + e.identity, D)
+                if e.router_bias:
+                    shapes[p + "mlp.router.b"] = (e.experts + e.identity,)
                 if e.score == "softmax":
                     shapes[p + "mlp.correction"] = (e.experts + e.identity,)
                 if e.shared_ff:
-                    shapes[p + "mlp.shared.gate"] = shapes[p + "mlp.shared.up"] = (e.shared_ff, D)
+                    if e.gated:
+                        shapes[p + "mlp.shared.gate"] = (e.shared_ff, D)
+                    shapes[p + "mlp.shared.up"] = (e.shared_ff, D)
                     shapes[p + "mlp.shared.down"] = (D, e.shared_ff)
+                    if e.shared_gate:
+                        shapes[p + "mlp.shared.sg"] = (1, D)
                 continue
             if layer.mlp.act != "relu2":
                 shapes[p + "mlp.gate"] = (layer.mlp.ff, D)
@@ -569,6 +589,7 @@ def load_layer_list(cfg, get: Callable[[str], torch.Tensor], device: str) -> Lay
         return g(name).to(torch.float32).reshape(-1).contiguous()
 
     tanh = getattr(cfg, "norm", "layernorm") == "tanh"
+    biased = tanh or getattr(cfg, "norm", "layernorm") == "layernorm_bias"
     S = getattr(cfg, "streams", 0)
     parallel = getattr(cfg, "residual", "post_ln") == "parallel"
 
@@ -641,7 +662,12 @@ def load_layer_list(cfg, get: Callable[[str], torch.Tensor], device: str) -> Lay
         elif m.kind == "attention":
             own = m.kv_from is None
             names = ["q"] + ((["k"] if m.values_are_keys else ["k", "v"]) if own else []) + (["g"] if m.gate else [])
-            lw = LayerListLayer(norm1=g(p + "norm1"), proj=cat([p + "mix." + n for n in names]), o=g(p + "mix.o"))
+            lw = LayerListLayer(norm1=g(p + "norm1"), proj=(cat8 if m.conv_taps else cat)([p + "mix." + n for n in names]),
+                                o=g(p + "mix.o"))
+            if m.conv_taps:
+                lw.conv_w = cat([p + f"mix.{n}.conv" for n in "qkv"]).to(torch.float32).contiguous()
+            if m.plus_one:           # a sink of score zero: exp(0) joins the denominator
+                lw.sink = torch.zeros(m.heads, dtype=torch.float32, device=device)
             if m.qkv_bias:
                 lw.proj_bias = cat([p + f"mix.{n}.b" for n in (["q", "k", "v"] if own else ["q"])])
             if m.qk_norm:
@@ -662,29 +688,40 @@ def load_layer_list(cfg, get: Callable[[str], torch.Tensor], device: str) -> Lay
             lw = LayerListLayer(norm1=g(p + "norm1"), proj=cat([p + "mix." + n for n in "qkvg"]), o=g(p + "mix.o"),
                                 gates=cat([p + "mix.i", p + "mix.f"]), gate_bias=cat([p + "mix.i.b", p + "mix.f.b"]),
                                 out_norm=g(p + "mix.norm"))
+        if biased:
+            lw.norm1_b = g(p + "norm1.b")
         if tanh:
-            lw.norm1_b, lw.norm1_alpha = g(p + "norm1.b"), f32(p + "norm1.alpha")
+            lw.norm1_alpha = f32(p + "norm1.alpha")
         if getattr(cfg, "residual", "post_ln") == "streams":
             lw.hc1 = hyper(p + "hc1")
         if layer.mlp is not None:
             if not parallel:
                 lw.norm2 = g(p + "norm2")
+            if biased:
+                lw.norm2_b = g(p + "norm2.b")
             if tanh:
-                lw.norm2_b, lw.norm2_alpha = g(p + "norm2.b"), f32(p + "norm2.alpha")
+                lw.norm2_alpha = f32(p + "norm2.alpha")
             if getattr(cfg, "residual", "post_ln") == "streams":
                 lw.hc2 = hyper(p + "hc2")
             if layer.mlp.kind == "moe":
                 e = layer.mlp.moe
                 # zero rows up to a whole GEMM weight tile: the router projection is an ordinary one-tile product
+                # (the gate of a shared expert is one more row behind the router outputs: no product of its own)
                 router = g(p + "mlp.router")
+                if e.shared_gate and e.shared_ff:
+                    router = torch.cat([router, g(p + "mlp.shared.sg")])
                 lw.router = torch.zeros(-(-router.shape[0] // 128) * 128, router.shape[1], dtype=BF16, device=device)
                 lw.router[:router.shape[0]] = router
-                lw.correction = f32(p + "mlp.correction") if e.score == "softmax" else None
-                lw.w13 = torch.cat([_interleave_rows(g(p + f"mlp.e{i}.gate"), g(p + f"mlp.e{i}.up"))
-                                    for i in range(e.experts)], dim=0).contiguous()
+                lw.correction = f32(p + "mlp.correction") if e.score == "softmax" else \
+                    (f32(p + "mlp.router.b") if e.router_bias else None)
+
+                def first(q):
+                    return _interleave_rows(g(q + ".gate"), g(q + ".up")) if e.gated else g(q + ".up")
+
+                lw.w13 = torch.cat([first(p + f"mlp.e{i}") for i in range(e.experts)], dim=0).contiguous()
                 lw.w2 = torch.cat([g(p + f"mlp.e{i}.down") for i in range(e.experts)], dim=0).contiguous()
                 if e.shared_ff:
-                    lw.shared13 = _interleave_rows(g(p + "mlp.shared.gate"), g(p + "mlp.shared.up"))
+                    lw.shared13 = first(p + "mlp.shared").contiguous()
                     lw.shared2 = g(p + "mlp.shared.down")
             elif layer.mlp.act == "relu2":
                 lw.up, lw.down = g(p + "mlp.up"), g(p + "mlp.down")
@@ -693,11 +730,25 @@ def load_layer_list(cfg, get: Callable[[str], torch.Tensor], device: str) -> Lay
         layers.append(lw)
     out = LayerListWeights(embed=g("embed"), layers=layers, final_norm=g("final.norm"), lm_head=g("head"),
                            vocab_start=0, vocab_end=cfg.vocab_size)
+    if biased:
+        out.final_norm_b = g("final.norm.b")
     if tanh:
-        out.final_norm_b, out.final_norm_alpha = g("final.norm.b"), f32("final.norm.alpha")
+        out.final_norm_alpha = f32("final.norm.alpha")
+    if getattr(cfg, "embed_norm", False):
+        out.embed_norm, out.embed_norm_b = g("embed.norm"), g("embed.norm.b")
+    if getattr(cfg, "sinusoidal_positions", False):
+        D = cfg.hidden_size
+        out.pos_freq = torch.tensor([10000.0 ** (-2.0 * i / D) for i in range((D + 1) // 2)], dtype=torch.float64).to(device)
     if getattr(cfg, "learned_positions", False):
         out.pos = g("pos")
     return out
+
+
+def pad_head_columns(o: torch.Tensor, heads: int, width: int, padded: int) -> torch.Tensor:
+    """Output projection [D, heads * width] for heads laid out `padded` wide: zero columns behind every head's own."""
+    out = torch.zeros(o.shape[0], heads, padded, dtype=o.dtype, device=o.device)
+    out[:, :, :width] = o.view(o.shape[0], heads, width)
+    return out.view(o.shape[0], heads * padded)
 
 
 def load_layer_list_dir(cfg, model_path: str, device: str) -> LayerListWeights:

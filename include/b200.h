@@ -421,7 +421,7 @@ int b200_paged_attn_decode_win(const void* q, int64_t q_stride, const void* k_ca
                                const float* sink, const void* gate, int64_t gate_stride, int window, void* stream);
 /* b200_moe_route_biased with sigmoid scores (sigmoid_scores != 0) and / or weights that are not renormalised. */
 int b200_moe_route_scored(const float* logits, int64_t ld, const float* correction, int32_t* topk_ids, float* topk_w, int T,
-                          int E, int K, float scale, int sigmoid_scores, int renormalize, void* stream);
+                          int E, int K, float scale, int score_mode, int renormalize, void* stream);
 /* b200_linear_simt_grouped whose row_scale multiplies the rows' input (before the activation) when scale_in != 0. */
 int b200_linear_simt_grouped_ex(const void* X, int x_f32, const void* W, void* Y, int y_f32, int M, int N, int K,
                                 int64_t ldx, int64_t ldw, int64_t ldy, int batch, int64_t bsx, int64_t bsw, int64_t bsy,
@@ -537,6 +537,53 @@ int b200_gla_scan(const float* x, int64_t ld, int q_col, int k_col, int v_col, c
 int b200_gla_scan_rows(const float* x, int64_t ld, int q_col, int k_col, int v_col, const float* z, int64_t ldz, float inv_tau,
                   const int32_t* cu_seq, const int32_t* ctx_lens, const int32_t* state_slots, float* S, float* o_raw,
                   int n_seqs, int H, int dk, int dv, int max_len, void* stream);
+
+/* ---- a norm on every sublayer's output; convolved q, k and v; capped scores and logits --------------------------- */
+/* z = x_in + LN(v; wb, bb) (layer norm with weight and bias); v is y [T][D], or (yp != NULL) the sum of the top_k rows
+ * yp[pair_row[t top_k + j]] plus sigmoid(gate[t ld_gate]) * shared[t] (gate NULL: factor 1; shared NULL: none), or absent
+ * (z = x_in).  x_out = z; h_out (bf16 or fp32) = z, or with wa / ba LN(z; wa, ba).  rows != NULL: gather, h_out only. */
+int b200_output_norm_join(const float* x_in, const float* y, const float* yp, const int32_t* pair_row, int top_k,
+                          const float* shared, const float* gate, int64_t ld_gate, const void* wb, const void* bb,
+                          const int32_t* rows, const void* wa, const void* ba, float* x_out, void* h_out, int h_f32, int T,
+                          int D, float eps, void* stream);
+/* x_out[t] = LN(table[ids[t]] + (sin, cos)(positions[t] * freq[i]) in entries (2i, 2i + 1)); w NULL: no norm. */
+int b200_embed_sinusoid(const int32_t* ids, const int32_t* positions, const void* table, const double* freq, const void* w,
+                        const void* b, float* x_out, void* xb_out, int xb_f32, int T, int D, int vocab, float eps,
+                        void* stream);
+/* Short causal convolution of the projected rows [q | k | v] (per channel, `taps` taps, ring [slots][taps - 1][channels]
+ * of earlier inputs, updated in the same launch), per-head RMS norm of q and k (weights may be NULL), queries to q_out
+ * [T][H wk], keys and values to their pages of widths wk / wv (zeros behind dk / dv).  cu_seq / ctx_lens / state_slots list
+ * the n_prompt prompt portions (row tiles tile_seq / tile_q0 of tile_rows rows), then n_single single rows. */
+int b200_conv_attn_prep(const void* proj, int f32, int64_t ld, const float* conv_w, int taps, const void* qnorm_w,
+                        const void* knorm_w, float* ring, const int32_t* cu_seq, const int32_t* ctx_lens,
+                        const int32_t* state_slots, const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles,
+                        int tile_rows, int n_prompt, int n_single, const int32_t* slots, void* q_out, void* k_cache,
+                        void* v_cache, int H, int G, int dk, int dv, int wk, int wv, int page, float eps, void* stream);
+/* The attention kernels with a soft cap on the scaled score, softcap * tanh(score / softcap) (0 = none). */
+int b200_attn_sink_prefill_cap(const void* proj, int f32, int64_t ld, int gate_col, const void* k_cache, const void* v_cache,
+                                const int32_t* block_table, int max_blocks, const int32_t* cu_q, const int32_t* ctx_lens,
+                                const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, int tile_rows, const float* sink,
+                                void* out, int64_t ldo, int H, int G, int dk, int dv, int page, float scale, int64_t v_ld,
+                                int window, int gate_per_head, const float* head_scale, const float* pool_k,
+                                const float* pool_v, int pool, int per_page, float softcap, void* stream);
+int b200_attn_sink_decode_cap(const void* proj, int f32, int64_t ld, int gate_col, const void* k_cache, const void* v_cache,
+                               const int32_t* block_table, int max_blocks, const int32_t* seq_lens, int B, const float* sink,
+                               void* out, int64_t ldo, int H, int G, int dk, int dv, int page, float scale, int64_t v_ld,
+                               int window, int gate_per_head, const float* head_scale, const float* pool_k,
+                               const float* pool_v, int pool, int per_page, float softcap, void* stream);
+int b200_paged_attn_prefill_cap(const void* q, int64_t q_stride, int num_tokens, const void* k_cache, const void* v_cache,
+                                int num_blocks, const int32_t* block_table, int max_blocks, const int32_t* cu_q,
+                                const int32_t* ctx_lens, const int32_t* tile_seq, const int32_t* tile_q0, int num_tiles,
+                                void* out, int Hq, int Hkv, int D, int block_size, float scale, const float* sink,
+                                const void* gate, int64_t gate_stride, int window, int gate_per_head, float* lse_out, float softcap, void* stream);
+int b200_paged_attn_decode_cap(const void* q, int64_t q_stride, const void* k_cache, const void* v_cache,
+                               const int32_t* block_table, int max_blocks, const int32_t* seq_lens, void* out,
+                               void* workspace, int num_splits, int B, int Hq, int Hkv, int D, int block_size, float scale,
+                               const float* sink, const void* gate, int64_t gate_stride, int window, int gate_per_head,
+                               float* lse_out, float softcap, void* stream);
+/* b200_sample_f32 whose logits first become softcap * tanh(logit / softcap), written back in the same pass. */
+int b200_sample_softcap_f32(float* logits, int64_t ld, float softcap, const float* temps, const uint32_t* seeds, int vocab_offset,
+                            int32_t* out_idx, float* out_val, int B, int V, void* stream);
 
 #ifdef __cplusplus
 }
