@@ -8,8 +8,8 @@
 //   columns behind dk / dv are zeros: a pair of widths that is no tensor-core tile is padded to one);
 //   the step's last taps - 1 inputs of every sequence replace the ring's entries: ring[slot][p mod (taps - 1)][channel].
 //
-// A CTA takes 16 consecutive rows of one sequence and some head slots; the threads that own a channel walk the rows in
-// order and keep the last taps - 1 inputs in registers, so a projected row is read once.  Only a sequence's first
+// A CTA takes 8 consecutive rows of one sequence and some head slots; the threads that own a channel issue all their loads
+// (8 rows and the taps - 1 before them) at once and walk the rows in registers.  Only a sequence's first
 // piece can need the ring (a piece is longer than the ring), and the SAME threads that read it there write the step's
 // last inputs into it after their reads: no second launch, no race.  The statistics and the convolution are fp32.
 #include "common.cuh"
@@ -18,7 +18,7 @@
 
 namespace b200 {
 
-constexpr int kCapRows = 16;       // rows of one sequence per CTA
+constexpr int kCapRows = 8;        // rows of one sequence per CTA
 constexpr int kCapMaxTaps = 8;
 constexpr int kCapWarps = 8;
 
@@ -30,7 +30,7 @@ __device__ __forceinline__ void ca_store(bf16* p, float v) { *p = __float2bfloat
 struct CapArgs {
   const void* proj;
   int64_t ld;
-  const float* conv_w;             // [C][taps], last column = current token
+  const float* conv_w;             // [taps][C], last row = current token
   const bf16* qnorm_w;             // null: no norm
   const bf16* knorm_w;
   float* ring;                     // [slots][taps - 1][C]; null when taps == 1
@@ -39,14 +39,14 @@ struct CapArgs {
   const int32_t* state_slots;
   const int32_t* tile_seq;         // row tiles of the prompt portions
   const int32_t* tile_q0;
-  int n_pieces;                    // tiles * (tile_rows / 16): CTAs [0, n_pieces) along x; then one per single row
-  int per_tile;                    // tile_rows / 16
+  int n_pieces;                    // tiles * (tile_rows / 8): CTAs [0, n_pieces) along x; then one per single row
+  int per_tile;                    // tile_rows / 8
   int n_prompt;                    // sequences with a prompt portion
   const int32_t* slots;            // cache slot of every row (-1: no write)
   void* q_out;
   void* k_cache;
   void* v_cache;
-  int H, G, dk, dv, wk, wv, page, taps;
+  int H, G, dk, dv, wk, wv, page, page_shift, taps;    // page_shift: log2(page), or -1
   float eps;
 };
 
@@ -73,17 +73,23 @@ __device__ __forceinline__ CapWork cap_work(const CapArgs& a) {
   return m;
 }
 
+// the (page, head) row of a cache slot, in rows of the cache
+__device__ __forceinline__ size_t cap_cache_row(const CapArgs& a, int slot, int g) {
+  const int pg = a.page_shift >= 0 ? slot >> a.page_shift : slot / a.page;
+  return ((size_t)pg * a.G + g) * a.page + (slot - pg * a.page);
+}
+
 // LPH lanes share a head, each owns one 16-byte piece of it.
 template <typename TA, int TAPS>
-__global__ void __launch_bounds__(kCapWarps * 32)
+__global__ void __launch_bounds__(kCapWarps * 32, 2)
 conv_attn_prep_vec_kernel(CapArgs a, int lph) {
-  constexpr int V = 16 / (int)sizeof(TA), R = TAPS - 1;
+  constexpr int V = 16 / (int)sizeof(TA), R = TAPS - 1, NB = kCapRows;
+  static_assert(R <= NB, "a sequence's first piece holds every row that reads the ring");
   const CapWork m = cap_work(a);
   if (m.n <= 0) return;
   const int lane = threadIdx.x & 31, per_warp = 32 / lph;
-  const int hs = (blockIdx.y * kCapWarps + (threadIdx.x >> 5)) * per_warp + lane / lph;
-  const int n_heads = a.H + 2 * a.G;
-  const bool live = hs < n_heads;
+  const int hs = (blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5)) * per_warp + lane / lph;
+  const bool live = hs < a.H + 2 * a.G;
   const bool is_q = hs < a.H, is_k = !is_q && hs < a.H + a.G;
   const int width = (is_q || is_k) ? a.dk : a.dv, wide = (is_q || is_k) ? a.wk : a.wv;
   const int col0 = (is_q || is_k) ? hs * a.dk : (a.H + a.G) * a.dk + (hs - a.H - a.G) * a.dv;
@@ -91,97 +97,87 @@ conv_attn_prep_vec_kernel(CapArgs a, int lph) {
   const bool act = live && d < width, pad = live && !act && d < wide;
   const int c = col0 + d, C = (a.H + a.G) * a.dk + a.G * a.dv;
   const TA* src = reinterpret_cast<const TA*>(a.proj) + (size_t)m.row0 * a.ld + c;
-  auto load = [&](int q, float (&x)[V]) {
-    const uint4 raw = *reinterpret_cast<const uint4*>(src + (size_t)q * a.ld);
-    const TA* rv = reinterpret_cast<const TA*>(&raw);
+  const uint4 zero4 = make_uint4(0, 0, 0, 0);
+  auto load = [&](int q) { return *reinterpret_cast<const uint4*>(src + (int64_t)q * a.ld); };
+  // win[R + i]: row i of the piece as loaded; win[R - 1 - b]: the input b + 1 positions before it (a ring entry is an
+  // input, so it fits the element type exactly)
+  uint4 win[R + NB];
 #pragma unroll
-    for (int i = 0; i < V; ++i) x[i] = ca_f32(rv[i]);
-  };
-  float w[TAPS][V], hist[R > 0 ? R : 1][V], nw[V];     // w[b]: weight of the input b positions back; hist[b]: that input, b + 1 back
+  for (int i = 0; i < NB; ++i) win[R + i] = (act && i < m.n) ? load(m.q0 + i) : zero4;
+#pragma unroll
+  for (int b = 0; b < R; ++b) win[b] = zero4;
   const bf16* norm = is_q ? a.qnorm_w : (is_k ? a.knorm_w : nullptr);
+  float w[TAPS][V], nw[V];         // w[b]: weight of the input b positions back
   if (act) {
-#pragma unroll
-    for (int i = 0; i < V; ++i) {
-#pragma unroll
-      for (int b = 0; b < TAPS; ++b) w[b][i] = a.conv_w[(size_t)(c + i) * TAPS + (R - b)];
-      nw[i] = norm != nullptr ? __bfloat162float(norm[d + i]) : 1.0f;
-    }
 #pragma unroll
     for (int b = 0; b < R; ++b) {
       const int q = m.q0 - 1 - b, p = m.ctx + q;
       if (q >= 0) {
-        load(q, hist[b]);
+        win[R - 1 - b] = load(q);
       } else if (p >= 0 && m.slot >= 0) {
         const float* rp = a.ring + ((size_t)m.slot * R + p % (R > 0 ? R : 1)) * C + c;
+        TA* wv = reinterpret_cast<TA*>(&win[R - 1 - b]);
 #pragma unroll
-        for (int i = 0; i < V; ++i) hist[b][i] = rp[i];
-      } else {
-#pragma unroll
-        for (int i = 0; i < V; ++i) hist[b][i] = 0.f;
+        for (int i = 0; i < V; ++i) ca_store(wv + i, rp[i]);
       }
     }
+#pragma unroll
+    for (int b = 0; b < TAPS; ++b)
+#pragma unroll
+      for (int i = 0; i < V; i += 4)
+        *reinterpret_cast<float4*>(&w[b][i]) = *reinterpret_cast<const float4*>(a.conv_w + (size_t)(R - b) * C + c + i);
+#pragma unroll
+    for (int i = 0; i < V; ++i) nw[i] = norm != nullptr ? __bfloat162float(norm[d + i]) : 1.0f;
     if (R > 0 && m.q0 == 0 && m.slot >= 0) {           // the ring has been read by its only readers: this step's last inputs
 #pragma unroll
       for (int b = 0; b < R; ++b) {
         const int q = m.qlen - 1 - b;
         if (q < 0) break;
-        float x[V];
-        load(q, x);
+        const uint4 raw = load(q);
+        const TA* x = reinterpret_cast<const TA*>(&raw);
         float* rp = a.ring + ((size_t)m.slot * R + (m.ctx + q) % (R > 0 ? R : 1)) * C + c;
 #pragma unroll
-        for (int i = 0; i < V; ++i) rp[i] = x[i];
+        for (int i = 0; i < V; i += 4)
+          *reinterpret_cast<float4*>(rp + i) = make_float4(ca_f32(x[i]), ca_f32(x[i + 1]), ca_f32(x[i + 2]), ca_f32(x[i + 3]));
       }
     }
   }
-  float nxt[V];
+  const float inv_dk = 1.0f / (float)a.dk;
+  const int g = is_k ? hs - a.H : hs - a.H - a.G;
+  TA* const q_dst = reinterpret_cast<TA*>(a.q_out) + ((size_t)(m.row0 + m.q0) * a.H + hs) * a.wk + d;
+  TA* const kv_dst = reinterpret_cast<TA*>(is_k ? a.k_cache : a.v_cache) + d;
+  const int32_t* slots = a.slots + m.row0 + m.q0;
 #pragma unroll
-  for (int i = 0; i < V; ++i) nxt[i] = 0.f;
-  if (act) load(m.q0, nxt);
-#pragma unroll 4
-  for (int i_row = 0; i_row < m.n; ++i_row) {
-    const int q = m.q0 + i_row;
-    float cur[V], y[V];
+  for (int r = 0; r < NB; ++r) {
+    if (r >= m.n) break;
+    float y[V], ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < V; ++i) cur[i] = nxt[i];
-    if (act && i_row + 1 < m.n) load(q + 1, nxt);
-    float ss = 0.f;
+    for (int i = 0; i < V; ++i) y[i] = 0.f;
+    if (act) {
 #pragma unroll
-    for (int i = 0; i < V; ++i) {
-      y[i] = 0.f;
-      if (act) {
-        float v = w[0][i] * cur[i];
+      for (int b = 0; b < TAPS; ++b) {
+        const TA* x = reinterpret_cast<const TA*>(&win[R + r - b]);
 #pragma unroll
-        for (int b = 0; b < R; ++b) v = fmaf(w[b + 1][i], hist[b][i], v);
-        y[i] = v;
-        ss = fmaf(v, v, ss);
+        for (int i = 0; i < V; ++i) y[i] = fmaf(w[b][i], ca_f32(x[i]), y[i]);
       }
-    }
 #pragma unroll
-    for (int b = R - 1; b > 0; --b)
-#pragma unroll
-      for (int i = 0; i < V; ++i) hist[b][i] = hist[b - 1][i];
-    if (R > 0) {
-#pragma unroll
-      for (int i = 0; i < V; ++i) hist[0][i] = cur[i];
+      for (int i = 0; i < V; ++i) ss = fmaf(y[i], y[i], ss);
     }
     for (int o = lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);    // all lanes take part
     if (!act && !pad) continue;
-    const float mul = norm != nullptr ? 1.0f / sqrtf(ss / (float)a.dk + a.eps) : 1.0f;
-    const size_t row = (size_t)(m.row0 + q);
-    TA* dst;
-    if (is_q) {
-      dst = reinterpret_cast<TA*>(a.q_out) + (row * a.H + hs) * a.wk;
-    } else {
-      const int slot = a.slots[row];
-      if (slot < 0) continue;
-      const int g = is_k ? hs - a.H : hs - a.H - a.G;
-      dst = reinterpret_cast<TA*>(is_k ? a.k_cache : a.v_cache) + (((size_t)(slot / a.page) * a.G + g) * a.page + (slot % a.page)) * wide;
-    }
-    uint4 outv;
-    TA* ov = reinterpret_cast<TA*>(&outv);
+    uint4 outv = zero4;
+    if (act) {
+      const float mul = norm != nullptr ? rsqrtf(fmaf(ss, inv_dk, a.eps)) : 1.0f;
+      TA* ov = reinterpret_cast<TA*>(&outv);
 #pragma unroll
-    for (int i = 0; i < V; ++i) ca_store(ov + i, act ? (norm != nullptr ? y[i] * mul * nw[i] : y[i]) : 0.f);
-    *reinterpret_cast<uint4*>(dst + d) = outv;
+      for (int i = 0; i < V; ++i) ca_store(ov + i, y[i] * mul * nw[i]);
+    }
+    if (is_q) {
+      *reinterpret_cast<uint4*>(q_dst + (size_t)r * a.H * a.wk) = outv;
+    } else {
+      const int slot = slots[r];
+      if (slot >= 0) *reinterpret_cast<uint4*>(kv_dst + cap_cache_row(a, slot, g) * wide) = outv;
+    }
   }
 }
 
@@ -207,14 +203,14 @@ conv_attn_prep_kernel(CapArgs a) {
       const int d = lane + 32 * i;
       y[i] = 0.f;
       if (d < width) {
-        const float* w = a.conv_w + (size_t)(col0 + d) * a.taps;
+        const float* w = a.conv_w + col0 + d;
         float v = 0.f;
         for (int b = 0; b <= R; ++b) {
           const int qq = q - b, p = m.ctx + qq;
           float x = 0.f;
           if (qq >= 0) x = ca_f32(src[(size_t)qq * a.ld + d]);
           else if (p >= 0 && m.slot >= 0) x = a.ring[((size_t)m.slot * R + p % R) * C + col0 + d];
-          v = fmaf(w[R - b], x, v);
+          v = fmaf(w[(size_t)(R - b) * C], x, v);
         }
         y[i] = v;
         ss = fmaf(v, v, ss);
@@ -230,7 +226,7 @@ conv_attn_prep_kernel(CapArgs a) {
       const int slot = a.slots[row];
       if (slot < 0) continue;
       const int g = is_k ? hs - a.H : hs - a.H - a.G;
-      dst = reinterpret_cast<TA*>(is_k ? a.k_cache : a.v_cache) + (((size_t)(slot / a.page) * a.G + g) * a.page + (slot % a.page)) * wide;
+      dst = reinterpret_cast<TA*>(is_k ? a.k_cache : a.v_cache) + cap_cache_row(a, slot, g) * wide;
     }
 #pragma unroll
     for (int i = 0; i < kPer; ++i) {
@@ -269,19 +265,24 @@ extern "C" int b200_conv_attn_prep(const void* proj, int f32, int64_t ld, const 
   const int per_tile = n_tiles > 0 ? tile_rows / kCapRows : 1;
   const int n_x = n_tiles * per_tile + n_single;
   if (n_x == 0) return B200_OK;
+  int shift = 0;
+  while ((1 << shift) < page) ++shift;
   const CapArgs a{proj, ld, conv_w, (const bf16*)qnorm_w, (const bf16*)knorm_w, taps > 1 ? ring : nullptr, cu_seq, ctx_lens,
                   state_slots, tile_seq, tile_q0, n_tiles * per_tile, per_tile, n_prompt, slots, q_out, k_cache, v_cache, H, G,
-                  dk, dv, wk, wv, page, taps, eps};
+                  dk, dv, wk, wv, page, (1 << shift) == page ? shift : -1, taps, eps};
   cudaStream_t s = (cudaStream_t)stream;
   const int n_heads = H + 2 * G, esz = f32 ? 4 : 2, vec = 16 / esz, wmax = wk > wv ? wk : wv;
+  const int C = (H + G) * dk + G * dv;
   const bool al = ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(k_cache) |
-                    reinterpret_cast<uintptr_t>(v_cache)) & 15) == 0;
-  if (al && taps <= 4 && dk % vec == 0 && dv % vec == 0 && wk % vec == 0 && wv % vec == 0 && ld % vec == 0 && wmax / vec <= 32) {
+                    reinterpret_cast<uintptr_t>(v_cache) | reinterpret_cast<uintptr_t>(conv_w) | reinterpret_cast<uintptr_t>(a.ring)) & 15) == 0;
+  if (al && taps <= 4 && dk % vec == 0 && dv % vec == 0 && wk % vec == 0 && wv % vec == 0 && ld % vec == 0 && C % 4 == 0 && wmax / vec <= 32) {
     int lph = 1;
     while (lph < wmax / vec) lph <<= 1;
-    const int per_block = kCapWarps * (32 / lph);
-    const dim3 grid(n_x, (n_heads + per_block - 1) / per_block);
-#define B200_CAP(TA, N) conv_attn_prep_vec_kernel<TA, N><<<grid, kCapWarps * 32, 0, s>>>(a, lph)
+    // warps that cover all head slots, in CTAs of equal size
+    const int all_warps = (n_heads + 32 / lph - 1) / (32 / lph), ny = (all_warps + kCapWarps - 1) / kCapWarps;
+    const int warps = (all_warps + ny - 1) / ny;
+    const dim3 grid(n_x, ny);
+#define B200_CAP(TA, N) conv_attn_prep_vec_kernel<TA, N><<<grid, warps * 32, 0, s>>>(a, lph)
 #define B200_CAPT(TA)                        \
   switch (taps) {                            \
     case 1: B200_CAP(TA, 1); break;          \

@@ -1,7 +1,7 @@
-"""Side benchmark of the layer-list family (Vodavik, Danipel, Resevik, Dotorax) beside the closest existing model of equal layer
+"""Side benchmark of the layer-list family (Vodavik, Danipel, Resevik, Dotorax, Kerarax) beside the closest existing model of equal layer
 sizes (a Llama-class decoder; for Resevik also Vodavik, the other design with attention and recurrent-state layers).
 
-`python bench.py --family vodavik|danipel|resevik|dotorax` prints ONE JSON line (not the serving benchmark's line; that workload and its
+`python bench.py --family vodavik|danipel|resevik|dotorax|kerarax` prints ONE JSON line (not the serving benchmark's line; that workload and its
 contract are untouched).  Random weights, synthetic tokens.  Two kinds of numbers:
 
   model:   prefill tokens/s (prompts of `prompt` tokens, `seqs` at a time through runner.prefill) and decode tokens/s
@@ -851,10 +851,186 @@ def _kernel_numbers_dotorax(size, T, B, ctx, log):
     return res
 
 
+# Kerarax at the same widths: taps, score cap, experts, top, expert (and shared expert) ff
+KERARAX = {"2k": (4, 30.0, 8, 2, 2048), "4k": (4, 30.0, 8, 2, 3584)}
+
+
+def kerarax_config(size: str, layers: int = 4) -> LayerListConfig:
+    """Convolved attention with capped scores and 8 routed relu^2 experts (2 chosen, a shared one of the same width) in
+    every layer."""
+    D, H, G, hd, ff, V = SIZES[size]
+    taps, cap, E, top, ffe = KERARAX[size]
+    specs = []
+    for _ in range(layers):
+        mix = AttentionSpec(H, G, hd, hd, hd ** -0.5, qk_norm=True, qkv_bias=False, sink=False, gate=False, softcap=cap,
+                            plus_one=True, conv_taps=taps)
+        moe = MoESpec(experts=E, top=top, ff=ffe, limit=0.0, shared_ff=ffe, score="chosen_softmax", act="relu2", router_bias=True,
+                      shared_gate=True)
+        specs.append(LayerSpec(mix, MLPSpec("moe", ffe, act="relu2", moe=moe)))
+    return LayerListConfig("Kerarax", V, D, specs, norm_eps=1e-5, residual="output_norm", norm="layernorm_bias",
+                           sinusoidal_positions=True, embed_norm=True, logit_softcap=30.0)
+
+
+def _kernel_numbers_kerarax(size, T, B, ctx, log):
+    """Kerarax's kernels beside the like kernels of the closest models at equal sizes: Vodavik (norm after the sum, head norms,
+    softmax sink, squared ReLU) and, for the routed feed-forward, Danipel (experts chosen with a correction, shared
+    expert)."""
+    D, H, G, hd, ff, V = SIZES[size]
+    taps, cap, E, top, ffe = KERARAX[size]
+    hbm, flops_peak, how = _peaks()
+    flush = _Flush()
+    dev = "cuda"
+    bf, f32 = torch.bfloat16, torch.float32
+    rnd = lambda *s, dt=bf, sc=1.0: (torch.randn(*s, device=dev, dtype=f32) * sc).to(dt)   # noqa: E731
+    i32 = lambda x: torch.as_tensor(x, dtype=torch.int32, device=dev)   # noqa: E731
+    res = {}
+
+    def put(name, new_s, new_work, like_name, like_s, like_work, kind):
+        peak = hbm if kind == "bytes" else flops_peak
+        fn, fl = new_work / new_s / peak, like_work / like_s / peak
+        res[name] = {"us": round(new_s * 1e6, 1), "frac_of_" + how + "_" + kind: round(fn, 4), "like": like_name,
+                     "like_us": round(like_s * 1e6, 1), "like_frac": round(fl, 4), "distance_ratio": round(fl / fn, 2)}
+        log(f"  {name:44s} {new_s * 1e6:9.1f} us  {fn:7.4f} of roofline | {like_name}: {like_s * 1e6:9.1f} us {fl:7.4f}"
+            f"  -> {fl / fn:5.2f}x as far")
+
+    S = max(1, T // 2048)
+    L = T // S
+    cu, ctx0, slot_s = i32(np.arange(S + 1) * L), i32(np.zeros(S)), i32(np.arange(S))
+    cud, ctxd, slot_b = i32(np.arange(B + 1)), i32(np.full(B, ctx)), i32(np.arange(B))
+    # ---- embedding
+    table = rnd(V, D)
+    ids, pos = i32(np.random.RandomState(0).randint(0, V, T)), i32(np.arange(T) % L)
+    freq = torch.tensor([10000.0 ** (-2.0 * i / D) for i in range(D // 2)], dtype=torch.float64, device=dev)
+    x32, y32, w, b = rnd(T, D, dt=f32), rnd(T, D, dt=f32), rnd(D), rnd(D)
+    xb = torch.empty(T, D, device=dev, dtype=bf)
+    t_new = _time(lambda: ops.embed_sinusoid(ids, pos, table, freq, x32, norm=(w, b), eps=1e-5, xb_out=xb), flush)
+    t_like = _time(lambda: ops.embed_rows(ids, table, x32, xb), flush)
+    put("embed_sinusoid (+ norm)", t_new, T * D * 8.0, "embed_rows", t_like, T * D * 8.0, "bytes")
+    # ---- norm of the output + sum, and the same with the combine of the routed feed-forward in it
+    t_new = _time(lambda: ops.output_norm_join(x32, 1e-5, y=y32, post=(w, b), x_out=x32, h_out=xb), flush)
+    t_like = _time(lambda: ops.sum_layer_norm(y32, x32, w, 2.0, 1e-5, x_out=x32, xb_out=xb), flush)
+    put("output_norm_join", t_new, T * D * 14.0, "sum_layer_norm", t_like, T * D * 14.0, "bytes")
+    xB, yB, xbB = x32[:B], y32[:B], xb[:B]
+    t_new = _time(lambda: ops.output_norm_join(xB, 1e-5, y=yB, post=(w, b), x_out=xB, h_out=xbB), flush)
+    t_like_b = _time(lambda: ops.sum_layer_norm(yB, xB, w, 2.0, 1e-5, x_out=xB, xb_out=xbB), flush)
+    put("output_norm_join (single rows)", t_new, B * D * 14.0, "sum_layer_norm (single rows)", t_like_b, B * D * 14.0, "bytes")
+    yp, sh = rnd(T * top, D, dt=f32), rnd(T, D, dt=f32)
+    pr = i32(np.random.RandomState(1).permutation(T * top))
+    lg = rnd(T, 128, dt=f32)
+    t_new = _time(lambda: ops.output_norm_join(x32, 1e-5, routed=(yp, pr, top, sh, lg[:, E]), post=(w, b), x_out=x32, h_out=xb), flush)
+    tid, tw = i32(np.zeros(T * top)), rnd(T * top, dt=f32)
+    from .lib import check, load
+
+    L_ = load()
+    st = torch.cuda.current_stream().cuda_stream
+    t_like = _time(lambda: check(L_.b200_moe_combine_mixed(yp.data_ptr(), 1, D, pr.data_ptr(), tid.data_ptr(), tw.data_ptr(),
+                                                           xb.data_ptr(), 0, D, sh.data_ptr(), D, y32.data_ptr(), D, T, D, top, E, st)), flush)
+    put("output_norm_join (routed combine in it)", t_new, T * D * (4.0 * (top + 1) + 10), "moe_combine_mixed (Danipel)", t_like,
+        T * D * 4.0 * (top + 2), "bytes")
+
+    # ---- convolution + head norms + page scatter in one launch vs bias + head norms + page scatter
+    C = (H + 2 * G) * hd
+    nblk = (B * ctx + T) // 16 + 8
+    proj = rnd(T, C)
+    kc, vc = rnd(nblk, G, 16, hd), rnd(nblk, G, 16, hd)
+    cw = rnd(taps, C, dt=f32, sc=0.5)
+    ring = torch.zeros(max(S, B), taps - 1, C, device=dev)
+    qn, kn, bias = rnd(hd), rnd(hd), rnd(C)
+    slots = i32(np.arange(T) + 16)
+    tile = ops.attn_prefill_tile(H, G)
+    ts_, tq_ = ops.build_prefill_tiles([L] * S, tile, [0] * S)
+    ts_d, tq_d = i32(ts_), i32(tq_)
+    q = torch.empty(T, H * hd, device=dev, dtype=bf)
+    t_new = _time(lambda: ops.conv_attn_prep(proj, cw, qn, kn, ring, cu, ctx0, slot_s, ts_d, tq_d, tile, S, 0, slots, q, kc, vc, H, G,
+                                             hd, hd, 1e-5), flush)
+    projv = rnd(T, C + H * hd)                       # Vodavik's rows also hold the output gate
+    t_like = _time(lambda: ops.attn_prep(projv, bias, qn, kn, pos, slots, kc, vc, H, G, hd, hd, 1e-5, 0.1, 512), flush)
+    put("conv_attn_prep (prefill)", t_new, T * C * 4.0, "attn_prep", t_like, T * C * 4.0, "bytes")
+    pB, sB, qB = proj[:B], slots[:B], q[:B]
+    t_new = _time(lambda: ops.conv_attn_prep(pB, cw, qn, kn, ring, cud, ctxd, slot_b, None, None, tile, 0, B, sB, qB, kc, vc, H, G,
+                                             hd, hd, 1e-5), flush)
+    pvB, posB = projv[:B], pos[:B]
+    t_like = _time(lambda: ops.attn_prep(pvB, bias, qn, kn, posB, sB, kc, vc, H, G, hd, hd, 1e-5, 0.1, 512), flush)
+    put("conv_attn_prep (single rows)", t_new, B * C * (4.0 + 4.0 * taps), "attn_prep (single rows)", t_like, B * C * 4.0, "bytes")
+
+    # ---- attention: capped scores + one in the denominator vs learned sink + output gate
+    nb = (L + 15) // 16
+    bt = i32(np.arange(S * nb).reshape(S, nb) + 1)
+    zero, sink = torch.zeros(H, device=dev), rnd(H, dt=f32)
+    out = torch.empty(T, H * hd, device=dev, dtype=bf)
+    gate = projv[:, C:]
+    t_new = _time(lambda: ops.paged_attn_prefill_ex(q, H * hd, kc, vc, bt, cu, ctx0, ts_d, tq_d, out, H, G, hd, hd ** -0.5, sink=zero,
+                                                    softcap=cap), flush)
+    t_like = _time(lambda: ops.paged_attn_prefill_ex(projv, projv.shape[1], kc, vc, bt, cu, ctx0, ts_d, tq_d, out, H, G, hd,
+                                                     hd ** -0.5, sink=sink, gate=gate), flush)
+    pairs = S * (L * L / 2) * H
+    put("attention prefill, capped", t_new, 4.0 * pairs * hd, "attention prefill, sink + gate tc", t_like, 4.0 * pairs * hd, "flops")
+    t_big = _time(lambda: ops.paged_attn_prefill_ex(q, H * hd, kc, vc, bt, cu, ctx0, ts_d, tq_d, out, H, G, hd, hd ** -0.5, sink=zero,
+                                                    softcap=80.0), flush)
+    put("attention prefill, capped at 80 (running maximum)", t_big, 4.0 * pairs * hd, "attention prefill, sink + gate tc", t_like,
+        4.0 * pairs * hd, "flops")
+    put("attention prefill, capped, 96-wide values padded", t_new, 2.0 * pairs * (hd + 96), "attention prefill, sink + gate tc", t_like,
+        4.0 * pairs * hd, "flops")
+    nbd = (ctx + 16) // 16
+    btd = i32(np.arange(B * nbd).reshape(B, nbd) % (nblk - 1) + 1)
+    lens = i32(np.full(B, ctx))
+    splits = ops.attn_decode_splits(B, G, ctx + 16)
+    ws = ops.attn_decode_workspace(B, H, hd, splits, dev)
+    outd = torch.empty(B, H * hd, device=dev, dtype=bf)
+    gB = gate[:B]
+    t_new = _time(lambda: ops.paged_attn_decode(qB, H * hd, kc, vc, btd, lens, outd, H, G, hd, hd ** -0.5, num_splits=splits,
+                                                workspace=ws, sink=zero, softcap=cap), flush)
+    t_like = _time(lambda: ops.paged_attn_decode(pvB, projv.shape[1], kc, vc, btd, lens, outd, H, G, hd, hd ** -0.5,
+                                                 num_splits=splits, workspace=ws, sink=sink, gate=gB), flush)
+    kvb = B * ctx * G * hd * 4.0
+    put("attention decode, capped", t_new, kvb, "attention decode, sink + gate", t_like, kvb, "bytes")
+    put("attention decode, capped, 96-wide values padded", t_new, B * ctx * G * (hd + 96) * 2.0, "attention decode, sink + gate", t_like,
+        kvb, "bytes")
+    # the generic kernels (fp32 pages, groups no tensor-core tile takes), with and without the cap
+    t16, q16 = ops.build_prefill_tiles([L] * S, 16, [0] * S)
+    t16, q16 = i32(t16), i32(q16)
+    t_new = _time(lambda: ops.attn_sink_prefill(q, -1, kc, vc, bt, cu, ctx0, t16, q16, zero, out, H, G, hd, hd, hd ** -0.5, softcap=cap),
+                  flush, iters=3, warm=1)
+    t_like = _time(lambda: ops.attn_sink_prefill(q, -1, kc, vc, bt, cu, ctx0, t16, q16, zero, out, H, G, hd, hd, hd ** -0.5), flush,
+                   iters=3, warm=1)
+    put("generic attention prefill, capped", t_new, 4.0 * pairs * hd, "generic attention prefill, sink", t_like, 4.0 * pairs * hd, "flops")
+    t_new = _time(lambda: ops.attn_sink_decode(qB, -1, kc, vc, btd, lens, zero, outd, H, G, hd, hd, hd ** -0.5, softcap=cap), flush)
+    t_like = _time(lambda: ops.attn_sink_decode(qB, -1, kc, vc, btd, lens, zero, outd, H, G, hd, hd, hd ** -0.5), flush)
+    put("generic attention decode, capped", t_new, kvb, "generic attention decode, sink", t_like, kvb, "bytes")
+
+    # ---- routed relu^2 experts vs Danipel's clamped gated experts (both with their combine)
+    xin = rnd(T, D)
+    router = torch.zeros(128, D, device=dev, dtype=bf)
+    router[:E + 1] = rnd(E + 1, D, sc=0.05)
+    corr = rnd(E, dt=f32, sc=0.01)
+    w1, w13, w2 = rnd(E * ffe, D, sc=0.02), rnd(E * 2 * ffe, D, sc=0.02), rnd(E * D, ffe, sc=0.02)
+    for rows, tag in ((T, "prefill"), (B, "decode")):
+        rws = ops.RoutedWorkspace(rows, top, E + 1, D, ffe, bf, dev)
+        xr, yo = xin[:rows], y32[:rows]
+        t_new = _time(lambda: ops.routed_experts(xr, router, corr, w1, w2, rws, yo, E, 0, top, 1.0, ffe, 0.0, act="relu2",
+                                                 score="chosen_softmax"), flush, iters=5, warm=2)
+        t_like = _time(lambda: ops.routed_experts(xr, router, corr, w13, w2, rws, yo, E, 0, top, 1.0, ffe, 7.0), flush, iters=5, warm=2)
+        put(f"routed relu^2 experts ({tag})", t_new, 4.0 * rows * top * D * ffe, f"routed clamped experts, Danipel ({tag})", t_like,
+            6.0 * rows * top * D * ffe, "flops")
+        wb_new, wb_like = E * 2.0 * D * ffe * 2, E * 3.0 * D * ffe * 2
+        if tag == "decode":      # every expert's weights are read once: the bound of a small batch
+            put("routed relu^2 experts (decode, weight bytes)", t_new, wb_new, "routed clamped experts, Danipel (decode)", t_like, wb_like,
+                "bytes")
+        del rws
+    # ---- sampler that caps the logits in its pass
+    logits, temps, seeds = rnd(B, V, dt=f32), torch.zeros(B, device=dev), i32(np.zeros(B))
+    t_new = _time(lambda: ops.sample(logits, temps, seeds, softcap=30.0), flush)
+    t_like = _time(lambda: ops.sample(logits, temps, seeds), flush)
+    put("sampler with capped logits", t_new, B * V * 8.0, "sampler", t_like, B * V * 4.0, "bytes")
+    return res
+
+
 FAMILIES = {"vodavik": (vodavik_config, _kernel_numbers), "danipel": (danipel_config, _kernel_numbers_danipel),
-            "resevik": (resevik_config, _kernel_numbers_resevik), "dotorax": (dotorax_config, _kernel_numbers_dotorax)}
+            "resevik": (resevik_config, _kernel_numbers_resevik), "dotorax": (dotorax_config, _kernel_numbers_dotorax),
+            "kerarax": (kerarax_config, _kernel_numbers_kerarax)}
 # a family whose closest existing model is another layer-list design is measured beside that one too
-CLOSEST = {"resevik": ("vodavik", vodavik_config), "dotorax": ("resevik", resevik_config)}
+CLOSEST = {"resevik": ("vodavik", vodavik_config), "dotorax": ("resevik", resevik_config),
+           "kerarax": ("danipel", danipel_config)}
 
 
 def run(sizes=("2k", "4k"), seqs=4, prompt=2048, batch=64, decode_steps=32, log=None, family="vodavik"):

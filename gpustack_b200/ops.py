@@ -834,12 +834,12 @@ def output_norm_join(x_in, eps: float, y=None, routed=None, post=None, final=Non
 def conv_attn_prep(proj, conv_w, q_norm, k_norm, ring, cu_seq, ctx_lens, state_slots, tile_seq, tile_q0, tile_rows: int,
                    n_prompt: int, n_single: int, slots, q_out, k_cache, v_cache, H, G, dk, dv, eps: float):
     """Short causal convolution of the projected rows [q | k | v] with per-sequence rings of earlier inputs, per-head norms,
-    queries to q_out [T, H * wk], keys and values to their pages (csrc/conv_attn_prep.cu).  conv_w fp32 [C, taps];
-    ring fp32 [slots, taps - 1, C] (None with one tap); the sequences are n_prompt prompt portions (covered by the row
+    queries to q_out [T, H * wk], keys and values to their pages (csrc/conv_attn_prep.cu).  conv_w fp32 [taps, C] (last row:
+    the current token); ring fp32 [slots, taps - 1, C] (None with one tap); the sequences are n_prompt prompt portions (covered by the row
     tiles) and then n_single single rows; page widths wk >= dk and wv >= dv come from the caches."""
     _cuda(proj, conv_w, q_norm, k_norm, ring, cu_seq, ctx_lens, state_slots, tile_seq, tile_q0, slots, q_out, k_cache, v_cache)
     _req(conv_w, torch.float32, "conv_w")
-    C_, taps = conv_w.shape
+    taps, C_ = conv_w.shape
     wk, wv = k_cache.shape[3], v_cache.shape[3]
     if C_ != (H + G) * dk + G * dv or proj.shape[1] < C_ or proj.stride(1) != 1:
         raise B200Error("conv_attn_prep: projection rows of [q | k | v] channels expected")

@@ -397,7 +397,7 @@ class LayerListLayer:
     # gated linear attention: proj rows = [q | k | v | gate | decay latent]; the decay's second projection and bias
     decay_up: Optional[torch.Tensor] = None      # bf16 [H*dk, rank]
     decay_bias: Optional[torch.Tensor] = None    # bf16 [H*dk]
-    conv_w: Optional[torch.Tensor] = None        # attention: fp32 [channels of q | k | v, taps], the convolutions after the projection
+    conv_w: Optional[torch.Tensor] = None        # attention: fp32 [taps, channels of q | k | v], the convolutions after the projection
 
 
 @dataclass
@@ -665,7 +665,7 @@ def load_layer_list(cfg, get: Callable[[str], torch.Tensor], device: str) -> Lay
             lw = LayerListLayer(norm1=g(p + "norm1"), proj=(cat8 if m.conv_taps else cat)([p + "mix." + n for n in names]),
                                 o=g(p + "mix.o"))
             if m.conv_taps:
-                lw.conv_w = cat([p + f"mix.{n}.conv" for n in "qkv"]).to(torch.float32).contiguous()
+                lw.conv_w = cat([p + f"mix.{n}.conv" for n in "qkv"]).to(torch.float32).t().contiguous()
             if m.plus_one:           # a sink of score zero: exp(0) joins the denominator
                 lw.sink = torch.zeros(m.heads, dtype=torch.float32, device=device)
             if m.qkv_bias:
