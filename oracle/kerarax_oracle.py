@@ -69,11 +69,11 @@ def capped_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: f
     T, H, _ = q.shape
     G = k.shape[1]
     out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
+    later = torch.ones(T, T, dtype=torch.bool).triu(1)
     for h in range(H):
         g = h // (H // G)
-        for i in range(T):
-            s = soft_cap((k[:i + 1, g] @ q[i, h]) * scale, cap)
-            out[i, h] = softmax_plus_one(s) @ v[:i + 1, g]
+        s = soft_cap((q[:, h] @ k[:, g].T) * scale, cap).masked_fill(later, -float("inf"))
+        out[:, h] = softmax_plus_one(s) @ v[:, g]
     return out
 
 
@@ -133,3 +133,54 @@ def forward(cfg: dict, weights: Dict[str, torch.Tensor], tokens: List[int], trac
         if trace is not None:
             trace.append(x.clone())
     return soft_cap(norm(x, "final.norm") @ w["head"].T, cfg["logit_softcap"])
+
+
+# ------------------------------------------------------------------------------ random checkpoints
+def tensor_shapes(cfg: dict) -> Dict[str, tuple]:
+    D, V = cfg["width"], cfg["vocab"]
+    out: Dict[str, tuple] = {"embed": (V, D), "head": (V, D)}
+
+    def norm(name):
+        out[name] = out[name + ".b"] = (D,)
+
+    norm("embed.norm")
+    norm("final.norm")
+    for l, layer in enumerate(cfg["layers"]):
+        p, mx, mlp = f"l{l}.", layer["mixer"], layer.get("mlp")
+        norm(p + "norm1")
+        for n, rows in (("q", mx["heads"] * mx["dim"]), ("k", mx["kv_heads"] * mx["dim"]), ("v", mx["kv_heads"] * mx["vdim"])):
+            out[p + "mix." + n] = (rows, D)
+            out[p + f"mix.{n}.conv"] = (rows, mx["conv"])
+        out[p + "mix.q.norm"] = out[p + "mix.k.norm"] = (mx["dim"],)
+        out[p + "mix.o"] = (D, mx["heads"] * mx["vdim"])
+        if not mlp:
+            continue
+        norm(p + "norm2")
+        E, ff = mlp["router"]["experts"], mlp["expert"]["ff"]
+        out[p + "mlp.router"], out[p + "mlp.router.b"] = (E, D), (E,)
+        for e in range(E):
+            out[p + f"mlp.e{e}.up"], out[p + f"mlp.e{e}.down"] = (ff, D), (D, ff)
+        if mlp.get("shared"):
+            fs = mlp["shared"]["ff"]
+            out[p + "mlp.shared.up"], out[p + "mlp.shared.down"], out[p + "mlp.shared.sg"] = (fs, D), (D, fs), (1, D)
+    return out
+
+
+def random_weights(cfg: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
+    """Seeded bf16 weights: linear weights N(0, 1 / in), norm weights around one, biases of a few tenths, convolution taps
+    of half."""
+    g = torch.Generator().manual_seed(seed)
+    out: Dict[str, torch.Tensor] = {}
+    for name, shape in tensor_shapes(cfg).items():
+        x = torch.randn(tuple(shape), generator=g)
+        leaf = name.split(".")[-1]
+        if leaf == "b":
+            x = 0.3 * x
+        elif leaf == "conv":
+            x = 0.5 * x
+        elif leaf in ("norm", "norm1", "norm2"):
+            x = 1.0 + 0.2 * x
+        elif name != "embed":
+            x = x / shape[-1] ** 0.5
+        out[name] = x.to(torch.bfloat16)
+    return out
