@@ -15,7 +15,7 @@ from typing import Optional
 
 SUPPORTED_ARCHS = ("LlamaForCausalLM", "MistralForCausalLM", "Qwen2ForCausalLM", "MixtralForCausalLM")
 # designs whose config.json lists their layers one by one (LayerListConfig below)
-LAYER_LIST_ARCHS = ("Vodavik", "Danipel", "Resevik", "Dotorax", "Kerarax")
+LAYER_LIST_ARCHS = ("Vodavik", "Danipel", "Resevik", "Dotorax", "Kerarax", "Bovitar")
 
 
 @dataclass
@@ -243,6 +243,7 @@ class AttentionSpec:
     # > 0: a short causal convolution over time (this many taps, no bias) on every channel of q, k and v right after
     # the projection, before the q / k norm; the last taps - 1 projected rows of a sequence are part of its state
     conv_taps: int = 0
+    qk_norm_joint: bool = False    # the q / k norm runs over the whole projection (all heads at once), weights of that size
 
     kind = "attention"
 
@@ -363,12 +364,96 @@ class GatedRecurrenceSpec:
 
 
 @dataclass
+class StateSpaceSpec:
+    """State-space recurrence with one decay per head and token (Mamba-2).  One projection gives [z | x | B | C | dt]; x, B
+    and C pass a causal convolution per channel (`conv` taps, with bias) and silu; d = softplus(dt + dt_bias);
+    S_t = exp(-exp(A_log) d) S_(t-1) + d B_t x_t^T (state x vdim per head, B and C shared by heads / groups heads),
+    y_t = S_t^T C_t + D x_t; then y silu(z), an RMS norm in norm_groups equal parts with a weight, and a projection."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int
+    norm_groups: int = 1
+
+    kind = "state_space"
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def conv_width(self) -> int:
+        """Channels [x | B | C] of the convolution."""
+        return self.out_width + 2 * self.groups * self.state
+
+    @property
+    def proj_rows(self) -> int:
+        """Rows of the projection [z | x | B | C]; the dt rows are an fp32 product of their own."""
+        return self.out_width + self.conv_width
+
+    @property
+    def row_width(self) -> int:
+        """fp32 row of the recurrence's inputs [x | B | C], every head and group padded to a multiple of 4."""
+        return self.heads * _up4(self.vdim) + 2 * self.groups * _up4(self.state)
+
+    @property
+    def state_width(self) -> int:
+        """Floats of a sequence's recurrent state (key index fastest, padded to a multiple of 4)."""
+        return self.heads * self.vdim * _up4(self.state)
+
+
+@dataclass
+class DeltaRuleSpec:
+    """Gated delta rule.  q, k (kv_heads x dim) and v (heads x vdim) pass a causal convolution per channel (`conv` taps, no
+    bias) and silu; q and k become unit vectors x / sqrt(sum(x^2) + 1e-6), q times dim^(-1/2); beta = sigmoid(b),
+    g = exp(-exp(A_log) softplus(a + dt_bias)) per head; S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q; every
+    head of o is RMS-normed with one weight of vdim entries and multiplied by silu of a gate projection."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+
+    kind = "delta"
+
+    @property
+    def out_width(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def conv_width(self) -> int:
+        """Channels [q | k | v] of the convolution."""
+        return 2 * self.kv_heads * self.dim + self.out_width
+
+    @property
+    def proj_rows(self) -> int:
+        """Rows of the fused projection [q | k | v | gate]; the b and a rows are an fp32 product of their own."""
+        return self.conv_width + self.out_width
+
+    @property
+    def row_width(self) -> int:
+        """fp32 row of the recurrence's inputs [q | k | v], every head padded to a multiple of 4."""
+        return 2 * self.kv_heads * _up4(self.dim) + self.heads * _up4(self.vdim)
+
+    @property
+    def state_width(self) -> int:
+        return self.heads * self.vdim * _up4(self.dim)
+
+
+def _up4(n: int) -> int:
+    return -(-n // 4) * 4
+
+
+@dataclass
 class SideBySideSpec:
-    """Two mixers that read the same input; the mixer's output is left_scale * left + right_scale * right."""
+    """Two mixers that read the same input; the mixer's output is left_scale * left + right_scale * right, with branch_norm
+    each of the two after an RMS norm over the model width with a weight of its own."""
     left: "AttentionSpec"
-    right: GatedRecurrenceSpec
+    right: object                  # GatedRecurrenceSpec | StateSpaceSpec
     left_scale: float
     right_scale: float
+    branch_norm: bool = False
 
     kind = "side_by_side"
 
@@ -416,6 +501,12 @@ class RotarySpec:
     yarn_original: float = 0.0
     yarn_fast: float = 0.0
     yarn_slow: float = 0.0
+    # scaling by wavelength (as in Llama 3.1; wave_factor > 0): with w = 2 pi / f, f stays where w < original / high, becomes
+    # f / factor where w > original / low, and a blend (1 - s) f / factor + s f, s = (original / w - low) / (high - low), between
+    wave_factor: float = 0.0
+    wave_original: float = 0.0
+    wave_low: float = 0.0
+    wave_high: float = 0.0
 
     def frequencies(self):
         """(fp64 list of dims/2 angular frequencies, the factor on cos and sin)."""
@@ -423,6 +514,17 @@ class RotarySpec:
 
         half = self.dims // 2
         f = [self.base ** (-2.0 * i / self.dims) for i in range(half)]
+        if self.wave_factor > 0.0:
+            out = []
+            for x in f:
+                turns = self.wave_original * x / (2.0 * math.pi)      # original / wavelength
+                if turns < self.wave_low:
+                    x = x / self.wave_factor
+                elif turns <= self.wave_high:
+                    s = (turns - self.wave_low) / (self.wave_high - self.wave_low)
+                    x = (1.0 - s) * x / self.wave_factor + s * x
+                out.append(x)
+            return out, 1.0
         if self.yarn_factor <= 0.0:
             return f, 1.0
 
@@ -442,6 +544,9 @@ class RotarySpec:
         if self.yarn_factor > 0.0:
             d["scaling"] = {"factor": self.yarn_factor, "original": self.yarn_original, "fast": self.yarn_fast,
                             "slow": self.yarn_slow}
+        if self.wave_factor > 0.0:
+            d["scaling"] = {"factor": self.wave_factor, "original": self.wave_original, "low": self.wave_low,
+                            "high": self.wave_high}
         return d
 
 
@@ -510,6 +615,10 @@ class MoESpec:
     act: str = "clamped_swish"
     router_bias: bool = False
     shared_gate: bool = False
+    # groups > 0: the experts form this many equal groups of neighbours; a group's score is the largest choice score (with the
+    # correction) in it, and only experts of the groups_keep best groups can be chosen
+    groups: int = 0
+    groups_keep: int = 0
 
     @property
     def gated(self) -> bool:
@@ -532,6 +641,7 @@ class MLPSpec:
 class LayerSpec:
     mixer: object                  # AttentionSpec | MLSTMSpec
     mlp: Optional[MLPSpec]
+    weights_of: Optional[int] = None   # the layer whose tensors this one uses (its cache and state are its own)
 
 
 @dataclass
@@ -553,6 +663,7 @@ class LayerListConfig:
     # x <- x + mixer(norm(x)) + ff(norm(x))
     # "sandwich": a norm before and after every sublayer, x <- x + residual_mult * norm_b(f(norm_a(x)))
     # "output_norm": a norm on what a sublayer puts out and nothing else, x <- x + norm(f(x))
+    # "pre_norm": x <- x + f(norm(x)), every sublayer with a norm of its own
     residual: str = "post_ln"
     # "layernorm" (bias-free) | "layernorm_bias" | "tanh": tanh(alpha x) w + b, no statistics | "rms" | "rms_zero_centred": an RMS norm
     # whose stored weight is the deviation from one, x / rms(x) * (1 + w)
@@ -606,8 +717,14 @@ class LayerListConfig:
     def has_state(self) -> bool:
         """True when some mixer carries a recurrent state per sequence (needs a state slot; no prefix reuse)."""
         return self.canon_taps > 1 or any(l.mixer.kind in ("mlstm", "linear_attention", "side_by_side",
-                                                           "gated_linear_attention")
+                                                           "gated_linear_attention", "delta")
                                            or (l.mixer.kind == "attention" and l.mixer.conv_taps > 1) for l in self.layers)
+
+    def weight_owner(self, l: int) -> int:
+        """The layer whose tensors layer l uses (itself unless weights_of)."""
+        while self.layers[l].weights_of is not None:
+            l = self.layers[l].weights_of
+        return l
 
     def kv_owner(self, l: int) -> Optional[int]:
         """Layer whose K/V cache layer l's attention reads (itself unless kv_from), None for other mixers."""
@@ -627,7 +744,7 @@ class LayerListConfig:
         mixers = [self.layers[l].mixer for l, _ in self.runs()]
         mixers = [m.left if m.kind == "side_by_side" else m for m in mixers]
         n = sum(m.kv_heads * sum(m.cache_widths(elem_bytes == 2)) * elem_bytes for m in mixers
-                if m.kind == "attention" and m.kv_from is None)
+                if m.kind == "attention" and m.kv_from is None)     # (a side-by-side pair's left half is one of them)
         # pooled block means (fp32): ceil(16 / pool) entries per 16-token page
         n += sum(m.kv_heads * (m.dim + m.vdim) * 4 * m.pool_per_page(16) // 16 for m in mixers
                  if m.kind == "attention" and m.pool)
@@ -643,8 +760,13 @@ class LayerListConfig:
                 n += 4 * m.heads * m.dim * m.vdim
             elif m.kind == "attention" and m.conv_taps > 1:
                 n += 4 * m.qkv_width * (m.conv_taps - 1)
+            elif m.kind == "side_by_side" and m.right.kind == "state_space":
+                n += 4 * (m.left.qkv_width * max(0, m.left.conv_taps - 1) + m.right.state_width
+                          + m.right.conv_width * (m.right.conv - 1))
             elif m.kind == "side_by_side":
                 n += 4 * m.right.width * m.right.conv          # the recurrence and its convolution's last inputs
+            elif m.kind == "delta":
+                n += 4 * (m.state_width + m.conv_width * (m.conv - 1))
         if self.canon_taps > 1:
             n += 4 * self.hidden_size * (self.canon_taps - 1) * sum(1 + (self.layers[l].mlp is not None) for l, _ in self.runs())
         return n
@@ -653,7 +775,13 @@ class LayerListConfig:
         D, n = self.hidden_size, 0
         for l in self.layers:
             m = l.mixer
-            if m.kind == "side_by_side":
+            if l.weights_of is not None:
+                continue
+            if m.kind == "side_by_side" and m.right.kind == "state_space":
+                n += D * (m.left.qkv_width + m.right.proj_rows + m.right.heads + m.left.out_width + m.right.out_width)
+            elif m.kind == "delta":
+                n += D * (m.proj_rows + 2 * m.heads + m.out_width)
+            elif m.kind == "side_by_side":
                 a, r = m.left, m.right
                 n += D * (a.q_width + a.kv_heads * (a.dim + a.vdim)) + a.out_width * D
                 n += 3 * D * r.width + 2 * r.width * r.width // r.blocks
@@ -689,6 +817,8 @@ class LayerListConfig:
             return _dotorax_from_dict(d)
         if arch == "Kerarax":
             return _kerarax_from_dict(d)
+        if arch == "Bovitar":
+            return _bovitar_from_dict(d)
         layers = []
         for i, e in enumerate(d["layers"]):
             mx = e["mixer"]
@@ -733,6 +863,8 @@ class LayerListConfig:
             return _dotorax_to_dict(self)
         if self.architecture == "Kerarax":
             return _kerarax_to_dict(self)
+        if self.architecture == "Bovitar":
+            return _bovitar_to_dict(self)
         out = []
         for l in self.layers:
             m = l.mixer
@@ -1066,6 +1198,117 @@ def _kerarax_to_dict(c: "LayerListConfig") -> dict:
         out.append({"type": "attention", "mixer": mx, "mlp": mlp})
     return {"architecture": "Kerarax", "vocab": c.vocab_size, "width": c.hidden_size, "layers": out,
             "norm": {"eps": c.norm_eps}, "logit_softcap": c.logit_softcap}
+
+
+def _bovitar_from_dict(d: dict) -> "LayerListConfig":
+    """Bovitar: pre-norm layers with RMS norms, some of which use an earlier layer's tensors; mixers "delta" (gated delta
+    rule) and "parallel" (left: attention over convolved q, k and v, q and k normed over the whole projection, half-split
+    rotation with frequencies scaled by wavelength, capped scores; right: a state-space recurrence; half the sum of the two
+    normed outputs); routed gated-SiLU experts chosen by corrected softmax scores inside the best groups, with a shared
+    expert."""
+    layers = []
+    for i, e in enumerate(d["layers"]):
+        mx, kind = e["mixer"], e["type"]
+
+        def taps(x):
+            if not 1 <= int(x["conv"]) <= 8:
+                raise ValueError(f"layer {i}: conv {x['conv']} taps (1 .. 8)")
+            return int(x["conv"])
+
+        def split(n, parts, what):
+            if n < 1 or parts < 1 or n % parts:
+                raise ValueError(f"layer {i}: {n} {what} in {parts} equal parts")
+
+        if kind == "delta":
+            spec = DeltaRuleSpec(heads=int(mx["heads"]), kv_heads=int(mx.get("kv_heads", mx["heads"])), dim=int(mx["dim"]),
+                                 vdim=int(mx.get("vdim", mx["dim"])), conv=taps(mx))
+            split(spec.heads, spec.kv_heads, "heads")
+        elif kind == "parallel":
+            L, R = mx["left"], mx["right"]
+            r, sc = L["rot"], L["rot"].get("scaling") or {}
+            rot = RotarySpec(dims=int(r["dims"]), base=float(r["base"]), layout="half", wave_factor=float(sc.get("factor", 0.0)),
+                             wave_original=float(sc.get("original", 0.0)), wave_low=float(sc.get("low", 0.0)),
+                             wave_high=float(sc.get("high", 0.0)))
+            left = AttentionSpec(heads=int(L["heads"]), kv_heads=int(L.get("kv_heads", L["heads"])), dim=int(L["dim"]),
+                                 vdim=int(L.get("vdim", L["dim"])), scale=float(L["scale"]), qk_norm=True, qk_norm_joint=True,
+                                 qkv_bias=False, sink=False, gate=False, rot=rot, softcap=float(L["softcap"]), conv_taps=taps(L))
+            split(left.heads, left.kv_heads, "heads")
+            if rot.dims % 2 or rot.dims <= 0 or rot.dims > left.dim:
+                raise ValueError(f"layer {i}: rot.dims {rot.dims} must be even and at most dim {left.dim}")
+            if sc and not (rot.wave_factor > 0 and rot.wave_original > 0 and 0 < rot.wave_low < rot.wave_high):
+                raise ValueError(f"layer {i}: rot.scaling {sc} needs positive factor and original, 0 < low < high")
+            if left.softcap <= 0.0:
+                raise ValueError(f"layer {i}: softcap {left.softcap} must be positive")
+            right = StateSpaceSpec(heads=int(R["heads"]), vdim=int(R["vdim"]), state=int(R["state"]),
+                                   groups=int(R.get("groups", 1)), conv=taps(R), norm_groups=int(R.get("norm_groups", 1)))
+            split(right.heads, right.groups, "heads")
+            split(right.out_width, right.norm_groups, "channels")
+            spec = SideBySideSpec(left=left, right=right, left_scale=0.5, right_scale=0.5, branch_norm=True)
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+        mlp = e.get("mlp")
+        if mlp is not None:
+            if mlp.get("kind") != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+            ro, ex, sh = mlp["router"], mlp["expert"], mlp.get("shared") or None
+            gr = ro.get("groups") or {}
+            moe = MoESpec(experts=int(ro["experts"]), top=int(ro["top"]), ff=int(ex["ff"]), limit=0.0,
+                          scale=float(ro.get("scale", 1.0)), shared_ff=int(sh["ff"]) if sh else 0, renormalize=False, act="silu",
+                          groups=int(gr.get("count", 0)), groups_keep=int(gr.get("keep", 0)))
+            reach = moe.experts
+            if moe.groups:
+                split(moe.experts, moe.groups, "experts")
+                if not 1 <= moe.groups_keep <= moe.groups:
+                    raise ValueError(f"layer {i}: keeps {moe.groups_keep} of {moe.groups} groups")
+                reach = moe.groups_keep * (moe.experts // moe.groups)
+            if not 1 <= moe.top <= reach:
+                raise ValueError(f"layer {i}: top {moe.top} of {reach} experts that can be chosen")
+            mlp = MLPSpec(kind="moe", ff=max(moe.ff, moe.shared_ff), act="silu", moe=moe)
+        src = e.get("weights_of")
+        layers.append(LayerSpec(mixer=spec, mlp=mlp, weights_of=None if src is None else int(src)))
+    for i, l in enumerate(layers):
+        seen, j = {i}, i
+        while layers[j].weights_of is not None:
+            j = layers[j].weights_of
+            if not 0 <= j < len(layers) or j in seen:
+                raise ValueError(f"layer {i}: weights_of must lead to a layer with tensors of its own")
+            seen.add(j)
+        if (layers[j].mixer, layers[j].mlp) != (l.mixer, l.mlp):
+            raise ValueError(f"layer {i}: differs from layer {j}, whose tensors it uses")
+    eos_all = _eos_of(d)
+    return LayerListConfig(architecture="Bovitar", vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers,
+                           norm_eps=float(d["norm"]["eps"]), residual="pre_norm", norm="rms",
+                           logit_scale=float(d.get("logit_scale", 1.0)), eos_token_ids=eos_all,
+                           eos_token_id=eos_all[0] if eos_all else None, bos_token_id=d.get("bos_token_id"))
+
+
+def _bovitar_to_dict(c: "LayerListConfig") -> dict:
+    out = []
+    for l in c.layers:
+        m = l.mixer
+        if m.kind == "delta":
+            kind, mx = "delta", {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "conv": m.conv}
+        else:
+            a, r = m.left, m.right
+            kind = "parallel"
+            mx = {"left": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale,
+                           "softcap": a.softcap, "conv": a.conv_taps, "rot": a.rot.to_dict()},
+                  "right": {"heads": r.heads, "vdim": r.vdim, "state": r.state, "groups": r.groups, "conv": r.conv,
+                            "norm_groups": r.norm_groups}}
+        mlp = None
+        if l.mlp is not None:
+            e = l.mlp.moe
+            mlp = {"kind": "moe", "expert": {"ff": e.ff}, "router": {"experts": e.experts, "top": e.top, "scale": e.scale}}
+            if e.groups:
+                mlp["router"]["groups"] = {"count": e.groups, "keep": e.groups_keep}
+            if e.shared_ff:
+                mlp["shared"] = {"ff": e.shared_ff}
+        entry = {"type": kind, "mixer": mx, "mlp": mlp}
+        if l.weights_of is not None:
+            entry["weights_of"] = l.weights_of
+        out.append(entry)
+    return {"architecture": "Bovitar", "vocab": c.vocab_size, "width": c.hidden_size, "layers": out,
+            "norm": {"eps": c.norm_eps}, "logit_scale": c.logit_scale}
 
 
 # Named shapes used by tests and bench (random-init; there are no checkpoints offline).

@@ -398,6 +398,14 @@ class LayerListLayer:
     decay_up: Optional[torch.Tensor] = None      # bf16 [H*dk, rank]
     decay_bias: Optional[torch.Tensor] = None    # bf16 [H*dk]
     conv_w: Optional[torch.Tensor] = None        # attention: fp32 [taps, channels of q | k | v], the convolutions after the projection
+    # delta rule: proj rows = [q | k | v | gate], gates = [b: H | a: H]; state space (the right half of a side-by-side pair, behind
+    # the attention's q | k | v rows): proj rows = [z | x | B | C], gates = [dt: H].  Both:
+    rec_conv_t: Optional[torch.Tensor] = None    # fp32 [taps, convolved channels]
+    dt_bias: Optional[torch.Tensor] = None       # fp32 [H]
+    decay_rate: Optional[torch.Tensor] = None    # fp32 [H]: exp(A_log)
+    skip: Optional[torch.Tensor] = None          # fp32 [H]: factor of the input added to a head's output
+    left_norm: Optional[torch.Tensor] = None     # [D]: norms of a side-by-side pair's two outputs
+    right_norm: Optional[torch.Tensor] = None
 
 
 @dataclass
@@ -452,10 +460,35 @@ def layer_list_tensor_shapes(cfg) -> Dict[str, tuple]:
             shapes[q + "temp"] = (m.heads,)
         shapes[q + "o"] = (D, m.out_width)
 
+    def conv_attention_shapes(q, m):
+        for n, rows in (("q", m.q_width), ("k", m.kv_heads * m.dim), ("v", m.kv_heads * m.vdim)):
+            shapes[q + n], shapes[q + n + ".conv"] = (rows, D), (rows, m.conv_taps)
+            if n != "v":
+                shapes[q + n + ".norm"] = (rows,) if m.qk_norm_joint else (m.dim,)
+        shapes[q + "o"] = (D, m.out_width)
+
     for l, layer in enumerate(cfg.layers):
         p, m = f"l{l}.", layer.mixer
+        if layer.weights_of is not None:
+            continue
         norm_shapes(p + "norm1")
-        if sandwich:
+        if m.kind == "delta":
+            q = p + "mix."
+            for n, rows in (("q", m.kv_heads * m.dim), ("k", m.kv_heads * m.dim), ("v", m.out_width)):
+                shapes[q + n], shapes[q + n + ".conv"] = (rows, D), (rows, m.conv)
+            shapes[q + "b"] = shapes[q + "a"] = (m.heads, D)
+            shapes[q + "A_log"] = shapes[q + "dt_bias"] = (m.heads,)
+            shapes[q + "g"], shapes[q + "norm"], shapes[q + "o"] = (m.out_width, D), (m.vdim,), (D, m.out_width)
+        elif m.kind == "side_by_side" and m.right.kind == "state_space":
+            r, q = m.right, p + "mix.right."
+            conv_attention_shapes(p + "mix.left.", m.left)
+            shapes[q + "in"] = (r.proj_rows + r.heads, D)
+            shapes[q + "conv"], shapes[q + "conv.b"] = (r.conv_width, r.conv), (r.conv_width,)
+            shapes[q + "dt_bias"] = shapes[q + "A_log"] = shapes[q + "D"] = (r.heads,)
+            shapes[q + "norm"], shapes[q + "o"] = (r.out_width,), (D, r.out_width)
+            if m.branch_norm:
+                shapes[p + "mix.left.out"] = shapes[p + "mix.right.out"] = (D,)
+        elif sandwich:
             shapes[p + "norm1b"] = (D,)
             if taps:
                 shapes[p + "canon1"] = (D, taps)
@@ -487,7 +520,9 @@ def layer_list_tensor_shapes(cfg) -> Dict[str, tuple]:
             continue
         for q in ((1, 2) if layer.mlp is not None else (1,)) if S else ():
             shapes[p + f"hc{q}.in"], shapes[p + f"hc{q}.out"], shapes[p + f"hc{q}.mix"] = (S,), (S,), (S, S)
-        if m.kind == "latent_attention":
+        if m.kind in ("delta", "side_by_side"):
+            pass                       # (above)
+        elif m.kind == "latent_attention":
             if m.q_rank:
                 shapes[p + "mix.dq"], shapes[p + "mix.dq.norm"] = (m.q_rank, D), (m.q_rank,)
                 shapes[p + "mix.uq"] = (m.q_width, m.q_rank)
@@ -600,9 +635,15 @@ def load_layer_list(cfg, get: Callable[[str], torch.Tensor], device: str) -> Lay
 
     def cat8(names):
         """Fused projection rows, zero rows up to a multiple of 8 (16-byte output rows for the tensor-core GEMM)."""
-        w = cat(names)
+        return pad8(cat(names))
+
+    def pad8(w):
         pad = -w.shape[0] % 8
-        return w if not pad else torch.cat([w, torch.zeros(pad, w.shape[1], dtype=BF16, device=device)]).contiguous()
+        return w.contiguous() if not pad else torch.cat([w, torch.zeros(pad, w.shape[1], dtype=BF16, device=device)]).contiguous()
+
+    def conv_t(names):
+        """Convolution weights [channels, taps] of neighbouring channels as ONE fp32 [taps, channels] array."""
+        return cat(names).to(torch.float32).t().contiguous()
 
     def freq_of(rot):
         return torch.tensor(list(rot.frequencies()[0]), dtype=torch.float64).to(device)
@@ -646,7 +687,29 @@ def load_layer_list(cfg, get: Callable[[str], torch.Tensor], device: str) -> Lay
                 lw.gate_up, lw.down = _interleave_rows(g(p + "mlp.gate"), g(p + "mlp.up")), g(p + "mlp.down")
             layers.append(lw)
             continue
-        if m.kind == "latent_attention":
+        if layer.weights_of is not None:       # another layer's tensors (filled in once all of those are loaded)
+            layers.append(None)
+            continue
+        if m.kind == "delta":
+            q = p + "mix."
+            lw = LayerListLayer(norm1=g(p + "norm1"), o=g(q + "o"), out_norm=g(q + "norm"),
+                                proj=cat8([q + n for n in "qkvg"]), gates=cat([q + "b", q + "a"]))
+            lw.rec_conv_t = conv_t([q + n + ".conv" for n in "qkv"])
+            lw.dt_bias, lw.decay_rate = f32(q + "dt_bias"), torch.exp(f32(q + "A_log"))
+        elif m.kind == "side_by_side":
+            a, r, q = m.left, m.right, p + "mix.right."
+            win = g(q + "in")
+            rows = torch.cat([g(p + f"mix.left.{n}") for n in "qkv"] + [win[:r.proj_rows]], dim=0)
+            lw = LayerListLayer(norm1=g(p + "norm1"), o=g(p + "mix.left.o"), o2=g(q + "o"), proj=pad8(rows),
+                                gates=win[r.proj_rows:].contiguous(), out_norm=g(q + "norm"))
+            lw.conv_w = conv_t([p + f"mix.left.{n}.conv" for n in "qkv"])
+            lw.q_norm, lw.k_norm = g(p + "mix.left.q.norm"), g(p + "mix.left.k.norm")
+            lw.rot_freq = freq_of(a.rot)
+            lw.rec_conv_t, lw.rec_conv_bias = conv_t([q + "conv"]), f32(q + "conv.b")
+            lw.dt_bias, lw.decay_rate, lw.skip = f32(q + "dt_bias"), torch.exp(f32(q + "A_log")), f32(q + "D")
+            if m.branch_norm:
+                lw.left_norm, lw.right_norm = g(p + "mix.left.out"), g(p + "mix.right.out")
+        elif m.kind == "latent_attention":
             first = g(p + "mix.dq") if m.q_rank else g(p + "mix.q")
             lw = LayerListLayer(norm1=g(p + "norm1"), proj=torch.cat([first, g(p + "mix.dkv")], dim=0).contiguous(),
                                 o=g(p + "mix.o"))
@@ -665,7 +728,7 @@ def load_layer_list(cfg, get: Callable[[str], torch.Tensor], device: str) -> Lay
             lw = LayerListLayer(norm1=g(p + "norm1"), proj=(cat8 if m.conv_taps else cat)([p + "mix." + n for n in names]),
                                 o=g(p + "mix.o"))
             if m.conv_taps:
-                lw.conv_w = cat([p + f"mix.{n}.conv" for n in "qkv"]).to(torch.float32).t().contiguous()
+                lw.conv_w = conv_t([p + f"mix.{n}.conv" for n in "qkv"])
             if m.plus_one:           # a sink of score zero: exp(0) joins the denominator
                 lw.sink = torch.zeros(m.heads, dtype=torch.float32, device=device)
             if m.qkv_bias:
@@ -728,6 +791,7 @@ def load_layer_list(cfg, get: Callable[[str], torch.Tensor], device: str) -> Lay
             else:
                 lw.gate_up, lw.down = _interleave_rows(g(p + "mlp.gate"), g(p + "mlp.up")), g(p + "mlp.down")
         layers.append(lw)
+    layers = [layers[cfg.weight_owner(l)] for l in range(len(layers))]
     out = LayerListWeights(embed=g("embed"), layers=layers, final_norm=g("final.norm"), lm_head=g("head"),
                            vocab_start=0, vocab_end=cfg.vocab_size)
     if biased:
@@ -803,6 +867,14 @@ def random_layer_list_state(cfg, seed: int = 0, device: str = "cpu") -> Dict[str
             x = 2.0 + x                                   # sigmoid(z) mostly near one: a long memory
         elif leaf.endswith("norm") or leaf in ("norm1", "norm2"):
             x = 1.0 + 0.2 * x
+        elif leaf in ("mix.left.out", "mix.right.out"):
+            x = 1.0 + 0.2 * x                             # norms of a pair's two outputs
+        elif leaf.endswith("dt_bias"):
+            x = -2.0 + x                                  # step sizes spread around a tenth
+        elif leaf.endswith("A_log"):
+            x = -1.0 + x                                  # ... and decays between fast and slow
+        elif leaf.endswith(".D"):
+            x = 1.0 + 0.3 * x
         elif leaf == "mix.f.b":
             x = 3.0 + x
         elif leaf == "mix.sink":
