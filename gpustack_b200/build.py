@@ -42,6 +42,8 @@ SOURCES = [
     "gated_recurrence.cu",
     "gated_linear_attn.cu",
     "conv_attn_prep.cu",
+    "conv_rec_prep.cu",
+    "gated_scan.cu",
 ]
 # What a layer-list decoder (attention with a softmax sink / matrix-memory recurrence, norm after the
 # sum) launches: a fresh checkout that only serves such a model compiles these and nothing else.
@@ -116,8 +118,30 @@ OUTPUT_NORM_SOURCES = [
 ]
 
 
+# What a pre-norm decoder with a norm per sublayer, gated delta rules and attention beside state-space recurrences launches
+PRE_NORM_SOURCES = [
+    "runtime.cu",
+    "elementwise.cu",
+    "gemm_tcgen05.cu",
+    "gemm_simt.cu",
+    "gemm_simt_grouped.cu",
+    "streams.cu",
+    "prenorm.cu",
+    "conv_attn_prep.cu",
+    "conv_rec_prep.cu",
+    "gated_scan.cu",
+    "linear_attn.cu",
+    "attention_sink.cu",
+]
+
+
 def layer_list_sources(mcfg):
     """(tag, sources) of the library a process serving this layer-list model needs."""
+    if getattr(mcfg, "residual", "post_ln") == "pre_norm":
+        routed = any(l.mlp is not None for l in mcfg.layers)
+        tc = any(l.mixer.kind == "side_by_side" and l.mixer.left.tile_sized for l in mcfg.layers)
+        tag = "pre_norm" + ("_routed" if routed else "") + ("_tc" if tc else "")
+        return tag, PRE_NORM_SOURCES + (ROUTED_SOURCES if routed else []) + (ATTENTION_TC_SOURCES if tc else [])
     if getattr(mcfg, "residual", "post_ln") == "output_norm":
         routed = any(l.mlp is not None for l in mcfg.layers)
         tc = any(l.mixer.tile_sized for l in mcfg.layers)

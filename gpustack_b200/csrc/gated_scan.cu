@@ -1,0 +1,438 @@
+// Recurrences on a matrix state per head with ONE decay per head and token, state in fp32.
+//
+//   state space:  S_t = g S_(t-1) + beta k_t v_t^T                      g = exp(-rate softplus(a + bias)), beta = softplus(a + bias)
+//                 o_t = S_t^T q_t + skip v_t
+//   delta rule:   S  <- g S_(t-1);  u = beta (v_t - S^T k_t);  S_t = S + k_t u^T;  o_t = S_t^T q_t
+//                 g = exp(-rate softplus(a + bias)), beta = sigmoid(b)
+// (S: dk x dv, zero before a sequence's first token; head h reads query / key head h / (H / G).)  Queries, keys and values
+// arrive as fp32 rows whose heads are padded with zeros to a multiple of 4 entries (conv_rec_prep.cu); the gates' raw
+// projections are fp32 rows, and everything formed from them is fp32.  The state of slot s is S [slots][H][dv][dkp] (key index
+// fastest, dkp = dk rounded up to 4).  A sequence whose context is empty starts from zero, whatever its slot held.
+//
+// Every value column of S is a recurrence of its own, so columns are the unit of work: L lanes share a column, lane l holds
+// the key entries 4 (i L + l) .. + 3 (i < R4) of it in registers, and a warp walks its 32 / L columns through the sequence's
+// new rows one token after the other.  Per token: S^T k (a butterfly over the L lanes; delta rule only), the update, and
+// the lane's share of S^T q.  Those shares stay in registers for 8 tokens and are then summed over the lanes in one
+// transposing exchange (7 shuffles for 8 tokens).  Keys, queries, values and gates are staged 16 tokens at a time by
+// cp.async into two buffers, so the walk never waits for memory; a column's sums do not depend on how a prompt was cut
+// beyond the order of the lanes' addends in S^T q.
+#include "common.cuh"
+#include "runtime.h"
+#include "../../include/b200.h"
+
+namespace b200 {
+
+constexpr int kGsWarps = 8, kGsTok = 16;
+
+struct GatedScanArgs {
+  const float* x;
+  int64_t ld;
+  int q_col, k_col, v_col;
+  const float* gates;              // [T][ld_g]: delta [b: H | a: H], state space [a: H]
+  int64_t ld_g;
+  const float* rate;               // [H]
+  const float* dt_bias;            // [H]
+  const float* skip;               // [H] or null
+  const int32_t* cu_seq;
+  const int32_t* ctx_lens;
+  const int32_t* state_slots;
+  float* S;
+  float* o;                        // [T][H dv]
+  int H, G, dkp, dv, dvp;
+};
+
+// two fp32 numbers in one 64-bit register pair: the packed fused multiply-add of sm_100
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float a, float b) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ float sum2(f32x2 v) {
+  float a, b;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
+  return a + b;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
+__device__ __forceinline__ float gs_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+
+// (decay, step) of a token from the raw gates
+template <bool DELTA>
+__device__ __forceinline__ float2 gs_gate(float a, float b, float rate, float bias) {
+  const float sp = gs_softplus(a + bias);
+  return make_float2(expf(-rate * sp), DELTA ? 1.0f / (1.0f + expf(-b)) : sp);
+}
+
+__device__ __forceinline__ void cp16(float* dst, const float* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 16;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
+template <int L>
+__device__ __forceinline__ float lanes_sum(float v) {
+#pragma unroll
+  for (int o = L / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+
+// One token of a column: the decayed, updated state and the lane's share of S^T q
+template <int L, int R2, bool DELTA>
+__device__ __forceinline__ float gs_token(f32x2 (&S)[R2], const f32x2 (&k)[R2], const f32x2 (&q)[R2], float v, float2 gb) {
+  float u = gb.y * v;
+  if (DELTA) {
+    f32x2 p0 = mul2(S[0], k[0]), p1 = mul2(S[1], k[1]);
+#pragma unroll
+    for (int i = 2; i < R2; i += 2) {
+      p0 = fma2(S[i], k[i], p0);
+      p1 = fma2(S[i + 1], k[i + 1], p1);
+    }
+    u = gb.y * (v - gb.x * lanes_sum<L>(sum2(p0) + sum2(p1)));
+  }
+  const f32x2 g2 = pack2(gb.x, gb.x), u2 = pack2(u, u);
+  f32x2 o0 = 0, o1 = 0;            // (two positive zeros)
+#pragma unroll
+  for (int i = 0; i < R2; i += 2) {
+    S[i] = fma2(k[i], u2, mul2(g2, S[i]));
+    S[i + 1] = fma2(k[i + 1], u2, mul2(g2, S[i + 1]));
+    o0 = fma2(S[i], q[i], o0);
+    o1 = fma2(S[i + 1], q[i + 1], o1);
+  }
+  return sum2(o0) + sum2(o1);
+}
+
+// 4 R4 entries of a row of key entries: lane l of L takes entries 4 (i L + l) .. + 3
+template <int L, int R4>
+__device__ __forceinline__ void gs_row(const float* __restrict__ row, int l, f32x2 (&r)[2 * R4]) {
+#pragma unroll
+  for (int i = 0; i < R4; ++i) {
+    const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(row + 4 * (i * L + l));
+    r[2 * i] = t.x;
+    r[2 * i + 1] = t.y;
+  }
+}
+
+template <int L, int R4, bool DELTA>
+__global__ void __launch_bounds__(kGsWarps * 32)
+gated_scan_kernel(GatedScanArgs a) {
+  extern __shared__ __align__(16) float smem[];
+  constexpr int R2 = 2 * R4, DKP = 4 * R4 * L, CPW = 32 / L, COLS = kGsWarps * CPW;
+  float* ks = smem;                                   // [2][16][DKP]
+  float* qs = ks + 2 * kGsTok * DKP;                  // [2][16][DKP]
+  float* vs = qs + 2 * kGsTok * DKP;                  // [2][16][COLS]
+  float2* gb = reinterpret_cast<float2*>(vs + 2 * kGsTok * COLS);   // [2][16]
+  float* os = reinterpret_cast<float*>(gb + 2 * kGsTok);            // [16][COLS + 1]
+  const int s = blockIdx.x, h = blockIdx.y, z = blockIdx.z, tid = threadIdx.x;
+  const int slot = a.state_slots[s];
+  if (slot < 0) return;
+  const int t0 = a.cu_seq[s], t1 = a.cu_seq[s + 1];
+  if (t1 <= t0) return;
+  const int warp = tid >> 5, lane = tid & 31, l = lane % L;
+  const int cw = warp * CPW + lane / L, col = z * COLS + cw;         // this lane's column, in the CTA and in the head
+  const int hk = h / (a.H / a.G);
+  const int dkp = a.dkp;
+  float* Sp = a.S + (((size_t)slot * a.H + h) * a.dv + col) * dkp;
+  const bool fresh = a.ctx_lens[s] == 0;
+  f32x2 S[R2];
+#pragma unroll
+  for (int i = 0; i < R4; ++i) {
+    ulonglong2 t = make_ulonglong2(0, 0);
+    if (!fresh && col < a.dv && 4 * (i * L + l) < dkp) t = *reinterpret_cast<const ulonglong2*>(Sp + 4 * (i * L + l));
+    S[2 * i] = t.x;
+    S[2 * i + 1] = t.y;
+  }
+  // key entries behind dkp: zeros in both buffers, written once
+  if (dkp < DKP) {
+    const int pad = DKP - dkp;
+    for (int i = tid; i < 2 * kGsTok * pad; i += kGsWarps * 32) {
+      const int r = i / pad, d = dkp + i % pad;
+      ks[r * DKP + d] = 0.f;
+      qs[r * DKP + d] = 0.f;
+    }
+  }
+  const float rate = a.rate[h], bias = a.dt_bias[h];
+  const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
+  auto stage = [&](int ch, int buf) {                 // rows ch .. ch + 15; rows behind the portion are zeros
+    const int nt = min(kGsTok, t1 - ch), dk4 = dkp >> 2;
+    for (int i = tid; i < kGsTok * dk4; i += kGsWarps * 32) {
+      const int tt = i / dk4, d = (i - tt * dk4) * 4, to = (buf * kGsTok + tt) * DKP + d;
+      if (tt < nt) {
+        const float* row = a.x + (size_t)(ch + tt) * a.ld + hk * dkp + d;
+        cp16(ks + to, row + a.k_col);
+        cp16(qs + to, row + a.q_col);
+      } else {
+        *reinterpret_cast<float4*>(ks + to) = zero4;
+        *reinterpret_cast<float4*>(qs + to) = zero4;
+      }
+    }
+    for (int i = tid; i < kGsTok * (COLS / 4); i += kGsWarps * 32) {
+      const int tt = i / (COLS / 4), c = (i - tt * (COLS / 4)) * 4;
+      float* to = vs + (buf * kGsTok + tt) * COLS + c;
+      if (tt < nt && z * COLS + c < a.dvp) cp16(to, a.x + (size_t)(ch + tt) * a.ld + a.v_col + h * a.dvp + z * COLS + c);
+      else *reinterpret_cast<float4*>(to) = zero4;
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  float ra = 0.f, rb = 0.f;
+  auto raw_gates = [&](int ch) {
+    if (tid < kGsTok && ch + tid < t1) {
+      const float* g = a.gates + (size_t)(ch + tid) * a.ld_g;
+      ra = DELTA ? g[a.H + h] : g[h];
+      if (DELTA) rb = g[h];
+    }
+  };
+  auto put_gates = [&](int ch, int buf) {             // rows behind the portion: decay 1, step 0 (the state stays)
+    if (tid < kGsTok) gb[buf * kGsTok + tid] = ch + tid < t1 ? gs_gate<DELTA>(ra, rb, rate, bias) : make_float2(1.f, 0.f);
+  };
+  stage(t0, 0);
+  raw_gates(t0);
+  put_gates(t0, 0);
+  int buf = 0;
+  for (int ch = t0; ch < t1; ch += kGsTok, buf ^= 1) {
+    const int nt = min(kGsTok, t1 - ch), next = ch + kGsTok;
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                  // this chunk is staged; the last one's outputs have left os
+    if (next < t1) {
+      stage(next, buf ^ 1);
+      raw_gates(next);
+    }
+#pragma unroll 1
+    for (int tb = 0; tb < nt; tb += 8) {
+      float o[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int tt = buf * kGsTok + tb + j;
+        f32x2 k[R2], q[R2];
+        gs_row<L, R4>(ks + tt * DKP, l, k);
+        gs_row<L, R4>(qs + tt * DKP, l, q);
+        o[j] = gs_token<L, R2, DELTA>(S, k, q, vs[tt * COLS + cw], gb[tt]);
+      }
+      // lane l ends with token tb + (l & 7), summed over the column's lanes
+      const bool b4 = l & 4, b2 = l & 2, b1 = l & 1;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float mine = b4 ? o[j + 4] : o[j], other = b4 ? o[j] : o[j + 4];
+        o[j] = mine + __shfl_xor_sync(0xffffffffu, other, 4);
+      }
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        const float mine = b2 ? o[j + 2] : o[j], other = b2 ? o[j] : o[j + 2];
+        o[j] = mine + __shfl_xor_sync(0xffffffffu, other, 2);
+      }
+      {
+        const float mine = b1 ? o[1] : o[0], other = b1 ? o[0] : o[1];
+        o[0] = mine + __shfl_xor_sync(0xffffffffu, other, 1);
+      }
+#pragma unroll
+      for (int w = 8; w < L; w <<= 1) o[0] += __shfl_xor_sync(0xffffffffu, o[0], w);
+      if (l < 8) os[(tb + l) * (COLS + 1) + cw] = o[0];
+    }
+    if (next < t1) put_gates(next, buf ^ 1);
+    __syncthreads();
+    const float sk = a.skip != nullptr ? a.skip[h] : 0.f;
+    for (int i = tid; i < nt * COLS; i += kGsWarps * 32) {
+      const int tt = i / COLS, c = i - tt * COLS;
+      if (z * COLS + c < a.dv)
+        a.o[(size_t)(ch + tt) * a.H * a.dv + h * a.dv + z * COLS + c] =
+            fmaf(sk, vs[(buf * kGsTok + tt) * COLS + c], os[tt * (COLS + 1) + c]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < R4; ++i)
+    if (col < a.dv && 4 * (i * L + l) < dkp)
+      *reinterpret_cast<ulonglong2*>(Sp + 4 * (i * L + l)) = make_ulonglong2(S[2 * i], S[2 * i + 1]);
+}
+
+// Single rows (a decode step): the state, the token's rows and its gates are in flight together; no staging, no barrier.
+template <int L, int R4, bool DELTA>
+__global__ void __launch_bounds__(kGsWarps * 32)
+gated_step_kernel(GatedScanArgs a) {
+  constexpr int R2 = 2 * R4, CPW = 32 / L, COLS = kGsWarps * CPW;
+  const int s = blockIdx.x, h = blockIdx.y, z = blockIdx.z;
+  const int slot = a.state_slots[s];
+  if (slot < 0) return;
+  const int t = a.cu_seq[s];
+  if (a.cu_seq[s + 1] <= t) return;
+  const int lane = threadIdx.x & 31, l = lane % L, col = z * COLS + (threadIdx.x >> 5) * CPW + lane / L;
+  const int hk = h / (a.H / a.G), dkp = a.dkp;
+  const bool live = col < a.dv, fresh = a.ctx_lens[s] == 0;
+  float* Sp = a.S + (((size_t)slot * a.H + h) * a.dv + col) * dkp;
+  const float* row = a.x + (size_t)t * a.ld;
+  f32x2 S[R2], k[R2], q[R2];
+#pragma unroll
+  for (int i = 0; i < R4; ++i) {
+    const int d = 4 * (i * L + l);
+    ulonglong2 ts = make_ulonglong2(0, 0), tk = ts, tq = ts;
+    if (d < dkp) {
+      if (live && !fresh) ts = *reinterpret_cast<const ulonglong2*>(Sp + d);
+      tk = *reinterpret_cast<const ulonglong2*>(row + a.k_col + hk * dkp + d);
+      tq = *reinterpret_cast<const ulonglong2*>(row + a.q_col + hk * dkp + d);
+    }
+    S[2 * i] = ts.x; S[2 * i + 1] = ts.y;
+    k[2 * i] = tk.x; k[2 * i + 1] = tk.y;
+    q[2 * i] = tq.x; q[2 * i + 1] = tq.y;
+  }
+  const float v = live ? row[a.v_col + h * a.dvp + col] : 0.f;
+  const float* g = a.gates + (size_t)t * a.ld_g;
+  const float2 gb = gs_gate<DELTA>(DELTA ? g[a.H + h] : g[h], DELTA ? g[h] : 0.f, a.rate[h], a.dt_bias[h]);
+  const float o = lanes_sum<L>(gs_token<L, R2, DELTA>(S, k, q, v, gb));
+  if (!live) return;
+#pragma unroll
+  for (int i = 0; i < R4; ++i) {
+    const int d = 4 * (i * L + l);
+    if (d < dkp) *reinterpret_cast<ulonglong2*>(Sp + d) = make_ulonglong2(S[2 * i], S[2 * i + 1]);
+  }
+  if (l == 0) a.o[(size_t)t * a.H * a.dv + h * a.dv + col] = a.skip != nullptr ? fmaf(a.skip[h], v, o) : o;
+}
+
+template <int L, int R4, bool DELTA>
+int gated_scan_launch(const GatedScanArgs& a, int n_seqs, int max_len, cudaStream_t s) {
+  constexpr int COLS = kGsWarps * (32 / L), DKP = 4 * R4 * L;
+  const dim3 grid(n_seqs, a.H, (a.dv + COLS - 1) / COLS);
+  if (max_len == 1) {
+    gated_step_kernel<L, R4, DELTA><<<grid, kGsWarps * 32, 0, s>>>(a);
+    return b200_check_launch("b200_gated_scan(step)");
+  }
+  constexpr size_t smem = sizeof(float) * (4 * (size_t)kGsTok * DKP + 2 * kGsTok * COLS + 4 * kGsTok + kGsTok * (COLS + 1));
+  if (smem > 48 * 1024) {
+    const cudaError_t e = cudaFuncSetAttribute(gated_scan_kernel<L, R4, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) {
+      b200_set_error("gated_scan: %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
+      return B200_ERR_CUDA;
+    }
+  }
+  gated_scan_kernel<L, R4, DELTA><<<grid, kGsWarps * 32, smem, s>>>(a);
+  return b200_check_launch("b200_gated_scan");
+}
+
+template <bool DELTA>
+int gated_scan_pick(const GatedScanArgs& a, int n_seqs, int max_len, cudaStream_t s) {
+  if (a.dkp <= 32) return gated_scan_launch<8, 1, DELTA>(a, n_seqs, max_len, s);
+  if (a.dkp <= 64) return gated_scan_launch<8, 2, DELTA>(a, n_seqs, max_len, s);
+  if (a.dkp <= 96) return gated_scan_launch<8, 3, DELTA>(a, n_seqs, max_len, s);
+  if (a.dkp <= 128) return gated_scan_launch<8, 4, DELTA>(a, n_seqs, max_len, s);
+  if (a.dkp <= 256) return gated_scan_launch<16, 4, DELTA>(a, n_seqs, max_len, s);
+  return gated_scan_launch<32, 4, DELTA>(a, n_seqs, max_len, s);
+}
+
+// ------------------------------------------------------------------------------------------- out
+// out = RMSnorm over `parts` equal pieces of (y * silu(z)), times w: the gate comes BEFORE the norm.  One CTA per row; the
+// gated row is staged in shared memory between the statistic and the product.
+template <typename TA>
+__device__ __forceinline__ float4 gs_ld4(const TA* p);
+template <>
+__device__ __forceinline__ float4 gs_ld4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <>
+__device__ __forceinline__ float4 gs_ld4<bf16>(const bf16* p) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  return make_float4(bf16_lo(r.x), bf16_hi(r.x), bf16_lo(r.y), bf16_hi(r.y));
+}
+__device__ __forceinline__ float gs_ld1(const float* p) { return *p; }
+__device__ __forceinline__ float gs_ld1(const bf16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void gs_st1(float* p, float v) { *p = v; }
+__device__ __forceinline__ void gs_st1(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ void gs_st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void gs_st4(bf16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
+__device__ __forceinline__ float gs_silu(float z) { return z / (1.0f + expf(-z)); }
+
+constexpr int kGnThreads = 256;
+
+template <typename TA, bool VEC>
+__global__ void __launch_bounds__(kGnThreads)
+gate_norm_kernel(const float* __restrict__ y, const TA* __restrict__ proj, int64_t ld, int z_col, const bf16* __restrict__ w,
+                 TA* out, int64_t ldo, int C, int parts, float eps) {
+  extern __shared__ __align__(16) float row[];        // [C], then the warps' partial sums
+  __shared__ float sums[kGnThreads / 32];
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  constexpr int NW = kGnThreads / 32, V = VEC ? 4 : 1;
+  const float* yr = y + (size_t)t * C;
+  const TA* zr = proj + (size_t)t * ld + z_col;
+  TA* o = out + (size_t)t * ldo;
+  const int W = C / parts, per = parts >= NW ? 1 : NW / parts;       // warps that share a part
+  for (int p0 = 0; p0 < parts; p0 += NW / per) {
+    const int p = p0 + warp / per, sub = warp % per;
+    const bool live = p < parts && warp / per < NW / per;
+    float ss = 0.f;
+    if (live)
+      for (int i = (sub * 32 + lane) * V; i < W; i += per * 32 * V) {
+        const int c = p * W + i;
+        if (VEC) {
+          float4 v = *reinterpret_cast<const float4*>(yr + c);
+          const float4 g = gs_ld4<TA>(zr + c);
+          v.x *= gs_silu(g.x); v.y *= gs_silu(g.y); v.z *= gs_silu(g.z); v.w *= gs_silu(g.w);
+          *reinterpret_cast<float4*>(row + c) = v;
+          ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+        } else {
+          const float v = yr[c] * gs_silu(gs_ld1(zr + c));
+          row[c] = v;
+          ss = fmaf(v, v, ss);
+        }
+      }
+    ss = warp_sum(ss);
+    if (per > 1) {
+      if (lane == 0) sums[warp] = ss;
+      __syncthreads();
+      if (live) {
+        ss = 0.f;
+        for (int i = 0; i < per; ++i) ss += sums[warp - sub + i];    // the same order in every warp
+      }
+    }
+    if (!live) continue;
+    const float rstd = 1.0f / sqrtf(ss / (float)W + eps);
+    for (int i = (sub * 32 + lane) * V; i < W; i += per * 32 * V) {  // (each thread reads back what it staged itself)
+      const int c = p * W + i;
+      if (VEC) {
+        float4 v = *reinterpret_cast<const float4*>(row + c);
+        const float4 g = gs_ld4<bf16>(w + c);
+        gs_st4(o + c, make_float4(v.x * rstd * g.x, v.y * rstd * g.y, v.z * rstd * g.z, v.w * rstd * g.w));
+      } else {
+        gs_st1(o + c, row[c] * rstd * gs_ld1(w + c));
+      }
+    }
+  }
+}
+
+}  // namespace b200
+
+using namespace b200;
+
+extern "C" int b200_gated_scan(const float* x, int64_t ld, int q_col, int k_col, int v_col, const float* gates, int64_t ld_g,
+                               const float* rate, const float* dt_bias, const float* skip, const int32_t* cu_seq,
+                               const int32_t* ctx_lens, const int32_t* state_slots, float* S, float* o_raw, int n_seqs, int H,
+                               int G, int dk, int dv, int delta, int max_len, void* stream) {
+  B200_REQUIRE(n_seqs >= 0 && H > 0 && G > 0 && H % G == 0 && dk > 0 && dv > 0 && dk <= 512,
+               "gated_scan: bad shape H=%d G=%d dk=%d dv=%d (dk <= 512)", H, G, dk, dv);
+  B200_REQUIRE(((ld | q_col | k_col | v_col) & 3) == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(S)) & 15) == 0,
+               "gated_scan: rows, columns and state in whole 16-byte pieces");
+  if (n_seqs == 0) return B200_OK;
+  const GatedScanArgs a{x, ld, q_col, k_col, v_col, gates, ld_g, rate, dt_bias, skip, cu_seq, ctx_lens, state_slots, S, o_raw, H, G,
+                        (dk + 3) & ~3, dv, (dv + 3) & ~3};
+  cudaStream_t s = (cudaStream_t)stream;
+  return delta ? gated_scan_pick<true>(a, n_seqs, max_len, s) : gated_scan_pick<false>(a, n_seqs, max_len, s);
+}
+
+extern "C" int b200_gate_norm(const float* y, const void* proj, int f32, int64_t ld, int z_col, const void* w, void* out,
+                              int64_t ldo, int T, int C, int parts, float eps, void* stream) {
+  B200_REQUIRE(T >= 0 && C > 0 && parts > 0 && C % parts == 0, "gate_norm: %d channels in %d parts", C, parts);
+  if (T == 0) return B200_OK;
+  const size_t smem = sizeof(float) * (size_t)C;
+  B200_REQUIRE(smem <= 48 * 1024, "gate_norm: %d channels exceed the staged row (12288)", C);
+  cudaStream_t s = (cudaStream_t)stream;
+  auto al = [](const void* p, int n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; };
+  const int n = f32 ? 16 : 8;
+  const bool vec = (C / parts) % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 && z_col % 4 == 0 && al(y, 16) && al(proj, n) && al(out, n) && al(w, 8);
+#define B200_GN(TA, V) \
+  gate_norm_kernel<TA, V><<<T, kGnThreads, smem, s>>>(y, (const TA*)proj, ld, z_col, (const bf16*)w, (TA*)out, ldo, C, parts, eps)
+  if (f32) { if (vec) B200_GN(float, true); else B200_GN(float, false); }
+  else { if (vec) B200_GN(bf16, true); else B200_GN(bf16, false); }
+#undef B200_GN
+  return b200_check_launch("b200_gate_norm");
+}

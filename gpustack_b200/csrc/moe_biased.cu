@@ -7,6 +7,8 @@
 //                      are the chosen scores as they are (times scale), not renormalised.
 //                      A third form chooses by z + correction (here the router's learned bias, part of the logit) and
 //                      weights with the softmax over the chosen logits alone.
+//                      With groups the outputs form equal groups of neighbours: only outputs of the groups_keep groups
+//                      with the largest choice scores (the best one in each) can be chosen, ties to the lowest index.
 //   moe_combine_mixed: out[t] = sum_j ( id_j < n_real ? yp[pair_row[t K + j]] : w_j * x[t] ) (+ shared[t]).
 //                      Routed rows arrive already multiplied by their weight (the down projection's row
 //                      scale); an identity expert returns the layer input itself times the weight.  fp32 sum in a
@@ -31,7 +33,8 @@ __device__ __forceinline__ float rb_f32(bf16 v) { return __bfloat162float(v); }
 __global__ void __launch_bounds__(128)
 moe_route_biased_kernel(const float* __restrict__ logits, int64_t ld, const float* __restrict__ correction,
                         int32_t* __restrict__ topk_ids, float* __restrict__ topk_w, int T, int E, int K, float scale,
-                        int score_mode, int renormalize) {
+                        int score_mode, int renormalize, int groups, int groups_keep) {
+  __shared__ float gc[4][32 * kRbPerLane], gbest[4][32 * kRbPerLane];    // choice scores, best of every group
   const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (t >= T) return;
   float s[kRbPerLane], c[kRbPerLane];
@@ -75,6 +78,32 @@ moe_route_biased_kernel(const float* __restrict__ logits, int64_t ld, const floa
       const int e = lane + 32 * i;
       s[i] *= inv;
       c[i] = e < E ? s[i] + (correction != nullptr ? correction[e] : 0.f) : -CUDART_INF_F;
+    }
+  }
+  if (groups > 1 && groups_keep < groups) {
+    float* cs = gc[threadIdx.x >> 5];
+    float* gs = gbest[threadIdx.x >> 5];
+    const int n = E / groups;
+#pragma unroll
+    for (int i = 0; i < kRbPerLane; ++i)
+      if (lane + 32 * i < E) cs[lane + 32 * i] = c[i];
+    __syncwarp();
+    for (int g = lane; g < groups; g += 32) {
+      float b = cs[g * n];
+      for (int j = 1; j < n; ++j) b = fmaxf(b, cs[g * n + j]);
+      gs[g] = b;
+    }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < kRbPerLane; ++i) {
+      const int e = lane + 32 * i;
+      if (e < E) {
+        const int g = e / n;
+        const float mine = gs[g];
+        int ahead = 0;
+        for (int j = 0; j < groups; ++j) ahead += (gs[j] > mine || (gs[j] == mine && j < g)) ? 1 : 0;
+        if (ahead >= groups_keep) c[i] = -CUDART_INF_F;
+      }
     }
   }
   float wsum = 0.f, mine_w = 0.f, top_z = 0.f;
@@ -134,17 +163,25 @@ moe_combine_mixed_kernel(const TP* __restrict__ yp, int64_t ldp, const int32_t* 
 
 using namespace b200;
 
-extern "C" int b200_moe_route_scored(const float* logits, int64_t ld, const float* correction, int32_t* topk_ids,
-                                     float* topk_w, int T, int E, int K, float scale, int score_mode,
-                                     int renormalize, void* stream) {
+extern "C" int b200_moe_route_grouped(const float* logits, int64_t ld, const float* correction, int32_t* topk_ids,
+                                      float* topk_w, int T, int E, int K, float scale, int score_mode, int renormalize,
+                                      int groups, int groups_keep, void* stream) {
   B200_REQUIRE(ld >= E, "moe_route_biased: row stride %lld < E=%d", (long long)ld, E);
   B200_REQUIRE(T >= 0 && E >= 1 && E <= 32 * kRbPerLane && K >= 1 && K <= kRbMaxTop && K <= E,
                "moe_route_biased: unsupported E=%d K=%d (E <= %d, K <= %d)", E, K, 32 * kRbPerLane, kRbMaxTop);
   B200_REQUIRE(score_mode >= 0 && score_mode <= 2, "moe_route_biased: unknown score form %d", score_mode);
+  B200_REQUIRE(groups == 0 || (groups > 0 && E % groups == 0 && groups_keep >= 1 && groups_keep <= groups && K <= groups_keep * (E / groups)),
+               "moe_route_biased: %d of %d groups of %d outputs, K=%d", groups_keep, groups, E, K);
   if (T == 0) return B200_OK;
   moe_route_biased_kernel<<<(T + 3) / 4, 128, 0, (cudaStream_t)stream>>>(logits, ld, correction, topk_ids, topk_w, T, E, K,
-                                                                       scale, score_mode, renormalize);
+                                                                       scale, score_mode, renormalize, groups, groups_keep);
   return b200_check_launch("b200_moe_route_biased");
+}
+
+extern "C" int b200_moe_route_scored(const float* logits, int64_t ld, const float* correction, int32_t* topk_ids,
+                                     float* topk_w, int T, int E, int K, float scale, int score_mode,
+                                     int renormalize, void* stream) {
+  return b200_moe_route_grouped(logits, ld, correction, topk_ids, topk_w, T, E, K, scale, score_mode, renormalize, 0, 0, stream);
 }
 
 extern "C" int b200_moe_route_biased(const float* logits, int64_t ld, const float* correction, int32_t* topk_ids,

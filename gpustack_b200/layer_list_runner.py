@@ -1,5 +1,5 @@
 """Model runner of the layer-list decoders (config.LayerListConfig: Vodavik, Danipel, Resevik, Dotorax,
-Kerarax).
+Kerarax, Bovitar).
 
 Same step interface as runner.ModelRunner -- the engine, the scheduler's plans, the staging buffer, CUDA-graph
 decode steps and the sampler are shared -- with this family's layer sequence:
@@ -32,6 +32,11 @@ decode steps and the sampler are shared -- with this family's layer sequence:
                    kernels with capped scores and one more in the softmax denominator.  In bf16 the heads are laid out at a
                    tensor-core tile width (zero columns behind dim / vdim), whatever dim and vdim are.
 
+  delta mixer:     fp32 gate projection -> conv_rec_prep (causal convolution with its ring, silu, unit norms -> fp32 q | k | v
+                   rows) -> gated_scan (delta rule, state slot in / out, fp32) -> per-head norm x silu gate.
+  side-by-side mixer with a state-space half:  attention as above beside [conv_rec_prep of x | B | C -> gated_scan ->
+                   silu gate x grouped norm], two output projections; the join that follows norms both and adds them.
+
 Residual schemes (config.residual): "post_ln" as drawn above; "parallel": pre-norm with ONE RMS norm per layer,
 
     embed * scale -> per layer run [ x += branches of the layer before (+ embedding before a repeated pass) ; h = RMSnorm(x)
@@ -59,7 +64,12 @@ decay per key channel and token.  "output_norm": a norm on every sublayer's outp
           -> x += LN(last output) -> LN of the wanted rows -> lm_head -> capped logits (in the sampler's pass)
 
 where ONE output_norm_join launch does the norm, the sum and the rounding -- for a routed feed-forward also the sum over
-the chosen experts and the gated shared expert.
+the chosen experts and the gated shared expert.  "pre_norm": a norm in front of every sublayer,
+
+    embed -> per sublayer [ x += output of the sublayer before ; h = RMSnorm(x) -> sublayer ] -> x += last output -> RMSnorm
+
+where ONE prenorm_join launch takes in the output (a pair of mixers' outputs through their norms, or a routed feed-forward's
+expert rows) and norms the sum for the next sublayer.  A layer may use another layer's tensors (LayerSpec.weights_of).
 
 Feed-forwards:
 relu^2 (ungated), gated GELU, a clamped gated unit, or a routed mixture of clamped gated experts with identity experts
@@ -113,6 +123,8 @@ class LayerListRunner(ModelRunner):
                                 and ops.attn_prefill_tile(m.heads, m.kv_heads) == self.prefill_tile) for l, m in attn}
         # ... and single rows on the split-KV decode kernel in the same way
         self.pool_dec = {l: bool(bf and ops.LAYER_LIST_TC and m.pool and m.tokens_tile_sized) for l, m in attn}
+        # an attention mixer whose q, k and v are convolved prepares its rows in one launch of its own (see _attend)
+        conv = [(l, m) for l, m in attn if m.conv_taps]
         if self.prefill_tile % base:
             raise B200Error("prefill tile sizes of the attention kernels do not nest")
         self._dec_ws = {}
@@ -120,6 +132,7 @@ class LayerListRunner(ModelRunner):
         self.parallel = cfg.residual == "parallel"
         self.sandwich = cfg.residual == "sandwich"
         self.output_norm = cfg.residual == "output_norm"
+        self.pre_norm = cfg.residual == "pre_norm"
         self.canon_taps = getattr(cfg, "canon_taps", 0)
         self.runs = cfg.runs()                 # [(layer, embedding added before it)]: caches and state belong to a run
         self.looped = any(again for _, again in self.runs)
@@ -128,11 +141,14 @@ class LayerListRunner(ModelRunner):
         self.proj_width = max(lw.proj.shape[0] for lw in self.w.layers)
         self.mix_width = max(l.mixer.out_width for l in cfg.layers)
         # attention over convolved q, k, v: prepared queries in rows of their own, heads at the cache's widths
-        conv = [(l, x.mixer) for l, x in enumerate(cfg.layers) if x.mixer.kind == "attention" and x.mixer.conv_taps]
         self.q_rows_width = max([m.heads * m.cache_widths(bf)[0] for _, m in conv] or [0])
-        self.mix_width = max([self.mix_width] + [m.heads * m.cache_widths(bf)[1] for _, m in conv])
+        self.mix_width = max([self.mix_width] + [m.heads * m.cache_widths(bf)[1] + self._right_width(cfg.layers[l].mixer)
+                                                 for l, m in conv])
         self.o_padded = {l: pad_head_columns(self.w.layers[l].o, m.heads, m.vdim, m.cache_widths(bf)[1]) for l, m in conv
-                         if m.cache_widths(bf)[1] != m.vdim}
+                         if m.cache_widths(bf)[1] != m.vdim and cfg.layers[l].weights_of is None}
+        for l, x in enumerate(cfg.layers):               # (a layer that uses another's tensors uses its padded copy too)
+            if x.weights_of is not None and cfg.weight_owner(l) in self.o_padded:
+                self.o_padded[l] = self.o_padded[cfg.weight_owner(l)]
         self.ff_width = max([(l.mlp.moe.shared_ff if l.mlp.kind == "moe" else l.mlp.ff) for l in cfg.layers
                              if l.mlp is not None] or [0])
         lat = [l.mixer for l in cfg.layers if l.mixer.kind == "latent_attention"]
@@ -144,17 +160,25 @@ class LayerListRunner(ModelRunner):
         rec = [l.mixer for l in cfg.layers if l.mixer.kind == "mlstm"]
         lin = [l.mixer for l in cfg.layers if l.mixer.kind in ("linear_attention", "gated_linear_attention")]
         gla = [l.mixer for l in cfg.layers if l.mixer.kind == "gated_linear_attention"]
-        gdr = [l.mixer.right for l in cfg.layers if l.mixer.kind == "side_by_side"]
+        pairs = [l.mixer for l in cfg.layers if l.mixer.kind == "side_by_side"]
+        gdr = [m.right for m in pairs if m.right.kind == "gated_recurrence"]
+        scans = [l.mixer for l in cfg.layers if l.mixer.kind == "delta"] + [m.right for m in pairs if m.right.kind == "state_space"]
         # (a side-by-side mixer's attention also parks its rows' log-sum-exp here, one number per head)
         self.gate_width = max([2 * m.heads for m in rec] + [m.heads * m.dim for m in gla] + [2 * m.width for m in gdr]
-                              + [l.mixer.left.heads for l in cfg.layers if l.mixer.kind == "side_by_side"] or [0])
-        self.rec_width = max([m.out_width for m in rec + lin] or [0])
-        self.lin_width = max([2 * m.heads * m.dim + m.out_width for m in lin] + [m.width for m in gdr] or [0])
+                              + [m.left.heads for m in pairs] + [2 * m.heads for m in scans] or [0])
+        self.rec_width = max([m.out_width for m in rec + lin + scans] or [0])
+        self.lin_width = max([2 * m.heads * m.dim + m.out_width for m in lin] + [m.width for m in gdr]
+                             + [m.row_width for m in scans] or [0])
         self.state: List[Optional[tuple]] = [None] * len(self.runs)
         self.canon_ring: List[Optional[tuple]] = [None] * len(self.runs)   # input-convolution rings (mixer, feed-forward) per run
         self.pool_k: List[Optional[torch.Tensor]] = [None] * len(self.runs)
         self.pool_v: List[Optional[torch.Tensor]] = [None] * len(self.runs)
         self.num_state_slots = 0
+
+    @staticmethod
+    def _right_width(m) -> int:
+        """Columns the right half of a side-by-side mixer needs in the buffer of mixer outputs."""
+        return m.right.out_width if m.kind == "side_by_side" else 0
 
     def _alloc_model_buffers(self):
         dev, T, D = self.device, self.max_tokens, self.H
@@ -170,10 +194,12 @@ class LayerListRunner(ModelRunner):
         self.gates = e(T * max(1, self.gate_width), dt=torch.float32)
         self.o_raw = e(T * max(1, self.rec_width), dt=torch.float32)
         self.lin32 = e(T * max(1, self.lin_width), dt=torch.float32)   # prepared q | k | v rows of a linear-attention mixer
-        gdr = [l.mixer.right.width for l in self.mcfg.layers if l.mixer.kind == "side_by_side"]
+        gdr = [l.mixer.right.width for l in self.mcfg.layers
+               if l.mixer.kind == "side_by_side" and l.mixer.right.kind == "gated_recurrence"]
         self.rec_ws = ops.gated_recurrence_workspace(T, self.max_seqs, max(gdr), dev) if gdr else None
-        if self.sandwich:
+        if self.sandwich or self.pre_norm:
             self.y2 = e(T, D, dt=torch.float32)           # the second output of a side-by-side mixer
+        if self.sandwich:
             self.h32 = e(T, D, dt=torch.float32)          # a sublayer's normed input before its convolution
         if self.parallel:
             self.y2 = e(T, D, dt=torch.float32)           # the feed-forward's output beside the mixer's (self.y)
@@ -206,6 +232,7 @@ class LayerListRunner(ModelRunner):
             m = cfg.layers[li].mixer
             if m.kind == "side_by_side":
                 m = m.left
+            if m.kind == "attention" and m.pool:
                 per_page = m.pool_per_page(self.block_size)
                 # mean key / value of every block of m.pool tokens, fp32, addressed through the KV block table
                 self.pool_k[l] = torch.zeros(num_blocks, m.kv_heads, per_page, m.dim, dtype=torch.float32, device=self.device)
@@ -239,7 +266,15 @@ class LayerListRunner(ModelRunner):
                 self.canon_ring[l] = (f(num_slots, R, D), f(num_slots, R, D) if self.mcfg.layers[li].mlp is not None else None)
             if m.kind == "attention" and m.conv_taps > 1:    # ring of the last projected rows, by position mod (taps - 1)
                 self.state[l] = (f(num_slots, m.conv_taps - 1, m.qkv_width),)
-            if m.kind == "side_by_side":             # S [slots, W], and the ring of its convolution's last inputs
+            if m.kind == "delta":                    # S [slots, H, dv, dk], and the ring of its convolutions' last inputs
+                self.state[l] = (f(num_slots, m.heads, m.vdim, m.state_width // (m.heads * m.vdim)),
+                                 f(num_slots, m.conv - 1, m.conv_width) if m.conv > 1 else None)
+            if m.kind == "side_by_side" and m.right.kind == "state_space":       # ... and the ring of the attention's convolutions
+                r, a = m.right, m.left
+                self.state[l] = (f(num_slots, r.heads, r.vdim, r.state_width // (r.heads * r.vdim)),
+                                 f(num_slots, r.conv - 1, r.conv_width) if r.conv > 1 else None,
+                                 f(num_slots, a.conv_taps - 1, a.qkv_width) if a.conv_taps > 1 else None)
+            elif m.kind == "side_by_side":           # S [slots, W], and the ring of its convolution's last inputs
                 r = m.right
                 self.state[l] = (f(num_slots, r.width), f(num_slots, r.conv - 1, r.width) if r.conv > 1 else None)
             if m.kind in ("linear_attention", "gated_linear_attention"):         # S [slots, H, dv, dk]
@@ -276,6 +311,11 @@ class LayerListRunner(ModelRunner):
             ops.embed_sinusoid(ids, self._pos[:T], self.w.embed, self.w.pos_freq, self.resid32[:T],
                                norm=(self.w.embed_norm, self.w.embed_norm_b), eps=self.mcfg.norm_eps, xb_out=self.xb[:T])
             self._pending = None
+            self.stats["kernel_launches"] += 1
+            return
+        if self.pre_norm:      # the first layer's norm follows in its own join
+            ops.embed_streams(ids, self.w.embed, self.resid32[:T], 1, self.mcfg.embed_scale)
+            self._pending = {}
             self.stats["kernel_launches"] += 1
             return
         if self.parallel:      # the first layer's norm reads the embedding output; a repeated span adds it again
@@ -331,6 +371,23 @@ class LayerListRunner(ModelRunner):
         ops.sandwich_join(self.resid32[:T], cfg.norm_eps, y=y, y2=y2, ya=ya, yb=yb, post_w=post_w, mult=cfg.residual_mult,
                           x_out=self.resid32[:T])
         self._pending = None
+        self.layer_trace.append(self.resid32[:T].clone())
+
+    def _prenorm_open(self, T: int, norm_w) -> None:
+        """Pre-norm residual: the output of the sublayer before (self._pending = the join's argument) enters the fp32 stream
+        and the sum is normed into self.xb for the next sublayer."""
+        ops.prenorm_join(self.resid32[:T], norm_w, self.mcfg.norm_eps, x_out=self.resid32[:T] if self._pending else None,
+                         h_out=self.xb[:T], **self._pending)
+        self._pending = {}
+        self.stats["kernel_launches"] += 1
+
+    def _prenorm_close(self, T: int) -> None:
+        """Materialise the stream after a layer (tracing only: on the serving path the next sublayer's join does it)."""
+        if self.layer_trace is None:
+            return
+        if self._pending:
+            ops.prenorm_join(self.resid32[:T], None, self.mcfg.norm_eps, x_out=self.resid32[:T], **self._pending)
+            self._pending = {}
         self.layer_trace.append(self.resid32[:T].clone())
 
     def _take_output(self, T: int) -> None:
@@ -407,10 +464,23 @@ class LayerListRunner(ModelRunner):
                 self._open_layer(T, l, lw, again)
             if self.output_norm:
                 self._take_output(T)
+            if self.pre_norm:
+                self._prenorm_open(T, lw.norm1)
             if self.sandwich:
                 ring = self.canon_ring[l] or (None, None)
                 self._sandwich_open(T, lw.norm1, lw.canon1, ring[0], cu_all, ctx_all, slots_all)
             ops.linear(self.xb[:T], lw.proj, proj)
+            if self.pre_norm:
+                args = (l, m, lw, proj, out, T, Tp, Bd, nt, bt_p, cu_p, ctx_p, ts, tq, lens_d, bt_d, cu_all, ctx_all, slots_all)
+                if m.kind == "delta":
+                    self._delta(*args)
+                else:
+                    self._attention_beside_scan(*args)
+                if layer.mlp is not None:
+                    self._prenorm_open(T, lw.norm2)
+                    self._pending = {"routed": self._routed_rows(T, layer.mlp.moe, lw)[:4]}
+                self._prenorm_close(T)
+                continue
             if m.kind == "side_by_side":
                 self._side_by_side(l, m, lw, proj, out, T, Tp, Bd, nt, bt_p, cu_p, ctx_p, ts, tq, lens_d, bt_d, cu_all, ctx_all,
                                    slots_all)
@@ -446,9 +516,8 @@ class LayerListRunner(ModelRunner):
                     wk, wv = self.k_cache[l].shape[3], self.v_cache[l].shape[3]
                     q, out = self._view(self.q_rows, T, H * wk), self._view(self.mix_out, T, H * wv)
                     wo = self.o_padded.get(li, wo)
-                    ops.conv_attn_prep(proj, lw.conv_w, lw.q_norm, lw.k_norm, self.state[l][0] if self.state[l] else None, cu_all,
-                                       ctx_all, slots_all, ts, tq, self.prefill_tile, cu_p.shape[0] - 1 if nt else 0, Bd, slots, q,
-                                       self.k_cache[l], self.v_cache[l], H, G, dk, dv, eps)
+                    self._conv_attention_rows(l, m, lw, proj, q, self.state[l][0] if self.state[l] else None, Bd, nt, cu_p, ts, tq,
+                                              cu_all, ctx_all, slots_all)
                     dk, dv = wk, wv
                 elif m.rot is not None or m.values_are_keys or m.qk_unit_norm:
                     # rotation, then the weightless q / k norm; keys to their pages, values = the keys as projected
@@ -463,26 +532,8 @@ class LayerListRunner(ModelRunner):
                                   self.v_cache[l] if own else None, H, G, dk, dv, eps, m.q_temp_coef, m.q_temp_every)
                 kv_cols = 0 if not own else (G * dk if m.values_are_keys else G * (dk + dv))
                 gate_col = (H * dk + kv_cols) if m.gate else -1
-                kc, vc = self.k_cache[l], self.v_cache[l]
-                if nt and self.fast_prefill[li]:
-                    ops.paged_attn_prefill_ex(q[:Tp], q.stride(0), kc, vc, bt_p, cu_p, ctx_p, ts, tq, out[:Tp], H, G, dk,
-                                              m.scale, sink=lw.sink, gate=proj[:Tp, gate_col:] if m.gate else None,
-                                              window=m.window, gate_per_head=m.gate_per_head, softcap=m.softcap)
-                elif nt:
-                    ops.attn_sink_prefill(q[:Tp], gate_col, kc, vc, bt_p, cu_p, ctx_p, ts, tq, lw.sink, out[:Tp],
-                                          H, G, dk, dv, m.scale, tile_rows=self.prefill_tile, window=m.window,
-                                          gate_per_head=m.gate_per_head, head_scale=lw.head_scale, softcap=m.softcap)
-                if Bd and self.fast_decode[li]:
-                    splits, ws = self._decode_plan(Bd, m)
-                    ops.paged_attn_decode(q[Tp:T], q.stride(0), kc, vc, bt_d, lens_d, out[Tp:T], H, G, dk, m.scale,
-                                          num_splits=splits, workspace=ws, sink=lw.sink,
-                                          gate=proj[Tp:T, gate_col:] if m.gate else None, window=m.window,
-                                          gate_per_head=m.gate_per_head, softcap=m.softcap)
-                elif Bd:
-                    ops.attn_sink_decode(q[Tp:T], gate_col, kc, vc, bt_d, lens_d, lw.sink, out[Tp:T], H, G, dk, dv,
-                                         m.scale, window=m.window, gate_per_head=m.gate_per_head, head_scale=lw.head_scale,
-                                         softcap=m.softcap)
-                self.stats["kernel_launches"] += 2 + (1 if nt else 0) + (1 if Bd else 0)
+                self._attend(l, m, lw, q, proj, gate_col, out, T, Tp, Bd, nt, bt_p, cu_p, ctx_p, ts, tq, lens_d, bt_d, dk, dv)
+                self.stats["kernel_launches"] += 2
             elif m.kind == "linear_attention":
                 H, dk, dv = m.heads, m.dim, m.vdim
                 kc, vc = H * dk, 2 * H * dk
@@ -534,6 +585,83 @@ class LayerListRunner(ModelRunner):
             if layer.mlp is not None:
                 self._feed_forward(T, layer.mlp, lw)
                 self._join(T, li, 2)
+
+    def _conv_attention_rows(self, l, m, lw, proj, q, ring, Bd, nt, cu_p, ts, tq, cu_all, ctx_all, slots_all) -> None:
+        """Convolution, norm and rotation of the projected rows: queries to q, keys and values to their pages."""
+        ops.conv_attn_prep(proj, lw.conv_w, lw.q_norm, lw.k_norm, ring, cu_all, ctx_all, slots_all, ts, tq, self.prefill_tile,
+                           cu_p.shape[0] - 1 if nt else 0, Bd, self._slots, q, self.k_cache[l], self.v_cache[l], m.heads, m.kv_heads,
+                           m.dim, m.vdim, self.mcfg.norm_eps, joint_norm=m.qk_norm_joint, rot_dims=m.rot.dims if m.rot is not None else 0,
+                           half_layout=m.rot is not None and m.rot.layout == "half", freq=lw.rot_freq)
+
+    def _attend(self, l, m, lw, q, proj, gate_col, out, T, Tp, Bd, nt, bt_p, cu_p, ctx_p, ts, tq, lens_d, bt_d, dk, dv) -> None:
+        """Attention of prepared queries over the run's pages (heads laid out dk / dv wide): prompt portions, then single rows."""
+        li, H, G = self.runs[l][0], m.heads, m.kv_heads
+        kc, vc = self.k_cache[l], self.v_cache[l]
+        if nt and self.fast_prefill[li]:
+            ops.paged_attn_prefill_ex(q[:Tp], q.stride(0), kc, vc, bt_p, cu_p, ctx_p, ts, tq, out[:Tp], H, G, dk,
+                                      m.scale, sink=lw.sink, gate=proj[:Tp, gate_col:] if m.gate else None,
+                                      window=m.window, gate_per_head=m.gate_per_head, softcap=m.softcap)
+        elif nt:
+            ops.attn_sink_prefill(q[:Tp], gate_col, kc, vc, bt_p, cu_p, ctx_p, ts, tq, lw.sink, out[:Tp],
+                                  H, G, dk, dv, m.scale, tile_rows=self.prefill_tile, window=m.window,
+                                  gate_per_head=m.gate_per_head, head_scale=lw.head_scale, softcap=m.softcap)
+        if Bd and self.fast_decode[li]:
+            splits, ws = self._decode_plan(Bd, m)
+            ops.paged_attn_decode(q[Tp:T], q.stride(0), kc, vc, bt_d, lens_d, out[Tp:T], H, G, dk, m.scale,
+                                  num_splits=splits, workspace=ws, sink=lw.sink,
+                                  gate=proj[Tp:T, gate_col:] if m.gate else None, window=m.window,
+                                  gate_per_head=m.gate_per_head, softcap=m.softcap)
+        elif Bd:
+            ops.attn_sink_decode(q[Tp:T], gate_col, kc, vc, bt_d, lens_d, lw.sink, out[Tp:T], H, G, dk, dv,
+                                 m.scale, window=m.window, gate_per_head=m.gate_per_head, head_scale=lw.head_scale,
+                                 softcap=m.softcap)
+        self.stats["kernel_launches"] += (1 if nt else 0) + (1 if Bd else 0)
+
+    def _delta(self, l, m, lw, proj, out, T, Tp, Bd, nt, bt_p, cu_p, ctx_p, ts, tq, lens_d, bt_d, cu_all, ctx_all, slots_all) -> None:
+        """Gated delta rule: [q | k | v | gate] rows; the step and decay projections b | a in fp32."""
+        H, G, dk, dv = m.heads, m.kv_heads, m.dim, m.vdim
+        gates = self._view(self.gates, T, 2 * H)
+        ops.linear(self.xb[:T], lw.gates, gates)
+        S, ring = self.state[l]
+        x32, o_raw = self._view(self.lin32, T, m.row_width), self._view(self.o_raw, T, m.out_width)
+        ops.conv_rec_prep(proj, lw.rec_conv_t, None, ring, cu_all, ctx_all, slots_all, ts, tq, self.prefill_tile,
+                          cu_p.shape[0] - 1 if nt else 0, Bd, ((G, dk, dk ** -0.5), (G, dk, 1.0), (H, dv, None)), x32)
+        kc = G * S.shape[3]
+        ops.gated_scan(x32, 0, kc, 2 * kc, gates, lw.decay_rate, lw.dt_bias, None, cu_all, ctx_all, slots_all, S, o_raw, H, G, dk, dv,
+                       True, max_len=Tp if Tp else 1)
+        ops.linattn_out(o_raw, proj, m.conv_width, lw.out_norm, out, H, dv, self.mcfg.norm_eps, False, "silu")
+        ops.linear(out, lw.o, self.y[:T])
+        self._pending = {"y": self.y[:T]}
+        self.stats["kernel_launches"] += 6
+
+    def _attention_beside_scan(self, l, m, lw, proj, out, T, Tp, Bd, nt, bt_p, cu_p, ctx_p, ts, tq, lens_d, bt_d, cu_all, ctx_all,
+                               slots_all) -> None:
+        """Attention over convolved q, k, v beside a state-space recurrence, [q | k | v | z | x | B | C] rows and the dt
+        projection in fp32.  Each side has its own output projection (fp32); the join that follows norms and adds them."""
+        a, r = m.left, m.right
+        S, ring, a_ring = self.state[l]
+        wk, wv = self.k_cache[l].shape[3], self.v_cache[l].shape[3]
+        n = T * a.heads * wv
+        left = self.mix_out[:n].view(T, a.heads * wv)
+        right = self.mix_out[n:n + T * r.out_width].view(T, r.out_width)
+        q = self._view(self.q_rows, T, a.heads * wk)
+        self._conv_attention_rows(l, a, lw, proj, q, a_ring, Bd, nt, cu_p, ts, tq, cu_all, ctx_all, slots_all)
+        self._attend(l, a, lw, q, proj, -1, left, T, Tp, Bd, nt, bt_p, cu_p, ctx_p, ts, tq, lens_d, bt_d, wk, wv)
+        ops.linear(left, self.o_padded.get(self.runs[l][0], lw.o), self.y[:T])
+        gates = self._view(self.gates, T, r.heads)
+        ops.linear(self.xb[:T], lw.gates, gates)
+        x32, o_raw = self._view(self.lin32, T, r.row_width), self._view(self.o_raw, T, r.out_width)
+        z_col = a.qkv_width
+        ops.conv_rec_prep(proj[:, z_col + r.out_width:], lw.rec_conv_t, lw.rec_conv_bias, ring, cu_all, ctx_all, slots_all, ts, tq,
+                          self.prefill_tile, cu_p.shape[0] - 1 if nt else 0, Bd,
+                          ((r.heads, r.vdim, None), (r.groups, r.state, None), (r.groups, r.state, None)), x32)
+        b_col = r.row_width - 2 * r.groups * S.shape[3]
+        ops.gated_scan(x32, b_col + r.groups * S.shape[3], b_col, 0, gates, lw.decay_rate, lw.dt_bias, lw.skip, cu_all, ctx_all,
+                       slots_all, S, o_raw, r.heads, r.groups, r.state, r.vdim, False, max_len=Tp if Tp else 1)
+        ops.gate_norm(o_raw, proj, z_col, lw.out_norm, right, r.norm_groups, self.mcfg.norm_eps)
+        ops.linear(right, lw.o2, self.y2[:T])
+        self._pending = {"pair": (self.y[:T], self.y2[:T], lw.left_norm, lw.right_norm, m.left_scale, m.right_scale)}
+        self.stats["kernel_launches"] += 8
 
     def _side_by_side(self, l, m, lw, proj, out, T, Tp, Bd, nt, bt_p, cu_p, ctx_p, ts, tq, lens_d, bt_d, cu_all, ctx_all,
                       slots_all) -> None:
@@ -638,17 +766,20 @@ class LayerListRunner(ModelRunner):
 
     def _routed_rows(self, T: int, e, lw) -> tuple:
         """Routed feed-forward of self.xb[:T] up to, but without, the sum over a token's rows: (expert rows, row of each
-        (token, choice), choices, shared expert's rows, its gate's logits), the `routed` argument of output_norm_join."""
+        (token, choice), choices, shared expert's rows, its gate's logits), the `routed` argument of the join that follows."""
         x, ws = self.xb[:T], self.routed_ws
         shared = gate = None
         if e.shared_ff:
             act, shared = self._view(self.act, T, e.shared_ff), ws.shared[:T]
-            ops.linear(x, lw.shared13, act, relu2=True)
+            if e.gated:
+                ops.gated_linear(x, lw.shared13, act, e.act, e.shared_limit)
+            else:
+                ops.linear(x, lw.shared13, act, relu2=True)
             ops.linear(act, lw.shared2, shared)
             gate = ws.logits[:T, e.experts] if e.shared_gate else None     # the router product's row behind the outputs
             self.stats["kernel_launches"] += 2
         ops.routed_experts(x, lw.router, lw.correction, lw.w13, lw.w2, ws, None, e.experts, 0, e.top, e.scale, e.ff, e.limit,
-                           renormalize=e.renormalize, act=e.act, score=e.score, combine=False)
+                           renormalize=e.renormalize, act=e.act, score=e.score, combine=False, groups=e.groups, groups_keep=e.groups_keep)
         self.stats["kernel_launches"] += ops.ROUTED_LAUNCHES - 1
         return ws.yp, ws.pair_row, e.top, shared, gate
 
@@ -706,6 +837,9 @@ class LayerListRunner(ModelRunner):
             y, y2, ya, yb, post_w = self._pending if self._pending is not None else (None, None, 1.0, 1.0, None)
             ops.sandwich_join(self.resid32, cfg.norm_eps, y=y, y2=y2, ya=ya, yb=yb, post_w=post_w, mult=cfg.residual_mult,
                               pre_w=self.w.final_norm, rows=rows, h_out=self.x_last[:n])
+        elif self.pre_norm:      # the last sublayer's output enters the sum here, for the wanted rows only
+            ops.prenorm_join(self.resid32, self.w.final_norm, cfg.norm_eps, rows=rows, h_out=self.x_last[:n],
+                             out_scale=cfg.logit_scale, **self._pending)
         elif self.output_norm:   # likewise: the last output's norm, the sum and the final norm in one pass
             ops.output_norm_join(self.resid32, cfg.norm_eps, rows=rows, final=(self.w.final_norm, self.w.final_norm_b),
                                  h_out=self.x_last[:n], **(self._pending or {}))

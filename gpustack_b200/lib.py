@@ -177,6 +177,16 @@ SIGNATURES = {
     "b200_embed_sinusoid": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _f32, _vp]),
     "b200_conv_attn_prep": (_i32, [_vp, _i32, _i64, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _vp,
                                    _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _vp]),
+    "b200_conv_attn_prep_ex": (_i32, [_vp, _i32, _i64, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _vp,
+                                      _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _i32, _i32, _i32, _vp, _vp]),
+    "b200_conv_rec_prep": (_i32, [_vp, _i32, _i64, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _vp, _vp, _vp,
+                                  _vp, _vp, _i64, _f32, _vp]),
+    "b200_gated_scan": (_i32, [_vp, _i64, _i32, _i32, _i32, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32,
+                               _i32, _i32, _i32, _vp]),
+    "b200_gate_norm": (_i32, [_vp, _vp, _i32, _i64, _i32, _vp, _vp, _i64, _i32, _i32, _i32, _f32, _vp]),
+    "b200_prenorm_join": (_i32, [_vp, _vp, _vp, _vp, _vp, _f32, _f32, _vp, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _f32,
+                                 _f32, _vp]),
+    "b200_moe_route_grouped": (_i32, [_vp, _i64, _vp, _vp, _vp, _i32, _i32, _i32, _f32, _i32, _i32, _i32, _i32, _vp]),
     "b200_sample_softcap_f32": (_i32, [_vp, _i64, _f32, _vp, _vp, _i32, _vp, _vp, _i32, _i32, _vp]),
     "b200_gla_scan_rows": (_i32, [_vp, _i64, _i32, _i32, _i32, _vp, _i64, _f32, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32,
                              _i32, _vp]),

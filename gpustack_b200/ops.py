@@ -832,12 +832,18 @@ def output_norm_join(x_in, eps: float, y=None, routed=None, post=None, final=Non
 
 
 def conv_attn_prep(proj, conv_w, q_norm, k_norm, ring, cu_seq, ctx_lens, state_slots, tile_seq, tile_q0, tile_rows: int,
-                   n_prompt: int, n_single: int, slots, q_out, k_cache, v_cache, H, G, dk, dv, eps: float):
+                   n_prompt: int, n_single: int, slots, q_out, k_cache, v_cache, H, G, dk, dv, eps: float, joint_norm: bool = False,
+                   rot_dims: int = 0, half_layout: bool = False, freq=None):
     """Short causal convolution of the projected rows [q | k | v] with per-sequence rings of earlier inputs, per-head norms,
     queries to q_out [T, H * wk], keys and values to their pages (csrc/conv_attn_prep.cu).  conv_w fp32 [taps, C] (last row:
     the current token); ring fp32 [slots, taps - 1, C] (None with one tap); the sequences are n_prompt prompt portions (covered by the row
-    tiles) and then n_single single rows; page widths wk >= dk and wv >= dv come from the caches."""
-    _cuda(proj, conv_w, q_norm, k_norm, ring, cu_seq, ctx_lens, state_slots, tile_seq, tile_q0, slots, q_out, k_cache, v_cache)
+    tiles) and then n_single single rows; page widths wk >= dk and wv >= dv come from the caches.  joint_norm: q and k are
+    normed over the whole projection (weights of that size); rot_dims > 0: rotation of every q / k head after the norm."""
+    _cuda(proj, conv_w, q_norm, k_norm, ring, cu_seq, ctx_lens, state_slots, tile_seq, tile_q0, slots, q_out, k_cache, v_cache, freq)
+    if freq is not None:
+        _req(freq, torch.float64, "freq")
+    if joint_norm and (q_norm.numel() != H * dk or k_norm.numel() != G * dk):
+        raise B200Error("conv_attn_prep: the joint norm has one weight per channel of the projection")
     _req(conv_w, torch.float32, "conv_w")
     taps, C_ = conv_w.shape
     wk, wv = k_cache.shape[3], v_cache.shape[3]
@@ -850,10 +856,81 @@ def conv_attn_prep(proj, conv_w, q_norm, k_norm, ring, cu_seq, ctx_lens, state_s
         if tuple(ring.shape[1:]) != (taps - 1, C_):
             raise B200Error("conv_attn_prep: a ring of [slots, taps - 1, channels]")
     n_tiles = 0 if tile_seq is None else tile_seq.shape[0]
-    check(load().b200_conv_attn_prep(_p(proj), _is_f32(proj), proj.stride(0), _p(conv_w), taps, _p(q_norm), _p(k_norm), _p(ring),
-                                     _p(cu_seq), _p(ctx_lens), _p(state_slots), _p(tile_seq), _p(tile_q0), n_tiles, tile_rows,
-                                     n_prompt, n_single, _p(slots), _p(q_out), _p(k_cache), _p(v_cache), H, G, dk, dv, wk, wv,
-                                     k_cache.shape[2], eps, _stream()), "conv_attn_prep")
+    check(load().b200_conv_attn_prep_ex(_p(proj), _is_f32(proj), proj.stride(0), _p(conv_w), taps, _p(q_norm), _p(k_norm), _p(ring),
+                                        _p(cu_seq), _p(ctx_lens), _p(state_slots), _p(tile_seq), _p(tile_q0), n_tiles, tile_rows,
+                                        n_prompt, n_single, _p(slots), _p(q_out), _p(k_cache), _p(v_cache), H, G, dk, dv, wk, wv,
+                                        k_cache.shape[2], eps, 1 if joint_norm else 0, rot_dims, 1 if half_layout else 0, _p(freq),
+                                        _stream()), "conv_attn_prep")
+
+
+# ------------------------------------------- recurrences with one decay per head and token, pre-norm joins
+def conv_rec_prep(proj, conv_w, bias, ring, cu_seq, ctx_lens, state_slots, tile_seq, tile_q0, tile_rows: int, n_prompt: int,
+                  n_single: int, segments, out, eps: float = 1e-6):
+    """Short causal convolution (+ bias), silu and an optional unit norm per head of a recurrence's inputs, to fp32 rows
+    (csrc/conv_rec_prep.cu).  proj: the convolved channels (a column slice of wider rows is fine); segments: up to three
+    (heads, width, None or the factor of the unit norm) in channel order; out fp32, every head padded to a multiple of 4."""
+    _cuda(proj, conv_w, bias, ring, cu_seq, ctx_lens, state_slots, tile_seq, tile_q0, out)
+    _req(conv_w, torch.float32, "conv_w")
+    taps, C_ = conv_w.shape
+    if sum(h * w for h, w, _ in segments) != C_ or proj.stride(1) != 1 or proj.shape[1] < C_ or out.stride(1) != 1:
+        raise B200Error("conv_rec_prep: segments that cover the convolved channels")
+    if out.dtype != torch.float32 or out.shape[1] < sum(h * (-(-w // 4) * 4) for h, w, _ in segments):
+        raise B200Error("conv_rec_prep: fp32 rows of padded heads expected")
+    if taps > 1 and (ring is None or ring.dtype != torch.float32 or tuple(ring.shape[1:]) != (taps - 1, C_)):
+        raise B200Error("conv_rec_prep: an fp32 ring of [slots, taps - 1, channels]")
+    segs = list(segments) + [(0, 1, None)] * (3 - len(segments))
+    ints = [(C.c_int32 * 3)(*v) for v in zip(*[(h, w, 0 if u is None else 1) for h, w, u in segs])]
+    mul = (C.c_float * 3)(*[1.0 if u is None else u for _, _, u in segs])
+    check(load().b200_conv_rec_prep(_p(proj), _is_f32(proj), proj.stride(0), _p(conv_w), taps, _p(bias), _p(ring), _p(cu_seq),
+                                    _p(ctx_lens), _p(state_slots), _p(tile_seq), _p(tile_q0), 0 if tile_seq is None else tile_seq.shape[0],
+                                    tile_rows, n_prompt, n_single, ints[0], ints[1], ints[2], mul, _p(out), out.stride(0), eps,
+                                    _stream()), "conv_rec_prep")
+
+
+def gated_scan(x, q_col: int, k_col: int, v_col: int, gates, rate, dt_bias, skip, cu_seq, ctx_lens, state_slots, S, o_raw, H, G, dk,
+               dv, delta: bool, max_len: int = 1):
+    """Delta rule (delta) or state-space recurrence over every sequence's new rows of the fp32 rows x (csrc/gated_scan.cu);
+    state S [slots, H, dv, dk rounded up to 4] in, state out.  max_len: an upper bound of the new rows per sequence."""
+    _cuda(x, gates, rate, dt_bias, skip, cu_seq, ctx_lens, state_slots, S, o_raw)
+    for t_, n_ in ((x, "x"), (gates, "gates"), (rate, "rate"), (dt_bias, "dt_bias"), (S, "S"), (o_raw, "o_raw")):
+        if t_.dtype != torch.float32:
+            raise B200Error(f"gated_scan: {n_} is fp32")
+    if tuple(S.shape[1:]) != (H, dv, -(-dk // 4) * 4) or not S.is_contiguous() or not o_raw.is_contiguous():
+        raise B200Error("gated_scan: a contiguous state of [slots, heads, dv, dk rounded up to 4]")
+    check(load().b200_gated_scan(_p(x), x.stride(0), q_col, k_col, v_col, _p(gates), gates.stride(0), _p(rate), _p(dt_bias), _p(skip),
+                                 _p(cu_seq), _p(ctx_lens), _p(state_slots), _p(S), _p(o_raw), state_slots.shape[0], H, G, dk, dv,
+                                 1 if delta else 0, int(max_len), _stream()), "gated_scan")
+
+
+def gate_norm(y, proj, z_col: int, norm_w, out, parts: int, eps: float):
+    """out = RMS norm over `parts` equal pieces of (y * silu(z)) * w; z: columns z_col .. of proj; y fp32 contiguous rows."""
+    _cuda(y, proj, norm_w, out)
+    _req(y, torch.float32, "y")
+    check(load().b200_gate_norm(_p(y), _p(proj), _is_f32(proj), proj.stride(0), z_col, _p(norm_w), _p(out), out.stride(0), y.shape[0],
+                                y.shape[1], parts, eps, _stream()), "gate_norm")
+
+
+def prenorm_join(x_in, w, eps: float, y=None, pair=None, routed=None, x_out=None, h_out=None, rows=None, out_scale: float = 1.0):
+    """z = x_in + c; x_out = z; h_out = RMS norm(z) * w * out_scale (bf16 or fp32).  c: y (fp32 rows); pair = (y, y2, weight,
+    weight2, factor, factor2): two outputs, each normed over the row first; routed = (expert rows, row of each (token,
+    choice), choices, shared expert's rows or None): a routed feed-forward's sum.  rows: gather, h_out only."""
+    py = y2 = wy = wy2 = yp = pr = sh = None
+    ya = yb = 1.0
+    K = 0
+    if pair is not None:
+        py, y2, wy, wy2, ya, yb = pair
+    elif routed is not None:
+        yp, pr, K, sh = routed
+    else:
+        py = y
+    _cuda(x_in, w, py, y2, wy, wy2, yp, pr, sh, x_out, h_out, rows)
+    for t_, n_ in ((x_in, "x_in"), (py, "y"), (y2, "y2"), (yp, "yp"), (sh, "shared"), (x_out, "x_out")):
+        if t_ is not None:
+            _req(t_, torch.float32, n_)
+    T = rows.shape[0] if rows is not None else (h_out if h_out is not None else x_out).shape[0]
+    check(load().b200_prenorm_join(_p(x_in), _p(py), _p(y2), _p(wy), _p(wy2), ya, yb, _p(yp), _p(pr), K, _p(sh), _p(rows), _p(w), _p(x_out),
+                                   _p(h_out), 0 if h_out is None else _is_f32(h_out), T, x_in.shape[1], eps, out_scale, _stream()),
+          "prenorm_join")
 
 
 # ------------------------------------------- residual streams, latent attention, gated / routed feed-forward
@@ -1002,6 +1079,8 @@ def gated_linear(x, w_interleaved, out, act: str, limit: float = 0.0):
     of 64: the tcgen05 GEMM with the activation in its epilogue; otherwise the CUDA-core kernel."""
     M, K = x.shape
     N = w_interleaved.shape[0] // 2
+    if act == "silu" and out.dtype == torch.bfloat16 and N % 8 == 0 and _tc_gemm_ok(x, w_interleaved, out, K):
+        return gemm_silu_mul(x, w_interleaved, out=out)
     if out.dtype == torch.bfloat16 and act in TC_GATED_ACTS and _tc_gemm_ok(x, w_interleaved, out, K):
         timed = TIMER is not None and not torch.cuda.is_current_stream_capturing()
         if timed:
@@ -1051,7 +1130,8 @@ TC_GROUPED_ACTS = {"silu": 0, "gelu_tanh": 1, "clamped_swish": 2}
 
 def routed_experts(x, router, correction, w13, w2, ws: RoutedWorkspace, out, n_real: int, n_identity: int, top_k: int,
                    scale: float, ff: int, limit: float, shared=None, sigmoid: bool = False, renormalize: bool = True,
-                   weight_on: str = "output", act: str = "clamped_swish", score: Optional[str] = None, combine: bool = True):
+                   weight_on: str = "output", act: str = "clamped_swish", score: Optional[str] = None, combine: bool = True,
+                   groups: int = 0, groups_keep: int = 0):
     """out[t] (fp32) = sum over the top_k chosen router outputs of weight * expert(x[t]) (identity experts return
     x[t]) + shared[t].  router [n_real + n_identity, D]; w13 [n_real * 2 ff, D] interleaved; w2 [n_real * D, ff];
     shared: the shared expert's output rows (fp32) or None.  Six launches, no host synchronisation.
@@ -1060,7 +1140,8 @@ def routed_experts(x, router, correction, w13, w2, ws: RoutedWorkspace, out, n_r
     the activation (CUDA cores) and the output rows are not scaled; act: the experts' gate activation, or "relu2": experts
     without a gate, w13 [n_real * ff, D] as stored.  score "chosen_softmax": the largest logits + correction are chosen and
     weighted by the softmax over the chosen.  combine False: the weighted expert rows stay in ws.yp (ws.pair_row names
-    them) for output_norm_join, `out` is not written."""
+    them) for the join that follows, `out` is not written.  groups: only the groups_keep best of this many groups of
+    neighbouring outputs can be chosen from."""
     T, D = x.shape
     E = n_real + n_identity
     n_pairs = T * top_k
@@ -1081,9 +1162,9 @@ def routed_experts(x, router, correction, w13, w2, ws: RoutedWorkspace, out, n_r
     w_in = weight_on == "input"
     if w_in and n_identity:
         raise B200Error("routed_experts: identity experts with input weights are not defined")
-    check(L.b200_moe_route_scored(_p(lg), lg.stride(0), _p(correction), _p(ws.topk_ids), _p(ws.topk_w), T, E, top_k, scale,
-                                  SCORE_MODES[score] if score else (1 if sigmoid else 0), 1 if renormalize else 0, st),
-          "moe_route_scored")
+    check(L.b200_moe_route_grouped(_p(lg), lg.stride(0), _p(correction), _p(ws.topk_ids), _p(ws.topk_w), T, E, top_k, scale,
+                                   SCORE_MODES[score] if score else (1 if sigmoid else 0), 1 if renormalize else 0, groups,
+                                   groups_keep, st), "moe_route_grouped")
     check(L.b200_moe_align(_p(ws.topk_ids), _p(ws.topk_w), n_pairs, E, bx, cap, _p(ws.pair_row), _p(ws.row_pair),
                            _p(ws.row_weight), _p(ws.tile_expert), _p(ws.num_tiles), st), "moe_align")
     act = ws.act[:cap * ff].view(cap, ff)

@@ -60,6 +60,15 @@ def _layer_list_workspace(m, e: EngineConfig) -> int:
             if x.conv_taps:
                 wk, wv = x.cache_widths(a == 2)
                 lat, mix = max(lat, x.heads * wk), max(mix, x.heads * wv)      # prepared query rows, padded head outputs
+        elif x.kind == "side_by_side" and x.right.kind == "state_space":
+            y, r = x.left, x.right
+            wk, wv = y.cache_widths(a == 2)
+            proj = max(proj, y.qkv_width + r.proj_rows + 7)
+            lat, mix = max(lat, y.heads * wk), max(mix, y.heads * wv + r.out_width)
+            gates, rec, lin = max(gates, r.heads, y.heads), max(rec, r.out_width), max(lin, r.row_width)
+        elif x.kind == "delta":
+            proj = max(proj, x.proj_rows + 7)
+            gates, rec, lin = max(gates, 2 * x.heads), max(rec, x.out_width), max(lin, x.row_width)
         elif x.kind == "side_by_side":
             y, r = x.left, x.right
             proj = max(proj, y.q_width + y.kv_heads * (y.dim + y.vdim) + r.proj_rows + 7)
@@ -86,6 +95,8 @@ def _layer_list_workspace(m, e: EngineConfig) -> int:
             ff = max(ff, l.mlp.ff)
     S_smp = min(T, max(S, e.max_logit_rows or 0))
     par = 4 * (1 + (1 if m.loop_times > 1 else 0)) if m.residual == "parallel" else 0    # second branch output, embedding copy
+    if m.residual == "pre_norm":
+        par = 4                                                                          # second output
     if m.residual == "sandwich":
         par = 8                                                                          # second output, normed input (fp32)
         routed += 8 * (T // 64 + S + 1) * max([x.mixer.right.width for x in m.layers if x.mixer.kind == "side_by_side"] or [0])

@@ -559,6 +559,46 @@ int b200_conv_attn_prep(const void* proj, int f32, int64_t ld, const float* conv
                         const int32_t* state_slots, const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles,
                         int tile_rows, int n_prompt, int n_single, const int32_t* slots, void* q_out, void* k_cache,
                         void* v_cache, int H, int G, int dk, int dv, int wk, int wv, int page, float eps, void* stream);
+/* The same with a q / k norm over the whole projection (joint_norm: weights of H dk / G dk entries) and a rotation of the
+ * first rot_dims entries of every q / k head by position * freq[i] after the norm (half_layout: pairs (i, i + rot_dims/2),
+ * else (2i, 2i + 1)). */
+int b200_conv_attn_prep_ex(const void* proj, int f32, int64_t ld, const float* conv_w, int taps, const void* qnorm_w,
+                           const void* knorm_w, float* ring, const int32_t* cu_seq, const int32_t* ctx_lens,
+                           const int32_t* state_slots, const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles,
+                           int tile_rows, int n_prompt, int n_single, const int32_t* slots, void* q_out, void* k_cache,
+                           void* v_cache, int H, int G, int dk, int dv, int wk, int wv, int page, float eps, int joint_norm,
+                           int rot_dims, int half_layout, const double* freq, void* stream);
+/* Short causal convolution (+ bias), silu and an optional unit norm x / sqrt(sum(x^2) + eps) * factor per head of the
+ * inputs of a recurrence: three segments of equal heads in neighbouring columns of proj, fp32 rows out with every head padded
+ * by zeros to a multiple of 4 entries.  Rings, row tiles and single rows as above; seg_* are host arrays of three entries. */
+int b200_conv_rec_prep(const void* proj, int f32, int64_t ld, const float* conv_w, int taps, const float* bias, float* ring,
+                       const int32_t* cu_seq, const int32_t* ctx_lens, const int32_t* state_slots, const int32_t* tile_seq,
+                       const int32_t* tile_q0, int n_tiles, int tile_rows, int n_prompt, int n_single,
+                       const int32_t* seg_heads, const int32_t* seg_width, const int32_t* seg_unit, const float* seg_mul,
+                       float* out, int64_t ldo, float eps, void* stream);
+/* Recurrence with one decay per head and token over every sequence's new rows of fp32 rows (heads padded to a multiple of
+ * 4), state S [slots][H][dv][dk rounded up to 4].  delta: gates [b: H | a: H], S <- g S, u = sigmoid(b) (v - S^T k),
+ * S += k u^T, o = S^T q with g = exp(-rate softplus(a + dt_bias)); otherwise gates [a: H], S = g S + d k v^T,
+ * o = S^T q + skip v with d = softplus(a + dt_bias).  max_len: the most new rows of a sequence. */
+int b200_gated_scan(const float* x, int64_t ld, int q_col, int k_col, int v_col, const float* gates, int64_t ld_g,
+                    const float* rate, const float* dt_bias, const float* skip, const int32_t* cu_seq, const int32_t* ctx_lens,
+                    const int32_t* state_slots, float* S, float* o_raw, int n_seqs, int H, int G, int dk, int dv, int delta,
+                    int max_len, void* stream);
+/* out = RMSnorm over `parts` equal pieces of (y * silu(z)) * w (the gate comes before the norm). */
+int b200_gate_norm(const float* y, const void* proj, int f32, int64_t ld, int z_col, const void* w, void* out, int64_t ldo,
+                   int T, int C, int parts, float eps, void* stream);
+/* z = x_in + c; x_out = z; h_out = z / rms(z) * w * out_scale.  c: y (NULL: nothing); or with y2 the normed pair
+ * ya * y / rms(y) * wy + yb * y2 / rms(y2) * wy2; or with yp a routed feed-forward, sum_j yp[pair_row[t top_k + j]] (+ shared[t]).
+ * rows != NULL: gather, h_out only. */
+int b200_prenorm_join(const float* x_in, const float* y, const float* y2, const void* wy, const void* wy2, float ya, float yb,
+                      const float* yp, const int32_t* pair_row, int top_k, const float* shared, const int32_t* rows,
+                      const void* w, float* x_out, void* h_out, int h_f32, int T, int D, float eps, float out_scale,
+                      void* stream);
+/* b200_moe_route_scored with the outputs in `groups` equal groups of neighbours of which only the groups_keep best (by
+ * their largest choice score) can be chosen from (0: no groups). */
+int b200_moe_route_grouped(const float* logits, int64_t ld, const float* correction, int32_t* topk_ids, float* topk_w, int T,
+                           int E, int K, float scale, int score_mode, int renormalize, int groups, int groups_keep,
+                           void* stream);
 /* The attention kernels with a soft cap on the scaled score, softcap * tanh(score / softcap) (0 = none). */
 int b200_attn_sink_prefill_cap(const void* proj, int f32, int64_t ld, int gate_col, const void* k_cache, const void* v_cache,
                                 const int32_t* block_table, int max_blocks, const int32_t* cu_q, const int32_t* ctx_lens,
