@@ -121,12 +121,11 @@ def ssd_scan(x: torch.Tensor, B: torch.Tensor, C: torch.Tensor, dt: torch.Tensor
     T, H, P = x.shape
     G, N = B.shape[1], B.shape[2]
     y = torch.zeros_like(x)
-    for h in range(H):
-        g = h // (H // G)
-        S = torch.zeros(N, P, dtype=x.dtype)
-        for t in range(T):
-            S = torch.exp(-torch.exp(A_log[h]) * dt[t, h]) * S + dt[t, h] * torch.outer(B[t, g], x[t, h])
-            y[t, h] = S.T @ C[t, g] + D[h] * x[t, h]
+    S = torch.zeros(H, N, P, dtype=x.dtype)
+    of = torch.arange(H) // (H // G)                     # the group a head reads
+    for t in range(T):
+        S = torch.exp(-torch.exp(A_log) * dt[t])[:, None, None] * S + dt[t][:, None, None] * (B[t, of][:, :, None] * x[t][:, None, :])
+        y[t] = torch.einsum("hnp,hn->hp", S, C[t, of]) + D[:, None] * x[t]
     return y
 
 
@@ -152,14 +151,14 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tenso
     T, H, dv = v.shape
     G, dk = k.shape[1], k.shape[2]
     o = torch.zeros_like(v)
-    for h in range(H):
-        j = h // (H // G)
-        S = torch.zeros(dk, dv, dtype=v.dtype)
-        for t in range(T):
-            S = g[t, h] * S
-            u = beta[t, h] * (v[t, h] - S.T @ k[t, j])
-            S = S + torch.outer(k[t, j], u)
-            o[t, h] = S.T @ q[t, j]
+    S = torch.zeros(H, dk, dv, dtype=v.dtype)
+    of = torch.arange(H) // (H // G)                     # the query / key head a value head reads
+    for t in range(T):
+        kt, qt = k[t, of], q[t, of]
+        S = g[t][:, None, None] * S
+        u = beta[t][:, None] * (v[t] - torch.einsum("hkv,hk->hv", S, kt))
+        S = S + kt[:, :, None] * u[:, None, :]
+        o[t] = torch.einsum("hkv,hk->hv", S, qt)
     return o
 
 
@@ -233,3 +232,78 @@ def forward(cfg: dict, weights: Dict[str, torch.Tensor], tokens: List[int], trac
         if trace is not None:
             trace.append(x.clone())
     return (rms(x, eps) * w["final.norm"]) @ w["head"].T * cfg["logit_scale"]
+
+
+# ------------------------------------------------------------------------------ random checkpoints
+def tensor_shapes(cfg: dict) -> Dict[str, tuple]:
+    W, V = cfg["width"], cfg["vocab"]
+    out: Dict[str, tuple] = {"embed": (V, W), "head": (V, W), "final.norm": (W,)}
+
+    def convolved(p, n, rows, taps):
+        out[p + n], out[p + n + ".conv"] = (rows, W), (rows, taps)
+
+    for l, layer in enumerate(cfg["layers"]):
+        if layer.get("weights_of") is not None:
+            continue
+        p, mx, mlp = f"l{l}.mix.", layer["mixer"], layer.get("mlp")
+        out[f"l{l}.norm1"] = (W,)
+        if layer["type"] == "delta":
+            H, G, dk, dv = mx["heads"], mx["kv_heads"], mx["dim"], mx["vdim"]
+            for n, rows in (("q", G * dk), ("k", G * dk), ("v", H * dv)):
+                convolved(p, n, rows, mx["conv"])
+            out[p + "a"] = out[p + "b"] = (H, W)
+            out[p + "A_log"] = out[p + "dt_bias"] = (H,)
+            out[p + "g"], out[p + "norm"], out[p + "o"] = (H * dv, W), (dv,), (W, H * dv)
+        else:
+            a, r = mx["left"], mx["right"]
+            for n, rows in (("q", a["heads"] * a["dim"]), ("k", a["kv_heads"] * a["dim"]), ("v", a["kv_heads"] * a["vdim"])):
+                convolved(p + "left.", n, rows, a["conv"])
+                if n != "v":
+                    out[p + f"left.{n}.norm"] = (rows,)
+            out[p + "left.o"] = (W, a["heads"] * a["vdim"])
+            inner, bc = r["heads"] * r["vdim"], 2 * r["groups"] * r["state"]
+            out[p + "right.in"] = (2 * inner + bc + r["heads"], W)
+            out[p + "right.conv"], out[p + "right.conv.b"] = (inner + bc, r["conv"]), (inner + bc,)
+            out[p + "right.A_log"] = out[p + "right.D"] = out[p + "right.dt_bias"] = (r["heads"],)
+            out[p + "right.norm"], out[p + "right.o"] = (inner,), (W, inner)
+            out[p + "left.out"] = out[p + "right.out"] = (W,)
+        if not mlp:
+            continue
+        q = f"l{l}.mlp."
+        out[f"l{l}.norm2"] = (W,)
+        E = mlp["router"]["experts"]
+        out[q + "router"], out[q + "correction"] = (E, W), (E,)
+        for e, ff in [(f"e{i}", mlp["expert"]["ff"]) for i in range(E)] + ([("shared", mlp["shared"]["ff"])] if mlp.get("shared") else []):
+            out[q + e + ".gate"] = out[q + e + ".up"] = (ff, W)
+            out[q + e + ".down"] = (W, ff)
+    return out
+
+
+def random_weights(cfg: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
+    """Seeded bf16 weights: linear weights N(0, 1 / in), norm weights around one, taps of half, decays between fast and slow,
+    router logits and corrections that decide most choices clearly."""
+    g = torch.Generator().manual_seed(seed)
+    out: Dict[str, torch.Tensor] = {}
+    for name, shape in tensor_shapes(cfg).items():
+        x = torch.randn(tuple(shape), generator=g)
+        leaf = name.split(".")[-1]
+        if leaf == "A_log":
+            x = x - 1.0
+        elif leaf == "dt_bias":
+            x = x - 2.0
+        elif leaf == "D":
+            x = 1.0 + 0.3 * x
+        elif leaf == "b" and name.endswith("conv.b"):
+            x = 0.3 * x
+        elif leaf == "correction":
+            x = 0.2 * x
+        elif leaf == "conv":
+            x = 0.5 * x
+        elif leaf in ("norm", "norm1", "norm2", "out"):
+            x = 1.0 + 0.2 * x
+        elif leaf == "router":
+            x = 3.0 * x / shape[-1] ** 0.5
+        elif name != "embed":
+            x = x / shape[-1] ** 0.5
+        out[name] = x.to(torch.bfloat16)
+    return out
