@@ -5,7 +5,8 @@
 //                                                    older than the step come from the sequence's ring
 //   q, k:  y / sqrt(mean(y^2) + eps) * weight        per head over dk, one weight vector for all heads (optional), or over
 //                                                    the whole projection (all heads at once) with weights of that size
-//   q, k:  rotation of the first `dims` entries by position * freq[i] (optional, after the norm)
+//   q, k:  rotation of the first `dims` entries by the rows' angles (optional, after the norm); cos and sin come from a table
+//          that rot_table fills once per step for all layers with the same frequencies
 //   q to its row of q_out, k and v to their pages (slot of the token), heads laid out wk / wv wide (>= dk / dv, the
 //   columns behind dk / dv are zeros: a pair of widths that is no tensor-core tile is padded to one);
 //   the step's last taps - 1 inputs of every sequence replace the ring's entries: ring[slot][p mod (taps - 1)][channel].
@@ -14,12 +15,16 @@
 // (8 rows and the taps - 1 before them) at once and walk the rows in registers.  Only a sequence's first
 // piece can need the ring (a piece is longer than the ring), and the SAME threads that read it there write the step's
 // last inputs into it after their reads: no second launch, no race.  The statistics and the convolution are fp32.
+#include <cooperative_groups.h>
+
 #include "common.cuh"
 #include "conv_prep.cuh"
 #include "runtime.h"
 #include "../../include/b200.h"
 
 namespace b200 {
+
+namespace cg = cooperative_groups;
 
 struct CapArgs {
   const void* proj;
@@ -44,7 +49,7 @@ struct CapArgs {
   float eps;
   int joint;                       // the norm runs over the whole projection (weights of H dk / G dk entries)
   int dims, half_layout;           // rotation of the first `dims` entries of a q / k head, pairs (i, i + dims/2) or (2i, 2i + 1)
-  const double* freq;              // [dims / 2] angular frequencies
+  const float2* cs;                // [rows][dims / 2] (cos, sin)
 };
 
 // the (page, head) row of a cache slot, in rows of the cache
@@ -219,158 +224,141 @@ conv_attn_prep_kernel(CapArgs a) {
   }
 }
 
-// cos / sin of the rows' angles, one table per CTA: the angle is formed and reduced to [-pi, pi] in fp64, sine and cosine
-// of the remainder in fp32
-__device__ __forceinline__ void cap_angles(const CapArgs& a, const CapWork& m, float2* cs) {
-  const int half = a.dims >> 1;
-  for (int i = threadIdx.x; i < m.n * half; i += blockDim.x) {
-    const int r = i / half, j = i - r * half;
-    const double ang = (double)(m.ctx + m.q0 + r) * a.freq[j];
-    float sn, c;
-    sincosf((float)(ang - 6.283185307179586 * rint(ang * 0.15915494309189535)), &sn, &c);
-    cs[i] = make_float2(c, sn);
-  }
+// (cos, sin) of position * freq[i] for every row of a step: the angle is formed and reduced to [-pi, pi] in fp64, sine and
+// cosine of the remainder in fp32
+__global__ void __launch_bounds__(256)
+rot_table_kernel(const int32_t* __restrict__ positions, const double* __restrict__ freq, float2* __restrict__ out, int half, int n) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const int r = i / half, j = i - r * half;
+  const double ang = (double)positions[r] * freq[j];
+  float sn, c;
+  sincosf((float)(ang - 6.283185307179586 * rint(ang * 0.15915494309189535)), &sn, &c);
+  out[i] = make_float2(c, sn);
 }
 
-// Sums of 2 NB values over the CTA (NB sums of q, NB of k), then the rows' factors: mul[0][r] for q, mul[1][r] for k
-template <int NB>
-__device__ __forceinline__ void cap_row_factors(const CapArgs& a, float (&ss)[2][NB], float (*red)[2][NB], float (*mul)[NB]) {
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = (blockDim.x + 31) >> 5;
-#pragma unroll
-  for (int p = 0; p < 2; ++p)
-#pragma unroll
-    for (int r = 0; r < NB; ++r) {
-      const float v = warp_sum(ss[p][r]);
-      if (lane == 0) red[warp][p][r] = v;
-    }
-  __syncthreads();
-  if (threadIdx.x < 2 * NB) {
-    const int p = threadIdx.x / NB, r = threadIdx.x % NB;
-    float v = 0.f;
-    for (int w = 0; w < nw; ++w) v += red[w][p][r];    // a fixed order
-    mul[p][r] = 1.0f / sqrtf(v / (float)((p == 0 ? a.H : a.G) * a.dk) + a.eps);
-  }
-  __syncthreads();
-}
+// The form with a rotation and / or a norm over the whole projection.  The head slots of a piece of rows are spread over the
+// CTAs of ONE cluster (along y); every thread keeps its window of inputs and weights in registers, convolves once for the sums
+// of squares, the CTAs exchange their partial sums through distributed shared memory (added in rank order), and a second
+// convolution from the same registers is scaled, rotated -- the partner of an entry sits dims / 2 further, in another lane
+// of the head's group, or beside it -- and stored.  No input is loaded twice.
+constexpr int kCapJointWarps = 6;    // per CTA: two CTAs per SM with the window and the weights in registers
 
-// The form with a rotation and / or a norm over the whole projection.  One CTA holds ALL head slots of NB rows (the joint
-// statistic is a sum over the CTA): one pass over the head slots for the sums of squares, one that convolves again (its
-// inputs are in L1), scales, rotates -- the partner of an entry sits dims / 2 further, in another lane of the head's
-// group, or beside it -- and stores.
-constexpr int kCapJointWarps = 16;
-
-template <typename TA, int TAPS, int NB>
-__global__ void __launch_bounds__(kCapJointWarps * 32)
+template <typename TA, int TAPS>
+__global__ void __launch_bounds__(kCapJointWarps * 32, 2)
 conv_attn_prep_joint_vec_kernel(CapArgs a, int lph) {
-  constexpr int V = 16 / (int)sizeof(TA), R = TAPS - 1;
+  constexpr int V = 16 / (int)sizeof(TA), R = TAPS - 1, NB = kCapRows;
   extern __shared__ __align__(16) float2 cs[];         // [NB][dims / 2]
-  __shared__ float red[kCapJointWarps][2][NB], mul[2][NB];
+  __shared__ float head_ss[kCapJointWarps * 32][NB], part[2][NB], mul[2][NB];
   const CapWork m = cap_work<NB>(a);
-  if (m.n <= 0) return;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, per_warp = 32 / lph, n_slots = a.H + 2 * a.G;
-  const int step = (blockDim.x >> 5) * per_warp, li = lane % lph, d = li * V, half = a.dims >> 1;
+  if (m.n <= 0) return;                                // (the same for every CTA of the cluster)
+  const int lane = threadIdx.x & 31, per_warp = 32 / lph, li = lane % lph, d = li * V, half = a.dims >> 1;
+  const int in_cta = (threadIdx.x >> 5) * per_warp + lane / lph, cta_heads = (blockDim.x >> 5) * per_warp;
+  const int hs = blockIdx.y * cta_heads + in_cta;
+  const bool live = hs < a.H + 2 * a.G, is_q = hs < a.H, is_k = !is_q && hs < a.H + a.G, qk = is_q || is_k;
+  const int width = qk ? a.dk : a.dv, wide = qk ? a.wk : a.wv;
   const int C = (a.H + a.G) * a.dk + a.G * a.dv;
-  const TA* rows = reinterpret_cast<const TA*>(a.proj) + (size_t)m.row0 * a.ld;
+  const int c = (qk ? hs * a.dk : (a.H + a.G) * a.dk + (hs - a.H - a.G) * a.dv) + d;
+  const bool act = live && d < width, pad = live && !act && d < wide;
   const bool norm = a.qnorm_w != nullptr;
-  if (a.joint && norm) {
-    float ss[2][NB];
-#pragma unroll
-    for (int r = 0; r < NB; ++r) ss[0][r] = ss[1][r] = 0.f;
-    for (int hs = warp * per_warp + lane / lph; hs < a.H + a.G; hs += step) {
-      if (d >= a.dk) continue;
-      const int c = hs * a.dk + d;
-      uint4 win[R + NB];
-      float w[TAPS][V];
-      conv_window<TA, TAPS, NB>(win, m, rows + c, a.ld, a.ring, c, C);
-      conv_weights<TAPS, V>(w, a.conv_w, c, C);
-#pragma unroll
-      for (int r = 0; r < NB; ++r) {
-        float y[V], s = 0.f;
-#pragma unroll
-        for (int i = 0; i < V; ++i) y[i] = 0.f;
-        conv_row<TA, TAPS, NB>(win, r, w, y);
-#pragma unroll
-        for (int i = 0; i < V; ++i) s = fmaf(y[i], y[i], s);
-        if (hs < a.H) ss[0][r] += s; else ss[1][r] += s;
-      }
-    }
-    cap_angles(a, m, cs);
-    cap_row_factors<NB>(a, ss, red, mul);
-  } else {
-    cap_angles(a, m, cs);
-    __syncthreads();
+  const TA* src = reinterpret_cast<const TA*>(a.proj) + (size_t)m.row0 * a.ld + c;
+  uint4 win[R + NB];
+  float w[TAPS][V];
+  if (act) {
+    conv_window<TA, TAPS, NB>(win, m, src, a.ld, a.ring, c, C);
+    conv_weights<TAPS, V>(w, a.conv_w, c, C);
+    conv_ring_put<TA, TAPS>(m, src, a.ld, a.ring, c, C);
   }
-  const int32_t* slots = a.slots + m.row0 + m.q0;
-  for (int hs0 = warp * per_warp; hs0 < n_slots; hs0 += step) {
-    const int hs = hs0 + lane / lph;
-    const bool is_q = hs < a.H, is_k = !is_q && hs < a.H + a.G, live = hs < n_slots, qk = is_q || is_k;
-    const int width = qk ? a.dk : a.dv, wide = qk ? a.wk : a.wv;
-    const int c = (qk ? hs * a.dk : (a.H + a.G) * a.dk + (hs - a.H - a.G) * a.dv) + d;
-    const bool act = live && d < width, pad = live && !act && d < wide;
-    uint4 win[R + NB];
-    float w[TAPS][V], nw[V];
-    if (act) {
-      conv_window<TA, TAPS, NB>(win, m, rows + c, a.ld, a.ring, c, C);
-      conv_weights<TAPS, V>(w, a.conv_w, c, C);
-      conv_ring_put<TA, TAPS>(m, rows + c, a.ld, a.ring, c, C);
-      const bf16* nv = is_q ? a.qnorm_w : a.knorm_w;
+  const float2* table = a.cs + (size_t)(m.row0 + m.q0) * half;
+  for (int i = threadIdx.x; i < m.n * half; i += blockDim.x) cs[i] = table[i];
+  auto row_ss = [&](int r) {                           // sum of squares of the head's convolved row, in all its lanes
+    float y[V], ss = 0.f;
 #pragma unroll
-      for (int i = 0; i < V; ++i)
-        nw[i] = norm && qk ? __bfloat162float(nv[(a.joint ? (is_q ? hs : hs - a.H) * a.dk : 0) + d + i]) : 1.0f;
-    }
-    const bool turn = act && qk && d < a.dims;          // (dims is a whole number of pieces)
-    const int partner = (turn && a.half_layout) ? (d < half ? lane + half / V : lane - half / V) : lane;
-    const int g = is_k ? hs - a.H : hs - a.H - a.G;
+    for (int i = 0; i < V; ++i) y[i] = 0.f;
+    if (act) conv_row<TA, TAPS, NB>(win, r, w, y);
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss = fmaf(y[i], y[i], ss);
+    for (int o = lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    return ss;
+  };
+  cg::cluster_group cluster = cg::this_cluster();
+  if (a.joint && norm) {
 #pragma unroll
     for (int r = 0; r < NB; ++r) {
-      if (r >= m.n) break;
-      float y[V], ss = 0.f;
-#pragma unroll
-      for (int i = 0; i < V; ++i) y[i] = 0.f;
-      if (act) conv_row<TA, TAPS, NB>(win, r, w, y);
-      if (norm && !a.joint) {
-#pragma unroll
-        for (int i = 0; i < V; ++i) ss = fmaf(y[i], y[i], ss);
-        for (int o = lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-      }
-      float f = 1.0f;
-      if (norm && qk) f = a.joint ? mul[is_q ? 0 : 1][r] : 1.0f / sqrtf(ss / (float)a.dk + a.eps);
-      if (act) {
-#pragma unroll
-        for (int i = 0; i < V; ++i) y[i] *= f * nw[i];
-      }
-      if (a.half_layout) {
-        float o[V];
-#pragma unroll
-        for (int i = 0; i < V; ++i) o[i] = __shfl_sync(0xffffffffu, y[i], partner);
-        if (turn) {
-          const float2* t = cs + r * half + (d < half ? d : d - half);
-#pragma unroll
-          for (int i = 0; i < V; ++i) y[i] = d < half ? y[i] * t[i].x - o[i] * t[i].y : y[i] * t[i].x + o[i] * t[i].y;
-        }
-      } else if (turn) {
-        const float2* t = cs + r * half + d / 2;
-#pragma unroll
-        for (int i = 0; i < V; i += 2) {
-          const float u = y[i], v = y[i + 1];
-          y[i] = u * t[i / 2].x - v * t[i / 2].y;
-          y[i + 1] = v * t[i / 2].x + u * t[i / 2].y;
-        }
-      }
-      if (!act && !pad) continue;
-      uint4 outv;
-      TA* ov = reinterpret_cast<TA*>(&outv);
-#pragma unroll
-      for (int i = 0; i < V; ++i) ca_store(ov + i, y[i]);       // (zeros behind the head's own columns)
-      if (is_q) {
-        *reinterpret_cast<uint4*>(reinterpret_cast<TA*>(a.q_out) + ((size_t)(m.row0 + m.q0 + r) * a.H + hs) * a.wk + d) = outv;
-      } else {
-        const int slot = slots[r];
-        if (slot >= 0)
-          *reinterpret_cast<uint4*>(reinterpret_cast<TA*>(is_k ? a.k_cache : a.v_cache) + cap_cache_row(a, slot, g) * wide + d) = outv;
-      }
+      const float ss = row_ss(r);                      // (rows behind the portion are zeros)
+      if (li == 0) head_ss[in_cta][r] = ss;
+    }
+    __syncthreads();
+    if (threadIdx.x < 2 * NB) {
+      const int p = threadIdx.x / NB, r = threadIdx.x % NB;
+      const int lo = p == 0 ? 0 : a.H, hi = p == 0 ? a.H : a.H + a.G, first = blockIdx.y * cta_heads;
+      float v = 0.f;
+      for (int h = max(lo, first); h < min(hi, first + cta_heads); ++h) v += head_ss[h - first][r];
+      part[p][r] = v;
+    }
+    cluster.sync();
+    if (threadIdx.x < 2 * NB) {
+      const int p = threadIdx.x / NB, r = threadIdx.x % NB;
+      float v = 0.f;
+      for (unsigned k = 0; k < gridDim.y; ++k) v += cluster.map_shared_rank(&part[0][0], k)[p * NB + r];
+      mul[p][r] = 1.0f / sqrtf(v / (float)((p == 0 ? a.H : a.G) * a.dk) + a.eps);
     }
   }
+  __syncthreads();
+  float nw[V];
+  const bf16* nv = is_q ? a.qnorm_w : a.knorm_w;
+#pragma unroll
+  for (int i = 0; i < V; ++i)
+    nw[i] = act && norm && qk ? __bfloat162float(nv[(a.joint ? (is_q ? hs : hs - a.H) * a.dk : 0) + d + i]) : 1.0f;
+  const bool turn = act && qk && d < a.dims;            // (dims is a whole number of pieces)
+  const int partner = (turn && a.half_layout) ? (d < half ? lane + half / V : lane - half / V) : lane;
+  const int g = is_k ? hs - a.H : hs - a.H - a.G;
+  const int32_t* slots = a.slots + m.row0 + m.q0;
+#pragma unroll
+  for (int r = 0; r < NB; ++r) {
+    if (r >= m.n) break;
+    float f = 1.0f;
+    if (norm && !a.joint) f = 1.0f / sqrtf(row_ss(r) / (float)a.dk + a.eps);      // (all lanes take part)
+    if (a.joint && qk) f = mul[is_q ? 0 : 1][r];
+    if (!qk) f = 1.0f;
+    float y[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) y[i] = 0.f;
+    if (act) conv_row<TA, TAPS, NB>(win, r, w, y);
+#pragma unroll
+    for (int i = 0; i < V; ++i) y[i] *= f * nw[i];
+    if (a.half_layout) {
+      float o[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) o[i] = __shfl_sync(0xffffffffu, y[i], partner);
+      if (turn) {
+        const float2* t = cs + r * half + (d < half ? d : d - half);
+#pragma unroll
+        for (int i = 0; i < V; ++i) y[i] = d < half ? y[i] * t[i].x - o[i] * t[i].y : y[i] * t[i].x + o[i] * t[i].y;
+      }
+    } else if (turn) {
+      const float2* t = cs + r * half + d / 2;
+#pragma unroll
+      for (int i = 0; i < V; i += 2) {
+        const float u = y[i], v = y[i + 1];
+        y[i] = u * t[i / 2].x - v * t[i / 2].y;
+        y[i + 1] = v * t[i / 2].x + u * t[i / 2].y;
+      }
+    }
+    if (!act && !pad) continue;
+    uint4 outv;
+    TA* ov = reinterpret_cast<TA*>(&outv);
+#pragma unroll
+    for (int i = 0; i < V; ++i) ca_store(ov + i, y[i]);         // (zeros behind the head's own columns)
+    if (is_q) {
+      *reinterpret_cast<uint4*>(reinterpret_cast<TA*>(a.q_out) + ((size_t)(m.row0 + m.q0 + r) * a.H + hs) * a.wk + d) = outv;
+    } else {
+      const int slot = slots[r];
+      if (slot >= 0)
+        *reinterpret_cast<uint4*>(reinterpret_cast<TA*>(is_k ? a.k_cache : a.v_cache) + cap_cache_row(a, slot, g) * wide + d) = outv;
+    }
+  }
+  if (a.joint && norm) cluster.sync();                  // nobody leaves while another CTA may still read its sums
 }
 
 // Any width, any number of taps: warps take the head slots in turn, lanes the columns; a head is staged in shared memory
@@ -379,13 +367,13 @@ template <typename TA>
 __global__ void __launch_bounds__(kCapWarps * 32)
 conv_attn_prep_joint_kernel(CapArgs a) {
   constexpr int NB = kCapRows;
-  extern __shared__ __align__(16) float2 cs[];         // [NB][dims / 2], then a head per warp
+  extern __shared__ __align__(16) float heads[];       // a head per warp
   __shared__ float red[kCapWarps][2][NB], mul[2][NB];
   const CapWork m = cap_work<NB>(a);
   if (m.n <= 0) return;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, half = a.dims >> 1, n_slots = a.H + 2 * a.G, R = a.taps - 1;
   const int C = (a.H + a.G) * a.dk + a.G * a.dv, wmax = a.dk > a.dv ? a.dk : a.dv;
-  float* head = reinterpret_cast<float*>(cs + NB * half) + warp * wmax;
+  float* head = heads + warp * wmax;
   const TA* rows = reinterpret_cast<const TA*>(a.proj) + (size_t)m.row0 * a.ld;
   const bool norm = a.qnorm_w != nullptr;
   if (a.joint && norm) {
@@ -400,10 +388,20 @@ conv_attn_prep_joint_kernel(CapArgs a) {
           const float y = conv_at<TA>(m, m.q0 + r, rows + hs * a.dk + d, a.ld, a.ring, a.conv_w, hs * a.dk + d, C, a.taps);
           if (hs < a.H) ss[0][r] = fmaf(y, y, ss[0][r]); else ss[1][r] = fmaf(y, y, ss[1][r]);
         }
-    cap_angles(a, m, cs);
-    cap_row_factors<NB>(a, ss, red, mul);
-  } else {
-    cap_angles(a, m, cs);
+#pragma unroll
+    for (int p = 0; p < 2; ++p)
+#pragma unroll
+      for (int r = 0; r < NB; ++r) {
+        const float v = warp_sum(ss[p][r]);
+        if (lane == 0) red[warp][p][r] = v;
+      }
+    __syncthreads();
+    if (threadIdx.x < 2 * NB) {
+      const int p = threadIdx.x / NB, r = threadIdx.x % NB;
+      float v = 0.f;
+      for (int w = 0; w < kCapWarps; ++w) v += red[w][p][r];     // a fixed order
+      mul[p][r] = 1.0f / sqrtf(v / (float)((p == 0 ? a.H : a.G) * a.dk) + a.eps);
+    }
     __syncthreads();
   }
   for (int hs = warp; hs < n_slots; hs += kCapWarps) {
@@ -439,7 +437,7 @@ conv_attn_prep_joint_kernel(CapArgs a) {
             const bool first = a.half_layout ? d < half : (d & 1) == 0;
             const int j = a.half_layout ? (first ? d : d - half) : d >> 1;
             const float o = head[a.half_layout ? (first ? d + half : d - half) : d ^ 1];
-            const float2 t = cs[r * half + j];
+            const float2 t = a.cs[row * half + j];
             y = first ? y * t.x - o * t.y : y * t.x + o * t.y;
           }
           ca_store(dst + d, y);
@@ -466,7 +464,7 @@ extern "C" int b200_conv_attn_prep_ex(const void* proj, int f32, int64_t ld, con
                                    const int32_t* state_slots, const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles,
                                    int tile_rows, int n_prompt, int n_single, const int32_t* slots, void* q_out,
                                    void* k_cache, void* v_cache, int H, int G, int dk, int dv, int wk, int wv, int page,
-                                   float eps, int joint_norm, int rot_dims, int half_layout, const double* freq, void* stream) {
+                                   float eps, int joint_norm, int rot_dims, int half_layout, const float* cos_sin, void* stream) {
   B200_REQUIRE(H > 0 && G > 0 && H % G == 0 && dk > 0 && dv > 0 && wk >= dk && wv >= dv && page > 0,
                "conv_attn_prep: bad shape H=%d G=%d dk=%d dv=%d in %d / %d", H, G, dk, dv, wk, wv);
   B200_REQUIRE(taps >= 1 && taps <= kCapMaxTaps, "conv_attn_prep: %d taps (1 .. %d)", taps, kCapMaxTaps);
@@ -474,17 +472,17 @@ extern "C" int b200_conv_attn_prep_ex(const void* proj, int f32, int64_t ld, con
   B200_REQUIRE(n_tiles == 0 || (tile_rows > 0 && tile_rows % kCapRows == 0), "conv_attn_prep: tiles of %d rows (multiples of %d)",
                tile_rows, kCapRows);
   B200_REQUIRE(n_tiles >= 0 && n_prompt >= 0 && n_single >= 0, "conv_attn_prep: bad counts");
-  B200_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk && (rot_dims == 0 || freq != nullptr),
+  B200_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dk && (rot_dims == 0 || cos_sin != nullptr),
                "conv_attn_prep: %d rotated entries of %d", rot_dims, dk);
   B200_REQUIRE(!joint_norm || (qnorm_w != nullptr && knorm_w != nullptr), "conv_attn_prep: the joint norm has weights");
-  int per_tile = n_tiles > 0 ? tile_rows / kCapRows : 1;
-  int n_x = n_tiles * per_tile + n_single;
+  const int per_tile = n_tiles > 0 ? tile_rows / kCapRows : 1;
+  const int n_x = n_tiles * per_tile + n_single;
   if (n_x == 0) return B200_OK;
   int shift = 0;
   while ((1 << shift) < page) ++shift;
-  CapArgs a{proj, ld, conv_w, (const bf16*)qnorm_w, (const bf16*)knorm_w, taps > 1 ? ring : nullptr, cu_seq, ctx_lens,
+  const CapArgs a{proj, ld, conv_w, (const bf16*)qnorm_w, (const bf16*)knorm_w, taps > 1 ? ring : nullptr, cu_seq, ctx_lens,
                   state_slots, tile_seq, tile_q0, n_tiles * per_tile, per_tile, n_prompt, slots, q_out, k_cache, v_cache, H, G,
-                  dk, dv, wk, wv, page, (1 << shift) == page ? shift : -1, taps, eps, joint_norm, rot_dims, half_layout, freq};
+                  dk, dv, wk, wv, page, (1 << shift) == page ? shift : -1, taps, eps, joint_norm, rot_dims, half_layout, (const float2*)cos_sin};
   cudaStream_t s = (cudaStream_t)stream;
   const int n_heads = H + 2 * G, esz = f32 ? 4 : 2, vec = 16 / esz, wmax = wk > wv ? wk : wv;
   const int C = (H + G) * dk + G * dv;
@@ -492,17 +490,30 @@ extern "C" int b200_conv_attn_prep_ex(const void* proj, int f32, int64_t ld, con
                     reinterpret_cast<uintptr_t>(v_cache) | reinterpret_cast<uintptr_t>(conv_w) | reinterpret_cast<uintptr_t>(a.ring)) & 15) == 0;
   if (joint_norm || rot_dims > 0) {
     const int piece = half_layout ? 2 * vec : vec;      // the rotated entries in whole pieces (and their partners too)
+    int lph = 1;
+    while (lph < wmax / vec) lph <<= 1;
+    // a power of two of CTAs (one cluster) that covers all head slots, in CTAs of equal size
+    const int all_warps = lph <= 32 ? (n_heads + 32 / lph - 1) / (32 / lph) : 1 << 20;
+    int ny = 1;
+    while (ny < 8 && ny * kCapJointWarps < all_warps) ny <<= 1;
+    const size_t smem_v = sizeof(float2) * kCapRows * (size_t)(rot_dims / 2);
     if (al && taps <= 4 && dk % vec == 0 && dv % vec == 0 && wk % vec == 0 && wv % vec == 0 && ld % vec == 0 && C % 4 == 0 &&
-        wmax / vec <= 32 && rot_dims % piece == 0) {
-      constexpr int NB = 4;
-      int lph = 1;
-      while (lph < wmax / vec) lph <<= 1;
-      a.per_tile = n_tiles > 0 ? tile_rows / NB : 1;
-      a.n_pieces = n_tiles * a.per_tile;
-      const int all_warps = (n_heads + 32 / lph - 1) / (32 / lph), rounds = (all_warps + kCapJointWarps - 1) / kCapJointWarps;
-      const int warps = (all_warps + rounds - 1) / rounds;
-      const size_t smem = sizeof(float2) * NB * (size_t)(rot_dims / 2);
-#define B200_CAJ(TA, N) conv_attn_prep_joint_vec_kernel<TA, N, NB><<<a.n_pieces + n_single, warps * 32, smem, s>>>(a, lph)
+        ny * kCapJointWarps >= all_warps && rot_dims % piece == 0 && smem_v <= 32 * 1024) {
+      const int warps = (all_warps + ny - 1) / ny;
+      cudaLaunchConfig_t cfg = {};
+      cudaLaunchAttribute at[1];
+      at[0].id = cudaLaunchAttributeClusterDimension;
+      at[0].val.clusterDim.x = 1;
+      at[0].val.clusterDim.y = ny;
+      at[0].val.clusterDim.z = 1;
+      cfg.gridDim = dim3(n_x, ny);
+      cfg.blockDim = dim3(warps * 32);
+      cfg.dynamicSmemBytes = smem_v;
+      cfg.stream = s;
+      cfg.attrs = at;
+      cfg.numAttrs = 1;
+      cudaError_t e = cudaSuccess;
+#define B200_CAJ(TA, N) e = cudaLaunchKernelEx(&cfg, conv_attn_prep_joint_vec_kernel<TA, N>, a, lph)
 #define B200_CAJT(TA)                        \
   switch (taps) {                            \
     case 1: B200_CAJ(TA, 1); break;          \
@@ -513,10 +524,14 @@ extern "C" int b200_conv_attn_prep_ex(const void* proj, int f32, int64_t ld, con
       if (f32) { B200_CAJT(float) } else { B200_CAJT(bf16) }
 #undef B200_CAJT
 #undef B200_CAJ
+      if (e != cudaSuccess) {
+        b200_set_error("conv_attn_prep(joint): %s", cudaGetErrorString(e));
+        return B200_ERR_CUDA;
+      }
       return b200_check_launch("b200_conv_attn_prep(joint)");
     }
-    const size_t smem = sizeof(float2) * kCapRows * (size_t)(rot_dims / 2) + sizeof(float) * kCapWarps * (dk > dv ? dk : dv);
-    B200_REQUIRE(smem <= 40 * 1024, "conv_attn_prep: heads of %d / %d entries, %d rotated, exceed the staged head", dk, dv, rot_dims);
+    const size_t smem = sizeof(float) * kCapWarps * (dk > dv ? dk : dv);
+    B200_REQUIRE(smem <= 40 * 1024, "conv_attn_prep: heads of %d / %d entries exceed the staged head", dk, dv);
     if (f32) conv_attn_prep_joint_kernel<float><<<n_x, kCapWarps * 32, smem, s>>>(a);
     else conv_attn_prep_joint_kernel<bf16><<<n_x, kCapWarps * 32, smem, s>>>(a);
     return b200_check_launch("b200_conv_attn_prep(joint)");
@@ -557,4 +572,11 @@ extern "C" int b200_conv_attn_prep(const void* proj, int f32, int64_t ld, const 
   return b200_conv_attn_prep_ex(proj, f32, ld, conv_w, taps, qnorm_w, knorm_w, ring, cu_seq, ctx_lens, state_slots, tile_seq, tile_q0,
                                 n_tiles, tile_rows, n_prompt, n_single, slots, q_out, k_cache, v_cache, H, G, dk, dv, wk, wv, page, eps,
                                 0, 0, 0, nullptr, stream);
+}
+
+extern "C" int b200_rot_table(const int32_t* positions, const double* freq, float* cos_sin, int T, int half, void* stream) {
+  B200_REQUIRE(T >= 0 && half > 0, "rot_table: bad shape");
+  if (T == 0) return B200_OK;
+  rot_table_kernel<<<(T * half + 255) / 256, 256, 0, (cudaStream_t)stream>>>(positions, freq, (float2*)cos_sin, half, T * half);
+  return b200_check_launch("b200_rot_table");
 }

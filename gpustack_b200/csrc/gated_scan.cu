@@ -9,11 +9,12 @@
 // projections are fp32 rows, and everything formed from them is fp32.  The state of slot s is S [slots][H][dv][dkp] (key index
 // fastest, dkp = dk rounded up to 4).  A sequence whose context is empty starts from zero, whatever its slot held.
 //
-// Every value column of S is a recurrence of its own, so columns are the unit of work: L lanes share a column, lane l holds
-// the key entries 4 (i L + l) .. + 3 (i < R4) of it in registers, and a warp walks its 32 / L columns through the sequence's
-// new rows one token after the other.  Per token: S^T k (a butterfly over the L lanes; delta rule only), the update, and
-// the lane's share of S^T q.  Those shares stay in registers for 8 tokens and are then summed over the lanes in one
-// transposing exchange (7 shuffles for 8 tokens).  Keys, queries, values and gates are staged 16 tokens at a time by
+// Every value column of S is a recurrence of its own, so columns are the unit of work: L lanes share C neighbouring columns,
+// lane l holds the key entries 4 (i L + l) .. + 3 (i < R4) of each in registers, and a warp walks its C 32 / L columns
+// through the sequence's new rows one token after the other.  Per token: S^T k (a butterfly over the L lanes; delta rule
+// only), the update, and the lane's share of S^T q.  Those shares stay in registers for 8 tokens and are then summed over the
+// lanes in one transposing exchange (about 2 shuffles a token).  A token's keys and queries are read from shared memory once
+// per lane and serve its C columns: with one column that read, not the arithmetic, bounds the walk.  Keys, queries, values and gates are staged 16 or 32 tokens at a time by
 // cp.async into two buffers, so the walk never waits for memory; a column's sums do not depend on how a prompt was cut
 // beyond the order of the lanes' addends in S^T q.
 #include "common.cuh"
@@ -22,7 +23,7 @@
 
 namespace b200 {
 
-constexpr int kGsWarps = 8, kGsTok = 16;
+constexpr int kGsWarps = 8;
 
 struct GatedScanArgs {
   const float* x;
@@ -58,6 +59,11 @@ __device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
   return r;
 }
+__device__ __forceinline__ f32x2 add2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
 __device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
   f32x2 r;
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
@@ -84,29 +90,64 @@ __device__ __forceinline__ float lanes_sum(float v) {
   return v;
 }
 
-// One token of a column: the decayed, updated state and the lane's share of S^T q
-template <int L, int R2, bool DELTA>
-__device__ __forceinline__ float gs_token(f32x2 (&S)[R2], const f32x2 (&k)[R2], const f32x2 (&q)[R2], float v, float2 gb) {
-  float u = gb.y * v;
-  if (DELTA) {
-    f32x2 p0 = mul2(S[0], k[0]), p1 = mul2(S[1], k[1]);
+// the lane's shares of S^T x for C columns
+template <int R2, int C>
+__device__ __forceinline__ void gs_dot(const f32x2 (&S)[C][R2], const f32x2 (&x)[R2], float (&o)[C]) {
+#pragma unroll
+  for (int c = 0; c < C; ++c) {
+    f32x2 p0 = mul2(S[c][0], x[0]), p1 = mul2(S[c][1], x[1]);
 #pragma unroll
     for (int i = 2; i < R2; i += 2) {
-      p0 = fma2(S[i], k[i], p0);
-      p1 = fma2(S[i + 1], k[i + 1], p1);
+      p0 = fma2(S[c][i], x[i], p0);
+      p1 = fma2(S[c][i + 1], x[i + 1], p1);
     }
-    u = gb.y * (v - gb.x * lanes_sum<L>(sum2(p0) + sum2(p1)));
+    o[c] = sum2(add2(p0, p1));
   }
-  const f32x2 g2 = pack2(gb.x, gb.x), u2 = pack2(u, u);
-  f32x2 o0 = 0, o1 = 0;            // (two positive zeros)
+}
+
+// sums over the L lanes of a group, in every lane.  Two columns: the lanes' halves take one each and exchange the sums.
+template <int L, int C>
+__device__ __forceinline__ void gs_lanes_sum(float (&p)[C]) {
+  if constexpr (C == 2 && L > 8) {
+    const bool hi = threadIdx.x & (L / 2);
+    float mine = (hi ? p[1] : p[0]) + __shfl_xor_sync(0xffffffffu, hi ? p[0] : p[1], L / 2);
 #pragma unroll
-  for (int i = 0; i < R2; i += 2) {
-    S[i] = fma2(k[i], u2, mul2(g2, S[i]));
-    S[i + 1] = fma2(k[i + 1], u2, mul2(g2, S[i + 1]));
-    o0 = fma2(S[i], q[i], o0);
-    o1 = fma2(S[i + 1], q[i + 1], o1);
+    for (int w = L / 4; w > 0; w >>= 1) mine += __shfl_xor_sync(0xffffffffu, mine, w);
+    const float other = __shfl_xor_sync(0xffffffffu, mine, L / 2);
+    p[0] = hi ? other : mine;
+    p[1] = hi ? mine : other;
+  } else {
+#pragma unroll
+    for (int w = L / 2; w > 0; w >>= 1)
+#pragma unroll
+      for (int c = 0; c < C; ++c) p[c] += __shfl_xor_sync(0xffffffffu, p[c], w);
   }
-  return sum2(o0) + sum2(o1);
+}
+
+// One token of C columns: S <- g S + k u^T with u = beta v, or beta (v - g S^T k) for the delta rule.  The read-out of the
+// token BEFORE (o, from q; none for a block's first token) and the decay of S need no other lane: they run while the
+// butterfly's shuffles are in flight.
+template <int L, int R2, int C, bool DELTA, bool READ>
+__device__ __forceinline__ void gs_token(f32x2 (&S)[C][R2], const f32x2 (&k)[R2], const f32x2 (&q)[R2], const float (&v)[C], float2 gb,
+                                         float (&o)[C]) {
+  float p[C];
+  if (DELTA) {
+    gs_dot<R2, C>(S, k, p);
+    gs_lanes_sum<L, C>(p);
+  }
+  if (READ) gs_dot<R2, C>(S, q, o);
+  const f32x2 g2 = pack2(gb.x, gb.x);
+#pragma unroll
+  for (int c = 0; c < C; ++c)
+#pragma unroll
+    for (int i = 0; i < R2; ++i) S[c][i] = mul2(g2, S[c][i]);
+#pragma unroll
+  for (int c = 0; c < C; ++c) {
+    const float u = DELTA ? gb.y * (v[c] - gb.x * p[c]) : gb.y * v[c];
+    const f32x2 u2 = pack2(u, u);
+#pragma unroll
+    for (int i = 0; i < R2; ++i) S[c][i] = fma2(k[i], u2, S[c][i]);
+  }
 }
 
 // 4 R4 entries of a row of key entries: lane l of L takes entries 4 (i L + l) .. + 3
@@ -120,39 +161,41 @@ __device__ __forceinline__ void gs_row(const float* __restrict__ row, int l, f32
   }
 }
 
-template <int L, int R4, bool DELTA>
-__global__ void __launch_bounds__(kGsWarps * 32)
+template <int L, int R4, int C, int TOK, bool DELTA>
+__global__ void __launch_bounds__(kGsWarps * 32, C * R4 <= 4 ? 2 : 1)
 gated_scan_kernel(GatedScanArgs a) {
   extern __shared__ __align__(16) float smem[];
-  constexpr int R2 = 2 * R4, DKP = 4 * R4 * L, CPW = 32 / L, COLS = kGsWarps * CPW;
-  float* ks = smem;                                   // [2][16][DKP]
-  float* qs = ks + 2 * kGsTok * DKP;                  // [2][16][DKP]
-  float* vs = qs + 2 * kGsTok * DKP;                  // [2][16][COLS]
-  float2* gb = reinterpret_cast<float2*>(vs + 2 * kGsTok * COLS);   // [2][16]
-  float* os = reinterpret_cast<float*>(gb + 2 * kGsTok);            // [16][COLS + 1]
+  constexpr int R2 = 2 * R4, DKP = 4 * R4 * L, CPW = C * 32 / L, COLS = kGsWarps * CPW, OP = COLS + 8;
+  float* ks = smem;                                   // [2][TOK][DKP]
+  float* qs = ks + 2 * TOK * DKP;                  // [2][TOK][DKP]
+  float* vs = qs + 2 * TOK * DKP;                  // [2][TOK][COLS]
+  float2* gb = reinterpret_cast<float2*>(vs + 2 * TOK * COLS);   // [2][TOK]
+  float* os = reinterpret_cast<float*>(gb + 2 * TOK);            // [TOK][OP]
   const int s = blockIdx.x, h = blockIdx.y, z = blockIdx.z, tid = threadIdx.x;
   const int slot = a.state_slots[s];
   if (slot < 0) return;
   const int t0 = a.cu_seq[s], t1 = a.cu_seq[s + 1];
   if (t1 <= t0) return;
   const int warp = tid >> 5, lane = tid & 31, l = lane % L;
-  const int cw = warp * CPW + lane / L, col = z * COLS + cw;         // this lane's column, in the CTA and in the head
+  const int cw = warp * CPW + lane / L * C, col = z * COLS + cw;     // this lane's first column, in the CTA and in the head
   const int hk = h / (a.H / a.G);
   const int dkp = a.dkp;
   float* Sp = a.S + (((size_t)slot * a.H + h) * a.dv + col) * dkp;
   const bool fresh = a.ctx_lens[s] == 0;
-  f32x2 S[R2];
+  f32x2 S[C][R2];
 #pragma unroll
-  for (int i = 0; i < R4; ++i) {
-    ulonglong2 t = make_ulonglong2(0, 0);
-    if (!fresh && col < a.dv && 4 * (i * L + l) < dkp) t = *reinterpret_cast<const ulonglong2*>(Sp + 4 * (i * L + l));
-    S[2 * i] = t.x;
-    S[2 * i + 1] = t.y;
-  }
+  for (int c = 0; c < C; ++c)
+#pragma unroll
+    for (int i = 0; i < R4; ++i) {
+      ulonglong2 t = make_ulonglong2(0, 0);
+      if (!fresh && col + c < a.dv && 4 * (i * L + l) < dkp) t = *reinterpret_cast<const ulonglong2*>(Sp + c * dkp + 4 * (i * L + l));
+      S[c][2 * i] = t.x;
+      S[c][2 * i + 1] = t.y;
+    }
   // key entries behind dkp: zeros in both buffers, written once
   if (dkp < DKP) {
     const int pad = DKP - dkp;
-    for (int i = tid; i < 2 * kGsTok * pad; i += kGsWarps * 32) {
+    for (int i = tid; i < 2 * TOK * pad; i += kGsWarps * 32) {
       const int r = i / pad, d = dkp + i % pad;
       ks[r * DKP + d] = 0.f;
       qs[r * DKP + d] = 0.f;
@@ -160,12 +203,16 @@ gated_scan_kernel(GatedScanArgs a) {
   }
   const float rate = a.rate[h], bias = a.dt_bias[h];
   const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
-  auto stage = [&](int ch, int buf) {                 // rows ch .. ch + 15; rows behind the portion are zeros
-    const int nt = min(kGsTok, t1 - ch), dk4 = dkp >> 2;
-    for (int i = tid; i < kGsTok * dk4; i += kGsWarps * 32) {
-      const int tt = i / dk4, d = (i - tt * dk4) * 4, to = (buf * kGsTok + tt) * DKP + d;
+  // this thread's share of the staging: entries d0 .. d0 + 3 of rows tt0, tt0 + per_pass, ... (dkp <= 512: at least one pass)
+  const int dk4 = dkp >> 2, per_pass = kGsWarps * 32 / dk4, d0 = tid % dk4 * 4;
+  const int tt0 = tid / dk4 < per_pass ? tid / dk4 : TOK;
+  const float* src = a.x + hk * dkp + d0;
+  auto stage = [&](int ch, int buf) {                 // rows ch .. ch + TOK - 1; rows behind the portion are zeros
+    const int nt = min(TOK, t1 - ch);
+    for (int tt = tt0; tt < TOK; tt += per_pass) {
+      const int to = (buf * TOK + tt) * DKP + d0;
       if (tt < nt) {
-        const float* row = a.x + (size_t)(ch + tt) * a.ld + hk * dkp + d;
+        const float* row = src + (size_t)(ch + tt) * a.ld;
         cp16(ks + to, row + a.k_col);
         cp16(qs + to, row + a.q_col);
       } else {
@@ -173,9 +220,9 @@ gated_scan_kernel(GatedScanArgs a) {
         *reinterpret_cast<float4*>(qs + to) = zero4;
       }
     }
-    for (int i = tid; i < kGsTok * (COLS / 4); i += kGsWarps * 32) {
+    for (int i = tid; i < TOK * (COLS / 4); i += kGsWarps * 32) {
       const int tt = i / (COLS / 4), c = (i - tt * (COLS / 4)) * 4;
-      float* to = vs + (buf * kGsTok + tt) * COLS + c;
+      float* to = vs + (buf * TOK + tt) * COLS + c;
       if (tt < nt && z * COLS + c < a.dvp) cp16(to, a.x + (size_t)(ch + tt) * a.ld + a.v_col + h * a.dvp + z * COLS + c);
       else *reinterpret_cast<float4*>(to) = zero4;
     }
@@ -183,21 +230,21 @@ gated_scan_kernel(GatedScanArgs a) {
   };
   float ra = 0.f, rb = 0.f;
   auto raw_gates = [&](int ch) {
-    if (tid < kGsTok && ch + tid < t1) {
+    if (tid < TOK && ch + tid < t1) {
       const float* g = a.gates + (size_t)(ch + tid) * a.ld_g;
       ra = DELTA ? g[a.H + h] : g[h];
       if (DELTA) rb = g[h];
     }
   };
   auto put_gates = [&](int ch, int buf) {             // rows behind the portion: decay 1, step 0 (the state stays)
-    if (tid < kGsTok) gb[buf * kGsTok + tid] = ch + tid < t1 ? gs_gate<DELTA>(ra, rb, rate, bias) : make_float2(1.f, 0.f);
+    if (tid < TOK) gb[buf * TOK + tid] = ch + tid < t1 ? gs_gate<DELTA>(ra, rb, rate, bias) : make_float2(1.f, 0.f);
   };
   stage(t0, 0);
   raw_gates(t0);
   put_gates(t0, 0);
   int buf = 0;
-  for (int ch = t0; ch < t1; ch += kGsTok, buf ^= 1) {
-    const int nt = min(kGsTok, t1 - ch), next = ch + kGsTok;
+  for (int ch = t0; ch < t1; ch += TOK, buf ^= 1) {
+    const int nt = min(TOK, t1 - ch), next = ch + TOK;
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                  // this chunk is staged; the last one's outputs have left os
     if (next < t1) {
@@ -206,34 +253,56 @@ gated_scan_kernel(GatedScanArgs a) {
     }
 #pragma unroll 1
     for (int tb = 0; tb < nt; tb += 8) {
-      float o[8];
+      float o[8][C];
+      f32x2 k[2][R2], q[2][R2];      // this token's and the next one's keys; the last token's and this one's queries
+      const float* kr = ks + (buf * TOK + tb) * DKP;
+      const float* qr = qs + (buf * TOK + tb) * DKP;
+      const float* vr = vs + (buf * TOK + tb) * COLS + cw;
+      const float2* gr = gb + buf * TOK + tb;
+      gs_row<L, R4>(kr, l, k[0]);
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        const int tt = buf * kGsTok + tb + j;
-        f32x2 k[R2], q[R2];
-        gs_row<L, R4>(ks + tt * DKP, l, k);
-        gs_row<L, R4>(qs + tt * DKP, l, q);
-        o[j] = gs_token<L, R2, DELTA>(S, k, q, vs[tt * COLS + cw], gb[tt]);
+        float v[C];
+#pragma unroll
+        for (int c = 0; c < C; ++c) v[c] = vr[j * COLS + c];
+        if (j < 7) gs_row<L, R4>(kr + (j + 1) * DKP, l, k[(j + 1) & 1]);
+        gs_row<L, R4>(qr + j * DKP, l, q[j & 1]);
+        if (j == 0) gs_token<L, R2, C, DELTA, false>(S, k[0], q[1], v, gr[0], o[0]);
+        else gs_token<L, R2, C, DELTA, true>(S, k[j & 1], q[(j + 1) & 1], v, gr[j], o[j - 1]);
       }
-      // lane l ends with token tb + (l & 7), summed over the column's lanes
+      gs_dot<R2, C>(S, q[1], o[7]);
+      // lane l ends with token tb + (l & 7), summed over the columns' lanes
       const bool b4 = l & 4, b2 = l & 2, b1 = l & 1;
+      float sum[C];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float mine = b4 ? o[j + 4] : o[j], other = b4 ? o[j] : o[j + 4];
-        o[j] = mine + __shfl_xor_sync(0xffffffffu, other, 4);
-      }
+      for (int c = 0; c < C; ++c) {
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const float mine = b2 ? o[j + 2] : o[j], other = b2 ? o[j] : o[j + 2];
-        o[j] = mine + __shfl_xor_sync(0xffffffffu, other, 2);
-      }
-      {
-        const float mine = b1 ? o[1] : o[0], other = b1 ? o[0] : o[1];
-        o[0] = mine + __shfl_xor_sync(0xffffffffu, other, 1);
-      }
+        for (int j = 0; j < 4; ++j) {
+          const float mine = b4 ? o[j + 4][c] : o[j][c], other = b4 ? o[j][c] : o[j + 4][c];
+          o[j][c] = mine + __shfl_xor_sync(0xffffffffu, other, 4);
+        }
 #pragma unroll
-      for (int w = 8; w < L; w <<= 1) o[0] += __shfl_xor_sync(0xffffffffu, o[0], w);
-      if (l < 8) os[(tb + l) * (COLS + 1) + cw] = o[0];
+        for (int j = 0; j < 2; ++j) {
+          const float mine = b2 ? o[j + 2][c] : o[j][c], other = b2 ? o[j][c] : o[j + 2][c];
+          o[j][c] = mine + __shfl_xor_sync(0xffffffffu, other, 2);
+        }
+        const float mine = b1 ? o[1][c] : o[0][c], other = b1 ? o[0][c] : o[1][c];
+        sum[c] = mine + __shfl_xor_sync(0xffffffffu, other, 1);
+      }
+      if constexpr (C == 2 && L > 8) {                 // the lanes' halves of 8 take one column each
+        const bool hi = l & 8;
+        float one = (hi ? sum[1] : sum[0]) + __shfl_xor_sync(0xffffffffu, hi ? sum[0] : sum[1], 8);
+#pragma unroll
+        for (int w = 16; w < L; w <<= 1) one += __shfl_xor_sync(0xffffffffu, one, w);
+        if (l < 16) os[(tb + (l & 7)) * OP + cw + (hi ? 1 : 0)] = one;
+      } else {
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+#pragma unroll
+          for (int w = 8; w < L; w <<= 1) sum[c] += __shfl_xor_sync(0xffffffffu, sum[c], w);
+          if (l < 8) os[(tb + l) * OP + cw + c] = sum[c];
+        }
+      }
     }
     if (next < t1) put_gates(next, buf ^ 1);
     __syncthreads();
@@ -242,18 +311,20 @@ gated_scan_kernel(GatedScanArgs a) {
       const int tt = i / COLS, c = i - tt * COLS;
       if (z * COLS + c < a.dv)
         a.o[(size_t)(ch + tt) * a.H * a.dv + h * a.dv + z * COLS + c] =
-            fmaf(sk, vs[(buf * kGsTok + tt) * COLS + c], os[tt * (COLS + 1) + c]);
+            fmaf(sk, vs[(buf * TOK + tt) * COLS + c], os[tt * OP + c]);
     }
   }
 #pragma unroll
-  for (int i = 0; i < R4; ++i)
-    if (col < a.dv && 4 * (i * L + l) < dkp)
-      *reinterpret_cast<ulonglong2*>(Sp + 4 * (i * L + l)) = make_ulonglong2(S[2 * i], S[2 * i + 1]);
+  for (int c = 0; c < C; ++c)
+#pragma unroll
+    for (int i = 0; i < R4; ++i)
+      if (col + c < a.dv && 4 * (i * L + l) < dkp)
+        *reinterpret_cast<ulonglong2*>(Sp + c * dkp + 4 * (i * L + l)) = make_ulonglong2(S[c][2 * i], S[c][2 * i + 1]);
 }
 
 // Single rows (a decode step): the state, the token's rows and its gates are in flight together; no staging, no barrier.
 template <int L, int R4, bool DELTA>
-__global__ void __launch_bounds__(kGsWarps * 32)
+__global__ void __launch_bounds__(kGsWarps * 32, 1)
 gated_step_kernel(GatedScanArgs a) {
   constexpr int R2 = 2 * R4, CPW = 32 / L, COLS = kGsWarps * CPW;
   const int s = blockIdx.x, h = blockIdx.y, z = blockIdx.z;
@@ -266,7 +337,7 @@ gated_step_kernel(GatedScanArgs a) {
   const bool live = col < a.dv, fresh = a.ctx_lens[s] == 0;
   float* Sp = a.S + (((size_t)slot * a.H + h) * a.dv + col) * dkp;
   const float* row = a.x + (size_t)t * a.ld;
-  f32x2 S[R2], k[R2], q[R2];
+  f32x2 S[1][R2], k[R2], q[R2];
 #pragma unroll
   for (int i = 0; i < R4; ++i) {
     const int d = 4 * (i * L + l);
@@ -276,51 +347,62 @@ gated_step_kernel(GatedScanArgs a) {
       tk = *reinterpret_cast<const ulonglong2*>(row + a.k_col + hk * dkp + d);
       tq = *reinterpret_cast<const ulonglong2*>(row + a.q_col + hk * dkp + d);
     }
-    S[2 * i] = ts.x; S[2 * i + 1] = ts.y;
+    S[0][2 * i] = ts.x; S[0][2 * i + 1] = ts.y;
     k[2 * i] = tk.x; k[2 * i + 1] = tk.y;
     q[2 * i] = tq.x; q[2 * i + 1] = tq.y;
   }
-  const float v = live ? row[a.v_col + h * a.dvp + col] : 0.f;
+  const float v[1] = {live ? row[a.v_col + h * a.dvp + col] : 0.f};
   const float* g = a.gates + (size_t)t * a.ld_g;
   const float2 gb = gs_gate<DELTA>(DELTA ? g[a.H + h] : g[h], DELTA ? g[h] : 0.f, a.rate[h], a.dt_bias[h]);
-  const float o = lanes_sum<L>(gs_token<L, R2, DELTA>(S, k, q, v, gb));
+  float o[1];
+  gs_token<L, R2, 1, DELTA, false>(S, k, q, v, gb, o);
+  gs_dot<R2, 1>(S, q, o);
+  o[0] = lanes_sum<L>(o[0]);
   if (!live) return;
 #pragma unroll
   for (int i = 0; i < R4; ++i) {
     const int d = 4 * (i * L + l);
-    if (d < dkp) *reinterpret_cast<ulonglong2*>(Sp + d) = make_ulonglong2(S[2 * i], S[2 * i + 1]);
+    if (d < dkp) *reinterpret_cast<ulonglong2*>(Sp + d) = make_ulonglong2(S[0][2 * i], S[0][2 * i + 1]);
   }
-  if (l == 0) a.o[(size_t)t * a.H * a.dv + h * a.dv + col] = a.skip != nullptr ? fmaf(a.skip[h], v, o) : o;
+  if (l == 0) a.o[(size_t)t * a.H * a.dv + h * a.dv + col] = a.skip != nullptr ? fmaf(a.skip[h], v[0], o[0]) : o[0];
 }
 
-template <int L, int R4, bool DELTA>
-int gated_scan_launch(const GatedScanArgs& a, int n_seqs, int max_len, cudaStream_t s) {
-  constexpr int COLS = kGsWarps * (32 / L), DKP = 4 * R4 * L;
+template <int L, int R4, int C, bool DELTA>
+int gated_scan_launch(const GatedScanArgs& a, int n_seqs, cudaStream_t s) {
+  constexpr int COLS = kGsWarps * C * (32 / L), DKP = 4 * R4 * L;
+  constexpr int TOK = DKP <= 128 ? 32 : 16;
   const dim3 grid(n_seqs, a.H, (a.dv + COLS - 1) / COLS);
-  if (max_len == 1) {
-    gated_step_kernel<L, R4, DELTA><<<grid, kGsWarps * 32, 0, s>>>(a);
-    return b200_check_launch("b200_gated_scan(step)");
-  }
-  constexpr size_t smem = sizeof(float) * (4 * (size_t)kGsTok * DKP + 2 * kGsTok * COLS + 4 * kGsTok + kGsTok * (COLS + 1));
+  constexpr size_t smem = sizeof(float) * (4 * (size_t)TOK * DKP + 2 * TOK * COLS + 4 * TOK + TOK * (COLS + 8));
   if (smem > 48 * 1024) {
-    const cudaError_t e = cudaFuncSetAttribute(gated_scan_kernel<L, R4, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const cudaError_t e = cudaFuncSetAttribute(gated_scan_kernel<L, R4, C, TOK, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) {
       b200_set_error("gated_scan: %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
       return B200_ERR_CUDA;
     }
   }
-  gated_scan_kernel<L, R4, DELTA><<<grid, kGsWarps * 32, smem, s>>>(a);
+  gated_scan_kernel<L, R4, C, TOK, DELTA><<<grid, kGsWarps * 32, smem, s>>>(a);
   return b200_check_launch("b200_gated_scan");
+}
+
+// L, R4: single rows; PL, PR4: prompt portions (fewer entries of two columns per lane: the same registers, half the reads)
+template <int L, int R4, int PL, int PR4, bool DELTA>
+int gated_scan_form(const GatedScanArgs& a, int n_seqs, int max_len, cudaStream_t s) {
+  if (max_len == 1) {
+    constexpr int COLS = kGsWarps * (32 / L);
+    gated_step_kernel<L, R4, DELTA><<<dim3(n_seqs, a.H, (a.dv + COLS - 1) / COLS), kGsWarps * 32, 0, s>>>(a);
+    return b200_check_launch("b200_gated_scan(step)");
+  }
+  return gated_scan_launch<PL, PR4, 2, DELTA>(a, n_seqs, s);
 }
 
 template <bool DELTA>
 int gated_scan_pick(const GatedScanArgs& a, int n_seqs, int max_len, cudaStream_t s) {
-  if (a.dkp <= 32) return gated_scan_launch<8, 1, DELTA>(a, n_seqs, max_len, s);
-  if (a.dkp <= 64) return gated_scan_launch<8, 2, DELTA>(a, n_seqs, max_len, s);
-  if (a.dkp <= 96) return gated_scan_launch<8, 3, DELTA>(a, n_seqs, max_len, s);
-  if (a.dkp <= 128) return gated_scan_launch<8, 4, DELTA>(a, n_seqs, max_len, s);
-  if (a.dkp <= 256) return gated_scan_launch<16, 4, DELTA>(a, n_seqs, max_len, s);
-  return gated_scan_launch<32, 4, DELTA>(a, n_seqs, max_len, s);
+  if (a.dkp <= 32) return gated_scan_form<8, 1, 8, 1, DELTA>(a, n_seqs, max_len, s);
+  if (a.dkp <= 64) return gated_scan_form<8, 2, 16, 1, DELTA>(a, n_seqs, max_len, s);
+  if (a.dkp <= 96) return gated_scan_form<8, 3, 8, 3, DELTA>(a, n_seqs, max_len, s);
+  if (a.dkp <= 128) return gated_scan_form<8, 4, 16, 2, DELTA>(a, n_seqs, max_len, s);
+  if (a.dkp <= 256) return gated_scan_form<16, 4, 32, 2, DELTA>(a, n_seqs, max_len, s);
+  return gated_scan_form<32, 4, 32, 4, DELTA>(a, n_seqs, max_len, s);
 }
 
 // ------------------------------------------------------------------------------------------- out

@@ -1,7 +1,7 @@
-"""Side benchmark of the layer-list family (Vodavik, Danipel, Resevik, Dotorax, Kerarax) beside the closest existing model of equal layer
+"""Side benchmark of the layer-list family (Vodavik, Danipel, Resevik, Dotorax, Kerarax, Bovitar) beside the closest existing model of equal layer
 sizes (a Llama-class decoder; for Resevik also Vodavik, the other design with attention and recurrent-state layers).
 
-`python bench.py --family vodavik|danipel|resevik|dotorax|kerarax` prints ONE JSON line (not the serving benchmark's line; that workload and its
+`python bench.py --family vodavik|danipel|resevik|dotorax|kerarax|bovitar` prints ONE JSON line (not the serving benchmark's line; that workload and its
 contract are untouched).  Random weights, synthetic tokens.  Two kinds of numbers:
 
   model:   prefill tokens/s (prompts of `prompt` tokens, `seqs` at a time through runner.prefill) and decode tokens/s
@@ -22,9 +22,9 @@ import numpy as np
 import torch
 
 from . import ops
-from .config import (AttentionSpec, EngineConfig, GatedLinearAttentionSpec, GatedRecurrenceSpec, LatentAttentionSpec,
+from .config import (AttentionSpec, DeltaRuleSpec, EngineConfig, GatedLinearAttentionSpec, GatedRecurrenceSpec, LatentAttentionSpec,
                      LayerListConfig, LayerSpec, LinearAttentionSpec, MLPSpec, MLSTMSpec, ModelConfig, MoESpec, RotarySpec,
-                     SideBySideSpec)
+                     SideBySideSpec, StateSpaceSpec)
 
 ROOT = Path(__file__).resolve().parent.parent
 SIZES = {
@@ -1025,12 +1025,212 @@ def _kernel_numbers_kerarax(size, T, B, ctx, log):
     return res
 
 
+# Bovitar at the same widths: taps, score cap, delta (heads, kv heads, width), state space (heads, width, state, groups),
+# experts, top, groups, kept groups, expert (and shared expert) ff
+BOVITAR = {"2k": (4, 30.0, (16, 8, 128), (32, 64, 128, 2), 8, 2, 4, 2, 2048), "4k": (4, 30.0, (32, 16, 128), (64, 64, 128, 2), 8, 2, 4, 2, 3584)}
+
+
+def bovitar_config(size: str, layers: int = 4) -> LayerListConfig:
+    """Delta-rule layers in turn with layers of attention beside a state-space recurrence, 8 routed SiLU experts (2 chosen
+    inside the best 2 of 4 groups, a shared one of the same width) in every layer."""
+    D, H, G, hd, ff, V = SIZES[size]
+    taps, cap, (dh, dg, dw), (sh, sw, sn, sg), E, top, groups, keep, ffe = BOVITAR[size]
+    specs = []
+    for i in range(layers):
+        moe = MoESpec(experts=E, top=top, ff=ffe, limit=0.0, scale=2.0, shared_ff=ffe, renormalize=False, act="silu", groups=groups,
+                      groups_keep=keep)
+        if i % 2 == 0:
+            mix = DeltaRuleSpec(dh, dg, dw, dw, taps)
+        else:
+            rot = RotarySpec(dims=hd, base=5e5, layout="half", wave_factor=8.0, wave_original=8192.0, wave_low=1.0, wave_high=4.0)
+            left = AttentionSpec(H, G, hd, hd, hd ** -0.5, qk_norm=True, qk_norm_joint=True, qkv_bias=False, sink=False, gate=False, rot=rot,
+                                 softcap=cap, conv_taps=taps)
+            mix = SideBySideSpec(left, StateSpaceSpec(sh, sw, sn, sg, taps, sg), 0.5, 0.5, branch_norm=True)
+        specs.append(LayerSpec(mix, MLPSpec("moe", ffe, act="silu", moe=moe)))
+    return LayerListConfig("Bovitar", V, D, specs, norm_eps=1e-5, residual="pre_norm", norm="rms", logit_scale=0.5)
+
+
+def _kernel_numbers_bovitar(size, T, B, ctx, log):
+    """Bovitar's kernels beside the like kernels of the closest models at equal sizes: Kerarax (convolved attention, joins with
+    the routed sum), Resevik and Dotorax (preparation of fp32 rows, linear attention with fixed and with data-dependent
+    decays), Danipel (corrected expert choice, shared expert)."""
+    D, H, G, hd, ff, V = SIZES[size]
+    taps, cap, (dh, dg, dw), (sh, sw, sn, sg), E, top, groups, keep, ffe = BOVITAR[size]
+    hbm, flops_peak, how = _peaks()
+    flush = _Flush()
+    dev = "cuda"
+    bf, f32 = torch.bfloat16, torch.float32
+    rnd = lambda *s, dt=bf, sc=1.0: (torch.randn(*s, device=dev, dtype=f32) * sc).to(dt)   # noqa: E731
+    i32 = lambda x: torch.as_tensor(x, dtype=torch.int32, device=dev)   # noqa: E731
+    res = {}
+
+    def put(name, new_s, new_work, like_name, like_s, like_work, kind):
+        peak = hbm if kind == "bytes" else flops_peak
+        fn, fl = new_work / new_s / peak, like_work / like_s / peak
+        res[name] = {"us": round(new_s * 1e6, 1), "frac_of_" + how + "_" + kind: round(fn, 4), "like": like_name,
+                     "like_us": round(like_s * 1e6, 1), "like_frac": round(fl, 4), "distance_ratio": round(fl / fn, 2)}
+        log(f"  {name:44s} {new_s * 1e6:9.1f} us  {fn:7.4f} of roofline | {like_name}: {like_s * 1e6:9.1f} us {fl:7.4f}"
+            f"  -> {fl / fn:5.2f}x as far")
+
+    S = max(1, T // 2048)
+    L = T // S
+    cu, ctx0, slot_s = i32(np.arange(S + 1) * L), i32(np.zeros(S)), i32(np.arange(S))
+    cud, ctxd, slot_b = i32(np.arange(B + 1)), i32(np.full(B, ctx)), i32(np.arange(B))
+    # ---- joins: one row, the normed pair, the routed sum
+    x32, y32, z32, w, w1, w2n = rnd(T, D, dt=f32), rnd(T, D, dt=f32), rnd(T, D, dt=f32), rnd(D), rnd(D), rnd(D)
+    xb = torch.empty(T, D, device=dev, dtype=bf)
+    yp, sh32 = rnd(T * top, D, dt=f32), rnd(T, D, dt=f32)
+    pr = i32(np.random.RandomState(1).permutation(T * top))
+    lg = rnd(T, 128, dt=f32)
+    for rows, tag in ((T, ""), (B, " (single rows)")):
+        x, y, z, h, s2, p = x32[:rows], y32[:rows], z32[:rows], xb[:rows], sh32[:rows], pr[:rows * top] % (rows * top)
+        t_like = _time(lambda: ops.add_rms_norm(x, w, 1e-5, a=y, x_out=x, xb_out=h), flush)
+        t_new = _time(lambda: ops.prenorm_join(x, w, 1e-5, y=y, x_out=x, h_out=h), flush)
+        put("prenorm_join" + tag, t_new, rows * D * 14.0, "add_rms_norm" + tag, t_like, rows * D * 14.0, "bytes")
+        t_like = _time(lambda: ops.add_rms_norm(x, w, 1e-5, a=y, b=z, x_out=x, xb_out=h), flush)
+        t_new = _time(lambda: ops.prenorm_join(x, w, 1e-5, pair=(y, z, w1, w2n, 0.5, 0.5), x_out=x, h_out=h), flush)
+        put("prenorm_join, normed pair" + tag, t_new, rows * D * 18.0, "add_rms_norm (2 branches)" + tag, t_like, rows * D * 18.0, "bytes")
+        lr = lg[:rows]
+        t_like = _time(lambda: ops.output_norm_join(x, 1e-5, routed=(yp, p, top, s2, lr[:, E]), post=(w, w1), x_out=x, h_out=h), flush)
+        t_new = _time(lambda: ops.prenorm_join(x, w, 1e-5, routed=(yp, p, top, s2), x_out=x, h_out=h), flush)
+        rb = rows * D * (4.0 * (top + 1) + 10)
+        put("prenorm_join, routed sum" + tag, t_new, rb, "output_norm_join, routed" + tag, t_like, rb, "bytes")
+
+    # ---- convolution + norm over the whole projection + rotation + pages vs convolution + head norms + pages
+    C = (H + 2 * G) * hd
+    nblk = (B * ctx + T) // 16 + 8
+    proj = rnd(T, C)
+    kc, vc = rnd(nblk, G, 16, hd), rnd(nblk, G, 16, hd)
+    cw = rnd(taps, C, dt=f32, sc=0.5)
+    ring = torch.zeros(max(S, B), taps - 1, C, device=dev)
+    qn, kn, qj, kj = rnd(hd), rnd(hd), rnd(H * hd), rnd(G * hd)
+    freq = torch.tensor(RotarySpec(dims=hd, base=5e5).frequencies()[0], dtype=torch.float64, device=dev)
+    slots = i32(np.arange(T) + 16)
+    tile = ops.attn_prefill_tile(H, G)
+    ts_, tq_ = ops.build_prefill_tiles([L] * S, tile, [0] * S)
+    ts_d, tq_d = i32(ts_), i32(tq_)
+    q = torch.empty(T, H * hd, device=dev, dtype=bf)
+    table = ops.rot_table(i32(np.arange(T) % L), freq, torch.empty(T, hd // 2, 2, device=dev))
+    rot = dict(joint_norm=True, rot_dims=hd, half_layout=True, cos_sin=table)
+    for args, tag, work in (((proj, cu, ctx0, slot_s, ts_d, tq_d, S, 0, slots, q), "prefill", T * C * 4.0),
+                            ((proj[:B], cud, ctxd, slot_b, None, None, 0, B, slots[:B], q[:B]), "single rows", B * C * (4.0 + 4.0 * taps))):
+        pr_, cu_, cx_, sl_, a_, b_, n_p, n_s, so_, q_ = args
+        t_new = _time(lambda: ops.conv_attn_prep(pr_, cw, qj, kj, ring, cu_, cx_, sl_, a_, b_, tile, n_p, n_s, so_, q_, kc, vc, H, G, hd, hd,
+                                                 1e-5, **rot), flush)
+        t_like = _time(lambda: ops.conv_attn_prep(pr_, cw, qn, kn, ring, cu_, cx_, sl_, a_, b_, tile, n_p, n_s, so_, q_, kc, vc, H, G, hd, hd,
+                                                  1e-5), flush)
+        put(f"conv_attn_prep, joint norm + rotation ({tag})", t_new, work, f"conv_attn_prep, head norms ({tag})", t_like, work, "bytes")
+
+    # ---- attention: capped scores, an ordinary softmax vs one more in the denominator
+    nb = (L + 15) // 16
+    bt = i32(np.arange(S * nb).reshape(S, nb) + 1)
+    zero = torch.zeros(H, device=dev)
+    out = torch.empty(T, H * hd, device=dev, dtype=bf)
+    pf = lambda **k: ops.paged_attn_prefill_ex(q, H * hd, kc, vc, bt, cu, ctx0, ts_d, tq_d, out, H, G, hd, hd ** -0.5, softcap=cap, **k)   # noqa: E731
+    t_new, t_like = _time(lambda: pf(), flush), _time(lambda: pf(sink=zero), flush)
+    work = 4.0 * S * (L * L / 2) * H * hd
+    put("attention prefill, capped", t_new, work, "attention prefill, capped, plus one", t_like, work, "flops")
+    nbd = (ctx + 16) // 16
+    btd = i32(np.arange(B * nbd).reshape(B, nbd) % (nblk - 1) + 1)
+    lens = i32(np.full(B, ctx))
+    splits = ops.attn_decode_splits(B, G, ctx + 16)
+    ws = ops.attn_decode_workspace(B, H, hd, splits, dev)
+    outd, qB = torch.empty(B, H * hd, device=dev, dtype=bf), q[:B]
+    dc = lambda **k: ops.paged_attn_decode(qB, H * hd, kc, vc, btd, lens, outd, H, G, hd, hd ** -0.5, num_splits=splits, workspace=ws,   # noqa: E731
+                                           softcap=cap, **k)
+    t_new, t_like = _time(lambda: dc(), flush), _time(lambda: dc(sink=zero), flush)
+    kvb = B * ctx * G * hd * 4.0
+    put("attention decode, capped", t_new, kvb, "attention decode, capped, plus one", t_like, kvb, "bytes")
+
+    # ---- inputs of the recurrences: convolution + silu (+ unit norms) -> fp32 rows vs rotation -> fp32 rows
+    Cd, Cs = (2 * dg + dh) * dw, sh * sw + 2 * sg * sn
+    forms = (("delta", Cd, ((dg, dw, dw ** -0.5), (dg, dw, 1.0), (dh, dw, None))), ("state space", Cs, ((sh, sw, None), (sg, sn, None), (sg, sn, None))))
+    Hm = Cd // 3 // hd
+    prj = rnd(T, max(Cd, Cs, 3 * Hm * hd), sc=0.5)
+    rows32 = torch.empty(T, max(Cd, Cs, 3 * Hm * hd), device=dev)
+    posT = i32(np.arange(T) % L)
+    kcl = Hm * hd
+    t_rot, t_rot_b = (_time(lambda: ops.rot_prep(prj[:n], 0, kcl, 2 * kcl, posT[:n], None, rows32[:n], rows32[:n, kcl:], rows32[:n, 2 * kcl:], Hm, Hm,
+                                                 hd, hd, paged=False, rot_dims=hd, half_layout=True, freq=freq), flush) for n in (T, B))
+    for name, Cx, segs in forms:
+        cwx, bx = rnd(taps, Cx, dt=f32, sc=0.5), (None if name == "delta" else rnd(Cx, dt=f32))
+        rg = torch.zeros(max(S, B), taps - 1, Cx, device=dev)
+        t_new = _time(lambda: ops.conv_rec_prep(prj, cwx, bx, rg, cu, ctx0, slot_s, ts_d, tq_d, tile, S, 0, segs, rows32), flush)
+        put(f"conv_rec_prep, {name} (prefill)", t_new, T * Cx * 6.0, "rot_prep (fp32 out)", t_rot, T * 3 * kcl * 6.0, "bytes")
+        t_new = _time(lambda: ops.conv_rec_prep(prj[:B], cwx, bx, rg, cud, ctxd, slot_b, None, None, tile, 0, B, segs, rows32[:B]), flush)
+        put(f"conv_rec_prep, {name} (single rows)", t_new, B * Cx * (6.0 + 4.0 * taps), "rot_prep (fp32 out, single rows)", t_rot_b,
+            B * 3 * kcl * 6.0, "bytes")
+
+    # ---- the two scans vs linear attention with one decay per key channel and token (prefill, decode) at equal heads and widths
+    for name, h_, g_, k_, v_, delta in (("delta", dh, dg, dw, dw, True), ("state space", sh, sg, sn, sw, False)):
+        W = 2 * g_ * k_ + h_ * v_
+        x, gates = rnd(T, W, dt=f32, sc=0.1), rnd(T, 2 * h_, dt=f32)
+        rate, bias = torch.full((h_,), 0.3, device=dev), torch.full((h_,), -2.0, device=dev)
+        skip = None if delta else rnd(h_, dt=f32)
+        St, o = torch.zeros(max(S, B), h_, v_, k_, device=dev), torch.empty(T, h_ * v_, device=dev)
+        sc = lambda n, c, cx, sl, ml: ops.gated_scan(x[:n], 0, g_ * k_, 2 * g_ * k_, gates[:n], rate, bias, skip, c, cx, sl, St, o[:n], h_, g_, k_,   # noqa: E731
+                                                     v_, delta, max_len=ml)
+        xl, z = rnd(T, h_ * (2 * k_ + v_), dt=f32, sc=0.1), rnd(T, h_ * k_, dt=f32) + 2.0
+        dec = torch.full((h_,), 0.97, device=dev)
+        gl = lambda n, c, cx, sl, ml: ops.gla_scan(xl[:n], 0, h_ * k_, 2 * h_ * k_, z[:n], 1 / 16, c, cx, sl, St, o[:n], h_, k_, v_, max_len=ml)   # noqa: E731
+        ln = lambda n, c, cx, sl, ml: ops.linattn_scan(xl[:n], 0, h_ * k_, 2 * h_ * k_, dec, c, cx, sl, St, o[:n], h_, k_, v_, max_len=ml)   # noqa: E731
+        t_new = _time(lambda: sc(T, cu, ctx0, slot_s, L), flush, iters=5, warm=2)
+        wn, wl = (6.0 if delta else 4.0) * T * h_ * k_ * v_, 4.0 * T * h_ * k_ * v_
+        put(f"gated_scan, {name} (prefill)", t_new, wn, "gla_scan (prefill)", _time(lambda: gl(T, cu, ctx0, slot_s, L), flush, iters=3, warm=1),
+            wl, "flops")
+        res[f"gated_scan, {name} (prefill)"]["fp32_tflops"] = round(wn / t_new / 1e12, 2)
+        put(f"gated_scan, {name} (prefill), vs fixed decay", t_new, wn, "linattn_scan (prefill, chunk)",
+            _time(lambda: ln(T, cu, ctx0, slot_s, L), flush, iters=3, warm=1), wl, "flops")
+        t_new, wb = _time(lambda: sc(B, cud, ctxd, slot_b, 1), flush), B * h_ * k_ * v_ * 8.0
+        put(f"gated_scan, {name} (decode)", t_new, wb, "gla_scan (decode)", _time(lambda: gl(B, cud, ctxd, slot_b, 1), flush), wb, "bytes")
+        put(f"gated_scan, {name} (decode), vs fixed decay", t_new, wb, "linattn_scan (decode)", _time(lambda: ln(B, cud, ctxd, slot_b, 1), flush),
+            wb, "bytes")
+        del x, gates, xl, z, St, o
+    # ---- gate before a grouped norm vs norm per head before a gate
+    Ci = sh * sw
+    o_raw, pz, mo, nw = rnd(T, Ci, dt=f32), rnd(T, 2 * Ci, sc=0.5), torch.empty(T, Ci, device=dev, dtype=bf), rnd(Ci)
+    for n, tag in ((T, ""), (B, " (single rows)")):
+        t_new = _time(lambda: ops.gate_norm(o_raw[:n], pz[:n], Ci, nw, mo[:n], sg, 1e-5), flush)
+        t_like = _time(lambda: ops.linattn_out(o_raw[:n], pz[:n], Ci, nw[:sw], mo[:n], sh, sw, 1e-5, False, "silu"), flush)
+        put("gate_norm" + tag, t_new, n * Ci * 8.0, "linattn_out" + tag, t_like, n * Ci * 8.0, "bytes")
+
+    # ---- routed SiLU experts chosen inside groups vs Danipel's clamped gated experts (both with their sum)
+    xin = rnd(T, D)
+    router = torch.zeros(128, D, device=dev, dtype=bf)
+    router[:E] = rnd(E, D, sc=0.05)
+    corr = rnd(E, dt=f32, sc=0.01)
+    w13, w2 = rnd(E * 2 * ffe, D, sc=0.02), rnd(E * D, ffe, sc=0.02)
+    for rows, tag in ((T, "prefill"), (B, "decode")):
+        rws = ops.RoutedWorkspace(rows, top, E, D, ffe, bf, dev)
+        xr, yo, hr = xin[:rows], y32[:rows], xb[:rows]
+
+        def new():
+            ops.routed_experts(xr, router, corr, w13, w2, rws, None, E, 0, top, 2.0, ffe, 0.0, act="silu", renormalize=False, combine=False,
+                               groups=groups, groups_keep=keep)
+            ops.prenorm_join(yo, w, 1e-5, routed=(rws.yp, rws.pair_row, top, None), x_out=yo, h_out=hr)
+
+        t_new = _time(new, flush, iters=5, warm=2)
+        t_like = _time(lambda: ops.routed_experts(xr, router, corr, w13, w2, rws, yo, E, 0, top, 1.0, ffe, 7.0), flush, iters=5, warm=2)
+        wf = 6.0 * rows * top * D * ffe
+        put(f"routed SiLU experts in groups + join ({tag})", t_new, wf, f"routed clamped experts, Danipel ({tag})", t_like, wf, "flops")
+        if tag == "decode":      # every expert's weights are read once: the bound of a small batch
+            wbytes = E * 3.0 * D * ffe * 2
+            put("routed SiLU experts (decode, weight bytes)", t_new, wbytes, "routed clamped experts, Danipel (decode)", t_like, wbytes, "bytes")
+        del rws
+    # ---- the fp32 gate projection beside a router's product (both one short fp32-output GEMM over the same rows)
+    gw, go, ro = rnd(2 * dh, D, sc=0.02), torch.empty(T, 2 * dh, device=dev), torch.empty(T, 128, device=dev)
+    for n, tag in ((T, "prefill"), (B, "decode")):
+        t_new, t_like = _time(lambda: ops.linear(xin[:n], gw, go[:n]), flush), _time(lambda: ops.linear(xin[:n], router, ro[:n]), flush)
+        put(f"gate projection, fp32 out ({tag})", t_new, n * D * 2.0, f"router product ({tag})", t_like, n * D * 2.0, "bytes")
+    return res
+
+
 FAMILIES = {"vodavik": (vodavik_config, _kernel_numbers), "danipel": (danipel_config, _kernel_numbers_danipel),
             "resevik": (resevik_config, _kernel_numbers_resevik), "dotorax": (dotorax_config, _kernel_numbers_dotorax),
-            "kerarax": (kerarax_config, _kernel_numbers_kerarax)}
-# a family whose closest existing model is another layer-list design is measured beside that one too
-CLOSEST = {"resevik": ("vodavik", vodavik_config), "dotorax": ("resevik", resevik_config),
-           "kerarax": ("danipel", danipel_config)}
+            "kerarax": (kerarax_config, _kernel_numbers_kerarax), "bovitar": (bovitar_config, _kernel_numbers_bovitar)}
+# a family whose closest existing models are other layer-list designs is measured beside those too
+CLOSEST = {"resevik": [("vodavik", vodavik_config)], "dotorax": [("resevik", resevik_config)],
+           "kerarax": [("danipel", danipel_config)], "bovitar": [("kerarax", kerarax_config), ("dotorax", dotorax_config)]}
 
 
 def run(sizes=("2k", "4k"), seqs=4, prompt=2048, batch=64, decode_steps=32, log=None, family="vodavik"):
@@ -1043,8 +1243,7 @@ def run(sizes=("2k", "4k"), seqs=4, prompt=2048, batch=64, decode_steps=32, log=
         log(f"size {size}: {SIZES[size]}")
         o = {"model": {}, "kernels": {}}
         models = [(family, make(size)), ("llama", llama_config(size))]
-        if family in CLOSEST:
-            models.insert(1, (CLOSEST[family][0], CLOSEST[family][1](size)))
+        models[1:1] = [(name, cfg(size)) for name, cfg in CLOSEST.get(family, [])]
         for name, cfg in models:
             o["model"][name] = _model_numbers(cfg, seqs, prompt, batch, decode_steps, log)
         o["kernels"] = kernels(size, seqs * prompt, batch, prompt, log)

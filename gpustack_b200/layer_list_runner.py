@@ -144,6 +144,8 @@ class LayerListRunner(ModelRunner):
         self.q_rows_width = max([m.heads * m.cache_widths(bf)[0] for _, m in conv] or [0])
         self.mix_width = max([self.mix_width] + [m.heads * m.cache_widths(bf)[1] + self._right_width(cfg.layers[l].mixer)
                                                  for l, m in conv])
+        # rotations of such mixers read cos / sin from a table per distinct set of frequencies
+        self.rot_key = {l: (m.rot.dims, tuple(m.rot.frequencies()[0])) for l, m in conv if m.rot is not None}
         self.o_padded = {l: pad_head_columns(self.w.layers[l].o, m.heads, m.vdim, m.cache_widths(bf)[1]) for l, m in conv
                          if m.cache_widths(bf)[1] != m.vdim and cfg.layers[l].weights_of is None}
         for l, x in enumerate(cfg.layers):               # (a layer that uses another's tensors uses its padded copy too)
@@ -204,6 +206,7 @@ class LayerListRunner(ModelRunner):
         if self.parallel:
             self.y2 = e(T, D, dt=torch.float32)           # the feed-forward's output beside the mixer's (self.y)
             self.emb32 = e(T, D, dt=torch.float32) if self.looped else None   # the embedding output, added again per pass
+        self.rot_tables = {key: (self.w.layers[l].rot_freq, e(T * key[0], dt=torch.float32)) for l, key in self.rot_key.items()}
         self._pending = (None, None)                      # branch outputs not yet summed into the residual
         self.lat_q = e(T * max(1, self.lat_q_width), dt=a)        # queries of a mixer whose queries have a latent
         self.lat_cq = e(T * max(1, self.lat_q_rank), dt=a)        # the normed query latent
@@ -455,6 +458,10 @@ class LayerListRunner(ModelRunner):
         rows (lens_d / bt_d).  cu_all / ctx_all / slots_all list both kinds for the recurrent scan."""
         cfg, eps = self.mcfg, self.mcfg.norm_eps
         pos, slots = self._pos, self._slots
+        self._angles = {}
+        for key, (freq, buf) in self.rot_tables.items():     # once per step for all layers with the same frequencies
+            self._angles[key] = ops.rot_table(pos[:T], freq, buf[:T * freq.shape[0] * 2].view(T, freq.shape[0], 2))
+            self.stats["kernel_launches"] += 1
         for l, (li, again) in enumerate(self.runs):      # l indexes the run (caches, state), li the layer (weights)
             layer, lw = cfg.layers[li], self.w.layers[li]
             m = layer.mixer
@@ -591,7 +598,8 @@ class LayerListRunner(ModelRunner):
         ops.conv_attn_prep(proj, lw.conv_w, lw.q_norm, lw.k_norm, ring, cu_all, ctx_all, slots_all, ts, tq, self.prefill_tile,
                            cu_p.shape[0] - 1 if nt else 0, Bd, self._slots, q, self.k_cache[l], self.v_cache[l], m.heads, m.kv_heads,
                            m.dim, m.vdim, self.mcfg.norm_eps, joint_norm=m.qk_norm_joint, rot_dims=m.rot.dims if m.rot is not None else 0,
-                           half_layout=m.rot is not None and m.rot.layout == "half", freq=lw.rot_freq)
+                           half_layout=m.rot is not None and m.rot.layout == "half",
+                           cos_sin=None if m.rot is None else self._angles[self.rot_key[self.runs[l][0]]])
 
     def _attend(self, l, m, lw, q, proj, gate_col, out, T, Tp, Bd, nt, bt_p, cu_p, ctx_p, ts, tq, lens_d, bt_d, dk, dv) -> None:
         """Attention of prepared queries over the run's pages (heads laid out dk / dv wide): prompt portions, then single rows."""

@@ -179,6 +179,7 @@ SIGNATURES = {
                                    _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _vp]),
     "b200_conv_attn_prep_ex": (_i32, [_vp, _i32, _i64, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _vp,
                                       _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _i32, _i32, _i32, _vp, _vp]),
+    "b200_rot_table": (_i32, [_vp, _vp, _vp, _i32, _i32, _vp]),
     "b200_conv_rec_prep": (_i32, [_vp, _i32, _i64, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _vp, _vp, _vp,
                                   _vp, _vp, _i64, _f32, _vp]),
     "b200_gated_scan": (_i32, [_vp, _i64, _i32, _i32, _i32, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32,

@@ -833,15 +833,17 @@ def output_norm_join(x_in, eps: float, y=None, routed=None, post=None, final=Non
 
 def conv_attn_prep(proj, conv_w, q_norm, k_norm, ring, cu_seq, ctx_lens, state_slots, tile_seq, tile_q0, tile_rows: int,
                    n_prompt: int, n_single: int, slots, q_out, k_cache, v_cache, H, G, dk, dv, eps: float, joint_norm: bool = False,
-                   rot_dims: int = 0, half_layout: bool = False, freq=None):
+                   rot_dims: int = 0, half_layout: bool = False, cos_sin=None):
     """Short causal convolution of the projected rows [q | k | v] with per-sequence rings of earlier inputs, per-head norms,
     queries to q_out [T, H * wk], keys and values to their pages (csrc/conv_attn_prep.cu).  conv_w fp32 [taps, C] (last row:
     the current token); ring fp32 [slots, taps - 1, C] (None with one tap); the sequences are n_prompt prompt portions (covered by the row
     tiles) and then n_single single rows; page widths wk >= dk and wv >= dv come from the caches.  joint_norm: q and k are
-    normed over the whole projection (weights of that size); rot_dims > 0: rotation of every q / k head after the norm."""
-    _cuda(proj, conv_w, q_norm, k_norm, ring, cu_seq, ctx_lens, state_slots, tile_seq, tile_q0, slots, q_out, k_cache, v_cache, freq)
-    if freq is not None:
-        _req(freq, torch.float64, "freq")
+    normed over the whole projection (weights of that size); rot_dims > 0: rotation of every q / k head after the norm by the
+    angles in cos_sin (rot_table of the step's rows)."""
+    _cuda(proj, conv_w, q_norm, k_norm, ring, cu_seq, ctx_lens, state_slots, tile_seq, tile_q0, slots, q_out, k_cache, v_cache, cos_sin)
+    if rot_dims and (cos_sin is None or cos_sin.dtype != torch.float32 or not cos_sin.is_contiguous()
+                     or cos_sin.shape[0] < proj.shape[0] or tuple(cos_sin.shape[1:]) != (rot_dims // 2, 2)):
+        raise B200Error("conv_attn_prep: cos_sin fp32 [rows, rot_dims / 2, 2]")
     if joint_norm and (q_norm.numel() != H * dk or k_norm.numel() != G * dk):
         raise B200Error("conv_attn_prep: the joint norm has one weight per channel of the projection")
     _req(conv_w, torch.float32, "conv_w")
@@ -859,8 +861,16 @@ def conv_attn_prep(proj, conv_w, q_norm, k_norm, ring, cu_seq, ctx_lens, state_s
     check(load().b200_conv_attn_prep_ex(_p(proj), _is_f32(proj), proj.stride(0), _p(conv_w), taps, _p(q_norm), _p(k_norm), _p(ring),
                                         _p(cu_seq), _p(ctx_lens), _p(state_slots), _p(tile_seq), _p(tile_q0), n_tiles, tile_rows,
                                         n_prompt, n_single, _p(slots), _p(q_out), _p(k_cache), _p(v_cache), H, G, dk, dv, wk, wv,
-                                        k_cache.shape[2], eps, 1 if joint_norm else 0, rot_dims, 1 if half_layout else 0, _p(freq),
+                                        k_cache.shape[2], eps, 1 if joint_norm else 0, rot_dims, 1 if half_layout else 0, _p(cos_sin),
                                         _stream()), "conv_attn_prep")
+
+
+def rot_table(positions, freq, out):
+    """(cos, sin) of positions[t] * freq[i] -> out fp32 [T, len(freq), 2]; angles formed and reduced in fp64."""
+    _cuda(positions, freq, out)
+    _req(positions, torch.int32, "positions"); _req(freq, torch.float64, "freq"); _req(out, torch.float32, "out")
+    check(load().b200_rot_table(_p(positions), _p(freq), _p(out), positions.shape[0], freq.shape[0], _stream()), "rot_table")
+    return out
 
 
 # ------------------------------------------- recurrences with one decay per head and token, pre-norm joins

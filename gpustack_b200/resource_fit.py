@@ -52,6 +52,7 @@ def _layer_list_workspace(m, e: EngineConfig) -> int:
     T, S, D = max(e.max_num_batched_tokens, e.max_num_seqs), e.max_num_seqs, m.hidden_size
     a = 4 if e.dtype == "float32" else 2
     proj = mix = ff = gates = rec = lat = routed = lin = 0
+    angles = set()
     for l in m.layers:
         x = l.mixer
         if x.kind == "attention":
@@ -66,6 +67,7 @@ def _layer_list_workspace(m, e: EngineConfig) -> int:
             proj = max(proj, y.qkv_width + r.proj_rows + 7)
             lat, mix = max(lat, y.heads * wk), max(mix, y.heads * wv + r.out_width)
             gates, rec, lin = max(gates, r.heads, y.heads), max(rec, r.out_width), max(lin, r.row_width)
+            angles.add((y.rot.dims, y.rot.base))
         elif x.kind == "delta":
             proj = max(proj, x.proj_rows + 7)
             gates, rec, lin = max(gates, 2 * x.heads), max(rec, x.out_width), max(lin, x.row_width)
@@ -97,6 +99,7 @@ def _layer_list_workspace(m, e: EngineConfig) -> int:
     par = 4 * (1 + (1 if m.loop_times > 1 else 0)) if m.residual == "parallel" else 0    # second branch output, embedding copy
     if m.residual == "pre_norm":
         par = 4                                                                          # second output
+        routed += T * 4 * sum(dims for dims, _ in angles)                                # cos / sin tables
     if m.residual == "sandwich":
         par = 8                                                                          # second output, normed input (fp32)
         routed += 8 * (T // 64 + S + 1) * max([x.mixer.right.width for x in m.layers if x.mixer.kind == "side_by_side"] or [0])

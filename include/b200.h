@@ -560,14 +560,15 @@ int b200_conv_attn_prep(const void* proj, int f32, int64_t ld, const float* conv
                         int tile_rows, int n_prompt, int n_single, const int32_t* slots, void* q_out, void* k_cache,
                         void* v_cache, int H, int G, int dk, int dv, int wk, int wv, int page, float eps, void* stream);
 /* The same with a q / k norm over the whole projection (joint_norm: weights of H dk / G dk entries) and a rotation of the
- * first rot_dims entries of every q / k head by position * freq[i] after the norm (half_layout: pairs (i, i + rot_dims/2),
- * else (2i, 2i + 1)). */
+ * first rot_dims entries of every q / k head after the norm (half_layout: pairs (i, i + rot_dims/2), else (2i, 2i + 1)) by the
+ * angles whose (cos, sin) are cos_sin [rows][rot_dims / 2][2], as b200_rot_table fills it: position * freq[i]. */
+int b200_rot_table(const int32_t* positions, const double* freq, float* cos_sin, int T, int half, void* stream);
 int b200_conv_attn_prep_ex(const void* proj, int f32, int64_t ld, const float* conv_w, int taps, const void* qnorm_w,
                            const void* knorm_w, float* ring, const int32_t* cu_seq, const int32_t* ctx_lens,
                            const int32_t* state_slots, const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles,
                            int tile_rows, int n_prompt, int n_single, const int32_t* slots, void* q_out, void* k_cache,
                            void* v_cache, int H, int G, int dk, int dv, int wk, int wv, int page, float eps, int joint_norm,
-                           int rot_dims, int half_layout, const double* freq, void* stream);
+                           int rot_dims, int half_layout, const float* cos_sin, void* stream);
 /* Short causal convolution (+ bias), silu and an optional unit norm x / sqrt(sum(x^2) + eps) * factor per head of the
  * inputs of a recurrence: three segments of equal heads in neighbouring columns of proj, fp32 rows out with every head padded
  * by zeros to a multiple of 4 entries.  Rings, row tiles and single rows as above; seg_* are host arrays of three entries. */

@@ -225,7 +225,7 @@ def test_attention_inputs_normed_over_the_whole_projection_and_rotated(H, G, dk,
     cw = _rnd(taps, C, seed=1, scale=0.6)
     qn, kn = (_rnd(n * dk if joint else dk, seed=2 + n, dtype=BF) + 1 for n in (H, G))
     rot = {"dims": dims, "base": 300.0}
-    freq = torch.tensor(O.scaled_frequencies(rot), dtype=F64, device="cuda") if dims else None
+    freq = torch.tensor(O.scaled_frequencies(rot), dtype=F64, device="cuda")
     seqs = {n: _rnd(m, C, seed=14 + i).to(dtype) for i, (n, m) in enumerate(LENS.items())}
 
     def turn(x):
@@ -259,8 +259,10 @@ def test_attention_inputs_normed_over_the_whole_projection_and_rotated(H, G, dk,
         wide[:, :C] = rows.cuda()
         where = [tables[n][p // page] * page + p % page for n, m, p0 in step for p in range(p0, p0 + m)]
         qo = torch.full((rows.shape[0], H * wk), 5.0, dtype=dtype, device="cuda")
+        pos = _i32([p for _, m, p0 in step for p in range(p0, p0 + m)])
+        cs = ops.rot_table(pos, freq, torch.zeros(len(pos), dims // 2, 2, device="cuda")) if dims else None
         ops.conv_attn_prep(wide, cw.cuda(), qn.cuda(), kn.cuda(), ring, cu_d, ctx, slots, ts, tq, 32, n_p, n_s, _i32(where), qo, kc, vc, H, G,
-                           dk, dv, eps, joint_norm=joint, rot_dims=dims, half_layout=half, freq=freq)
+                           dk, dv, eps, joint_norm=joint, rot_dims=dims, half_layout=half, cos_sin=cs)
         for (n, m, _), o in zip(step, cu):
             got[n].append(qo[o:o + m].cpu())
     tol = 3e-6 if dtype == torch.float32 else 8e-3
@@ -290,9 +292,10 @@ def test_rotation_far_from_the_start(position):
     u = _rnd(1, (H + 2 * G) * dk, seed=1)
     one = torch.ones(H * dk, dtype=BF, device="cuda")
     q, kc, vc = torch.zeros(1, H * dk, device="cuda"), *(torch.zeros(1, G, 16, dk, device="cuda") for _ in range(2))
+    freq = torch.tensor(O.scaled_frequencies(rot), dtype=F64, device="cuda")
     ops.conv_attn_prep(u.cuda(), torch.ones(1, u.shape[1], device="cuda"), one, one[:G * dk], None, _i32([0, 1]), _i32([position]), _i32([0]), None,
                        None, 16, 0, 1, _i32([3]), q, kc, vc, H, G, dk, dk, 0.0, joint_norm=True, rot_dims=32, half_layout=True,
-                       freq=torch.tensor(O.scaled_frequencies(rot), dtype=F64, device="cuda"))
+                       cos_sin=ops.rot_table(_i32([position]), freq, torch.zeros(1, 16, 2, device="cuda")))
     x = O.rms(u[:, :H * dk].to(F64), 0.0).view(1, H, dk)
     assert _rel(q.view(1, H, dk), O.rotate_half(x, torch.tensor([position]), rot)) < 2e-6
 
