@@ -238,64 +238,84 @@ rot_table_kernel(const int32_t* __restrict__ positions, const double* __restrict
 }
 
 // The form with a rotation and / or a norm over the whole projection.  The head slots of a piece of rows are spread over the
-// CTAs of ONE cluster (along y); every thread keeps its window of inputs and weights in registers, convolves once for the sums
-// of squares, the CTAs exchange their partial sums through distributed shared memory (added in rank order), and a second
-// convolution from the same registers is scaled, rotated -- the partner of an entry sits dims / 2 further, in another lane
-// of the head's group, or beside it -- and stored.  No input is loaded twice.
-constexpr int kCapJointWarps = 6;    // per CTA: two CTAs per SM with the window and the weights in registers
+// CTAs of ONE cluster (along y).  A thread convolves its piece of a head once: values go straight to their pages, queries and
+// keys to shared memory in fp32 with their sums of squares; the CTAs exchange their partial sums through distributed shared
+// memory (added in rank order), and the staged rows are scaled, rotated -- the partner of an entry sits dims / 2 further, or
+// beside it -- and stored.
+constexpr int kCapJointWarps = 6;    // per CTA
 
 template <typename TA, int TAPS>
 __global__ void __launch_bounds__(kCapJointWarps * 32, 2)
 conv_attn_prep_joint_vec_kernel(CapArgs a, int lph) {
   constexpr int V = 16 / (int)sizeof(TA), R = TAPS - 1, NB = kCapRows;
-  extern __shared__ __align__(16) float2 cs[];         // [NB][dims / 2]
+  extern __shared__ __align__(16) float smem[];
   __shared__ float head_ss[kCapJointWarps * 32][NB], part[2][NB], mul[2][NB];
   const CapWork m = cap_work<NB>(a);
   if (m.n <= 0) return;                                // (the same for every CTA of the cluster)
   const int lane = threadIdx.x & 31, per_warp = 32 / lph, li = lane % lph, d = li * V, half = a.dims >> 1;
   const int in_cta = (threadIdx.x >> 5) * per_warp + lane / lph, cta_heads = (blockDim.x >> 5) * per_warp;
+  float2* cs = reinterpret_cast<float2*>(smem);        // [NB][dims / 2] (cos, sin)
+  float* ys = smem + NB * a.dims;                      // [NB][head slot][V / 4][lph][4] convolved queries and keys
   const int hs = blockIdx.y * cta_heads + in_cta;
   const bool live = hs < a.H + 2 * a.G, is_q = hs < a.H, is_k = !is_q && hs < a.H + a.G, qk = is_q || is_k;
   const int width = qk ? a.dk : a.dv, wide = qk ? a.wk : a.wv;
-  const int C = (a.H + a.G) * a.dk + a.G * a.dv;
-  const int c = (qk ? hs * a.dk : (a.H + a.G) * a.dk + (hs - a.H - a.G) * a.dv) + d;
   const bool act = live && d < width, pad = live && !act && d < wide;
   const bool norm = a.qnorm_w != nullptr;
-  const TA* src = reinterpret_cast<const TA*>(a.proj) + (size_t)m.row0 * a.ld + c;
-  uint4 win[R + NB];
-  float w[TAPS][V];
-  if (act) {
-    conv_window<TA, TAPS, NB>(win, m, src, a.ld, a.ring, c, C);
-    conv_weights<TAPS, V>(w, a.conv_w, c, C);
-    conv_ring_put<TA, TAPS>(m, src, a.ld, a.ring, c, C);
-  }
+  const int32_t* slots = a.slots + m.row0 + m.q0;
+  const int g = is_k ? hs - a.H : hs - a.H - a.G;
   const float2* table = a.cs + (size_t)(m.row0 + m.q0) * half;
   for (int i = threadIdx.x; i < m.n * half; i += blockDim.x) cs[i] = table[i];
-  auto row_ss = [&](int r) {                           // sum of squares of the head's convolved row, in all its lanes
-    float y[V], ss = 0.f;
-#pragma unroll
-    for (int i = 0; i < V; ++i) y[i] = 0.f;
-    if (act) conv_row<TA, TAPS, NB>(win, r, w, y);
-#pragma unroll
-    for (int i = 0; i < V; ++i) ss = fmaf(y[i], y[i], ss);
-    for (int o = lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    return ss;
-  };
-  cg::cluster_group cluster = cg::this_cluster();
-  if (a.joint && norm) {
+  {
+    const int C = (a.H + a.G) * a.dk + a.G * a.dv;
+    const int c = (qk ? hs * a.dk : (a.H + a.G) * a.dk + (hs - a.H - a.G) * a.dv) + d;
+    const TA* src = reinterpret_cast<const TA*>(a.proj) + (size_t)m.row0 * a.ld + c;
+    uint4 win[R + NB];
+    float w[TAPS][V];
+    if (act) {
+      conv_window<TA, TAPS, NB>(win, m, src, a.ld, a.ring, c, C);
+      conv_weights<TAPS, V>(w, a.conv_w, c, C);
+      conv_ring_put<TA, TAPS>(m, src, a.ld, a.ring, c, C);
+    }
 #pragma unroll
     for (int r = 0; r < NB; ++r) {
-      const float ss = row_ss(r);                      // (rows behind the portion are zeros)
-      if (li == 0) head_ss[in_cta][r] = ss;
+      if (r >= m.n) break;
+      float y[V], ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < V; ++i) y[i] = 0.f;
+      if (act) conv_row<TA, TAPS, NB>(win, r, w, y);
+      if (qk) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss = fmaf(y[i], y[i], ss);
+#pragma unroll
+        for (int i = 0; i < V; i += 4)
+          *reinterpret_cast<float4*>(ys + (((size_t)r * cta_heads + in_cta) * (V / 4) + i / 4) * lph * 4 + li * 4) =
+              make_float4(y[i], y[i + 1], y[i + 2], y[i + 3]);
+      } else if (act || pad) {
+        const int slot = slots[r];
+        uint4 outv;
+        TA* ov = reinterpret_cast<TA*>(&outv);
+#pragma unroll
+        for (int i = 0; i < V; ++i) ca_store(ov + i, y[i]);     // (zeros behind the head's own columns)
+        if (slot >= 0)
+          *reinterpret_cast<uint4*>(reinterpret_cast<TA*>(a.v_cache) + cap_cache_row(a, slot, g) * wide + d) = outv;
+      }
+      if (norm) {
+        for (int o = lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);    // all lanes take part
+        if (li == 0) head_ss[in_cta][r] = ss;
+      }
     }
-    __syncthreads();
+  }
+  __syncthreads();
+  if (a.joint && norm) {
     if (threadIdx.x < 2 * NB) {
       const int p = threadIdx.x / NB, r = threadIdx.x % NB;
       const int lo = p == 0 ? 0 : a.H, hi = p == 0 ? a.H : a.H + a.G, first = blockIdx.y * cta_heads;
       float v = 0.f;
-      for (int h = max(lo, first); h < min(hi, first + cta_heads); ++h) v += head_ss[h - first][r];
+      if (r < m.n)
+        for (int h = max(lo, first); h < min(hi, first + cta_heads); ++h) v += head_ss[h - first][r];
       part[p][r] = v;
     }
+    cg::cluster_group cluster = cg::this_cluster();
     cluster.sync();
     if (threadIdx.x < 2 * NB) {
       const int p = threadIdx.x / NB, r = threadIdx.x % NB;
@@ -303,62 +323,66 @@ conv_attn_prep_joint_vec_kernel(CapArgs a, int lph) {
       for (unsigned k = 0; k < gridDim.y; ++k) v += cluster.map_shared_rank(&part[0][0], k)[p * NB + r];
       mul[p][r] = 1.0f / sqrtf(v / (float)((p == 0 ? a.H : a.G) * a.dk) + a.eps);
     }
+    __syncthreads();
   }
-  __syncthreads();
-  float nw[V];
-  const bf16* nv = is_q ? a.qnorm_w : a.knorm_w;
+  if (qk && (act || pad)) {
+    float nw[V];
+    const bf16* nv = is_q ? a.qnorm_w : a.knorm_w;
 #pragma unroll
-  for (int i = 0; i < V; ++i)
-    nw[i] = act && norm && qk ? __bfloat162float(nv[(a.joint ? (is_q ? hs : hs - a.H) * a.dk : 0) + d + i]) : 1.0f;
-  const bool turn = act && qk && d < a.dims;            // (dims is a whole number of pieces)
-  const int partner = (turn && a.half_layout) ? (d < half ? lane + half / V : lane - half / V) : lane;
-  const int g = is_k ? hs - a.H : hs - a.H - a.G;
-  const int32_t* slots = a.slots + m.row0 + m.q0;
+    for (int i = 0; i < V; ++i)
+      nw[i] = act && norm ? __bfloat162float(nv[(a.joint ? (is_q ? hs : hs - a.H) * a.dk : 0) + d + i]) : 1.0f;
+    const bool turn = act && d < a.dims;                // (dims is a whole number of pieces)
+    const int other = (turn && a.half_layout) ? (d < half ? li + half / V : li - half / V) : li;
+    float ow[V];                                         // the partner's norm weights
 #pragma unroll
-  for (int r = 0; r < NB; ++r) {
-    if (r >= m.n) break;
-    float f = 1.0f;
-    if (norm && !a.joint) f = 1.0f / sqrtf(row_ss(r) / (float)a.dk + a.eps);      // (all lanes take part)
-    if (a.joint && qk) f = mul[is_q ? 0 : 1][r];
-    if (!qk) f = 1.0f;
-    float y[V];
+    for (int i = 0; i < V; ++i)
+      ow[i] = turn && norm ? __bfloat162float(nv[(a.joint ? (is_q ? hs : hs - a.H) * a.dk : 0) + other * V + i]) : 1.0f;
 #pragma unroll
-    for (int i = 0; i < V; ++i) y[i] = 0.f;
-    if (act) conv_row<TA, TAPS, NB>(win, r, w, y);
+    for (int r = 0; r < NB; ++r) {
+      if (r >= m.n) break;
+      float f = 1.0f;
+      if (norm) f = a.joint ? mul[is_q ? 0 : 1][r] : 1.0f / sqrtf(head_ss[in_cta][r] / (float)a.dk + a.eps);
+      float y[V], o[V];
+      const float* row = ys + ((size_t)r * cta_heads + in_cta) * V * lph;
 #pragma unroll
-    for (int i = 0; i < V; ++i) y[i] *= f * nw[i];
-    if (a.half_layout) {
-      float o[V];
-#pragma unroll
-      for (int i = 0; i < V; ++i) o[i] = __shfl_sync(0xffffffffu, y[i], partner);
-      if (turn) {
+      for (int i = 0; i < V; i += 4) {
+        const float4 t = *reinterpret_cast<const float4*>(row + (i / 4) * lph * 4 + li * 4);
+        y[i] = t.x * f * nw[i]; y[i + 1] = t.y * f * nw[i + 1]; y[i + 2] = t.z * f * nw[i + 2]; y[i + 3] = t.w * f * nw[i + 3];
+      }
+      if (turn && a.half_layout) {
         const float2* t = cs + r * half + (d < half ? d : d - half);
 #pragma unroll
-        for (int i = 0; i < V; ++i) y[i] = d < half ? y[i] * t[i].x - o[i] * t[i].y : y[i] * t[i].x + o[i] * t[i].y;
-      }
-    } else if (turn) {
-      const float2* t = cs + r * half + d / 2;
+        for (int i = 0; i < V; i += 4) {
+          const float4 t4 = *reinterpret_cast<const float4*>(row + (i / 4) * lph * 4 + other * 4);
+          o[i] = t4.x; o[i + 1] = t4.y; o[i + 2] = t4.z; o[i + 3] = t4.w;
+        }
 #pragma unroll
-      for (int i = 0; i < V; i += 2) {
-        const float u = y[i], v = y[i + 1];
-        y[i] = u * t[i / 2].x - v * t[i / 2].y;
-        y[i + 1] = v * t[i / 2].x + u * t[i / 2].y;
-      }
-    }
-    if (!act && !pad) continue;
-    uint4 outv;
-    TA* ov = reinterpret_cast<TA*>(&outv);
+        for (int i = 0; i < V; ++i) {
+          const float p = o[i] * f * ow[i];
+          y[i] = d < half ? y[i] * t[i].x - p * t[i].y : y[i] * t[i].x + p * t[i].y;
+        }
+      } else if (turn) {
+        const float2* t = cs + r * half + d / 2;
 #pragma unroll
-    for (int i = 0; i < V; ++i) ca_store(ov + i, y[i]);         // (zeros behind the head's own columns)
-    if (is_q) {
-      *reinterpret_cast<uint4*>(reinterpret_cast<TA*>(a.q_out) + ((size_t)(m.row0 + m.q0 + r) * a.H + hs) * a.wk + d) = outv;
-    } else {
-      const int slot = slots[r];
-      if (slot >= 0)
-        *reinterpret_cast<uint4*>(reinterpret_cast<TA*>(is_k ? a.k_cache : a.v_cache) + cap_cache_row(a, slot, g) * wide + d) = outv;
+        for (int i = 0; i < V; i += 2) {
+          const float u = y[i], v = y[i + 1];
+          y[i] = u * t[i / 2].x - v * t[i / 2].y;
+          y[i + 1] = v * t[i / 2].x + u * t[i / 2].y;
+        }
+      }
+      uint4 outv;
+      TA* ov = reinterpret_cast<TA*>(&outv);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ca_store(ov + i, y[i]);       // (zeros behind the head's own columns)
+      if (is_q) {
+        *reinterpret_cast<uint4*>(reinterpret_cast<TA*>(a.q_out) + ((size_t)(m.row0 + m.q0 + r) * a.H + hs) * a.wk + d) = outv;
+      } else {
+        const int slot = slots[r];
+        if (slot >= 0) *reinterpret_cast<uint4*>(reinterpret_cast<TA*>(a.k_cache) + cap_cache_row(a, slot, g) * wide + d) = outv;
+      }
     }
   }
-  if (a.joint && norm) cluster.sync();                  // nobody leaves while another CTA may still read its sums
+  if (a.joint && norm) cg::this_cluster().sync();       // nobody leaves while another CTA may still read its sums
 }
 
 // Any width, any number of taps: warps take the head slots in turn, lanes the columns; a head is staged in shared memory
@@ -496,10 +520,10 @@ extern "C" int b200_conv_attn_prep_ex(const void* proj, int f32, int64_t ld, con
     const int all_warps = lph <= 32 ? (n_heads + 32 / lph - 1) / (32 / lph) : 1 << 20;
     int ny = 1;
     while (ny < 8 && ny * kCapJointWarps < all_warps) ny <<= 1;
-    const size_t smem_v = sizeof(float2) * kCapRows * (size_t)(rot_dims / 2);
+    const int warps_v = (all_warps + ny - 1) / ny;
+    const size_t smem_v = sizeof(float) * kCapRows * ((size_t)rot_dims + (size_t)warps_v * 32 * vec);
     if (al && taps <= 4 && dk % vec == 0 && dv % vec == 0 && wk % vec == 0 && wv % vec == 0 && ld % vec == 0 && C % 4 == 0 &&
-        ny * kCapJointWarps >= all_warps && rot_dims % piece == 0 && smem_v <= 32 * 1024) {
-      const int warps = (all_warps + ny - 1) / ny;
+        ny * kCapJointWarps >= all_warps && rot_dims % piece == 0 && smem_v <= 100 * 1024) {
       cudaLaunchConfig_t cfg = {};
       cudaLaunchAttribute at[1];
       at[0].id = cudaLaunchAttributeClusterDimension;
@@ -507,13 +531,18 @@ extern "C" int b200_conv_attn_prep_ex(const void* proj, int f32, int64_t ld, con
       at[0].val.clusterDim.y = ny;
       at[0].val.clusterDim.z = 1;
       cfg.gridDim = dim3(n_x, ny);
-      cfg.blockDim = dim3(warps * 32);
+      cfg.blockDim = dim3(warps_v * 32);
       cfg.dynamicSmemBytes = smem_v;
       cfg.stream = s;
       cfg.attrs = at;
       cfg.numAttrs = 1;
       cudaError_t e = cudaSuccess;
-#define B200_CAJ(TA, N) e = cudaLaunchKernelEx(&cfg, conv_attn_prep_joint_vec_kernel<TA, N>, a, lph)
+#define B200_CAJ(TA, N)                                                                                                           \
+  do {                                                                                                                            \
+    if (smem_v > 40 * 1024)                                                                                                       \
+      e = cudaFuncSetAttribute(conv_attn_prep_joint_vec_kernel<TA, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);  \
+    if (e == cudaSuccess) e = cudaLaunchKernelEx(&cfg, conv_attn_prep_joint_vec_kernel<TA, N>, a, lph);                           \
+  } while (0)
 #define B200_CAJT(TA)                        \
   switch (taps) {                            \
     case 1: B200_CAJ(TA, 1); break;          \
