@@ -52,7 +52,7 @@ def cfg_odd():
     key head for all and one per head, one to six taps, rotated parts of a head, frequencies on all three branches, a layer
     without feed-forward, one without shared expert, layers that use another's tensors (before and after a third)."""
     sc = {"factor": 3.0, "low": 1.5, "high": 6.0, "original": 90}
-    L = [_parallel((3, 1, 10, 14, 3, 6, 1.1, 3.0, sc), (2, 7, 9, 1, 5, 1), _moe(6, 2, 18, 22, (3, 2), 1.7)), _delta(4, 2, 13, 6, 2, None),
+    L = [_parallel((3, 1, 10, 14, 3, 6, 1.1, 3.0, sc), (2, 7, 9, 1, 5, 1), _moe(6, 2, 18, 22, (3, 1), 1.7)), _delta(4, 2, 13, 6, 2, None),
          _parallel((4, 2, 6, 70, 1, 6, 0.4, 40.0, None), (6, 5, 33, 3, 2, 5), _moe(5, 3, 10, None)),
          _delta(3, 3, 70, 33, 6, _moe(4, 1, 9, 30, (4, 1), 0.6))]
     return {"architecture": "Bovitar", "vocab": 131, "width": 51, "norm": {"eps": 1e-5}, "logit_scale": 0.7,
@@ -86,7 +86,7 @@ def cfg_wide():
     """128-wide heads, as they are and padded from either side, in groups of four (tcgen05 prefill, split-KV decode) and
     of eight; caps on both sides of the bound that lets the softmax do without a running maximum."""
     sc = {"factor": 2.0, "low": 1.0, "high": 3.0, "original": 40}
-    L = [_parallel((8, 2, 128, 96, 4, 64, 0.09, 25.0, sc), (4, 64, 128, 1, 4, 2), _moe(4, 2, 256, 256)),
+    L = [_parallel((8, 2, 128, 96, 4, 64, 0.2, 25.0, sc), (4, 64, 128, 1, 4, 2), _moe(4, 2, 256, 256)),
          _parallel((8, 1, 96, 128, 3, 96, 0.1, 90.0, None), (2, 128, 64, 2, 3, 1), None), _delta(2, 2, 128, 128, 4, _moe(3, 1, 256, 64))]
     return {"architecture": "Bovitar", "vocab": 256, "width": 256, "norm": {"eps": 1e-5}, "logit_scale": 0.3,
             "layers": [L[0], L[1], L[2], _same(L[0], 0)]}
