@@ -15,16 +15,12 @@
 // (8 rows and the taps - 1 before them) at once and walk the rows in registers.  Only a sequence's first
 // piece can need the ring (a piece is longer than the ring), and the SAME threads that read it there write the step's
 // last inputs into it after their reads: no second launch, no race.  The statistics and the convolution are fp32.
-#include <cooperative_groups.h>
-
 #include "common.cuh"
 #include "conv_prep.cuh"
 #include "runtime.h"
 #include "../../include/b200.h"
 
 namespace b200 {
-
-namespace cg = cooperative_groups;
 
 struct CapArgs {
   const void* proj;
@@ -237,152 +233,203 @@ rot_table_kernel(const int32_t* __restrict__ positions, const double* __restrict
   out[i] = make_float2(c, sn);
 }
 
-// The form with a rotation and / or a norm over the whole projection.  The head slots of a piece of rows are spread over the
-// CTAs of ONE cluster (along y).  A thread convolves its piece of a head once: values go straight to their pages, queries and
-// keys to shared memory in fp32 with their sums of squares; the CTAs exchange their partial sums through distributed shared
-// memory (added in rank order), and the staged rows are scaled, rotated -- the partner of an entry sits dims / 2 further, or
-// beside it -- and stored.
-constexpr int kCapJointWarps = 6;    // per CTA
+// The form with a rotation and / or a norm over the whole projection.  ONE CTA owns all channels of a run of rows (the joint
+// statistic is a sum over the CTA) and walks it two rows at a time; a thread owns one 16-byte piece of a head for the whole
+// run, its weights in registers, its inputs in a private ring of eight rows in shared memory that cp.async fills two steps
+// ahead.  Per step: convolve, sum the squares over the head's lanes, one barrier, sum over the heads (the same order in every
+// warp), scale, rotate -- the partner of an entry sits dims / 2 further, in another lane of the head's group, or beside it --
+// and store.
+constexpr int kCapRun = 16, kCapJointWarps = 24, kCapSlots = 8;
 
 template <typename TA, int TAPS>
-__global__ void __launch_bounds__(kCapJointWarps * 32, 2)
+__global__ void __launch_bounds__(kCapJointWarps * 32, 1)
 conv_attn_prep_joint_vec_kernel(CapArgs a, int lph) {
-  constexpr int V = 16 / (int)sizeof(TA), R = TAPS - 1, NB = kCapRows;
-  extern __shared__ __align__(16) float smem[];
-  __shared__ float head_ss[kCapJointWarps * 32][NB], part[2][NB], mul[2][NB];
-  const CapWork m = cap_work<NB>(a);
-  if (m.n <= 0) return;                                // (the same for every CTA of the cluster)
+  constexpr int V = 16 / (int)sizeof(TA), R = TAPS - 1, RR = R > 0 ? R : 1;
+  static_assert(R + 2 + 3 <= kCapSlots, "a step's rows, the ones before and the ones in flight have slots of their own");
+  extern __shared__ __align__(16) uint4 raw[];         // [8][threads]
+  __shared__ float head_ss[2][2][kCapJointWarps * 32]; // [step parity][row][head slot]
+  const CapWork m = cap_work<kCapRun>(a);
+  if (m.n <= 0) return;
   const int lane = threadIdx.x & 31, per_warp = 32 / lph, li = lane % lph, d = li * V, half = a.dims >> 1;
-  const int in_cta = (threadIdx.x >> 5) * per_warp + lane / lph, cta_heads = (blockDim.x >> 5) * per_warp;
-  float2* cs = reinterpret_cast<float2*>(smem);        // [NB][dims / 2] (cos, sin)
-  float* ys = smem + NB * a.dims;                      // [NB][head slot][V / 4][lph][4] convolved queries and keys
-  const int hs = blockIdx.y * cta_heads + in_cta;
+  const int hs = (threadIdx.x >> 5) * per_warp + lane / lph;
   const bool live = hs < a.H + 2 * a.G, is_q = hs < a.H, is_k = !is_q && hs < a.H + a.G, qk = is_q || is_k;
   const int width = qk ? a.dk : a.dv, wide = qk ? a.wk : a.wv;
   const bool act = live && d < width, pad = live && !act && d < wide;
   const bool norm = a.qnorm_w != nullptr;
-  const int32_t* slots = a.slots + m.row0 + m.q0;
+  const int C = (a.H + a.G) * a.dk + a.G * a.dv;
+  const int c = (qk ? hs * a.dk : (a.H + a.G) * a.dk + (hs - a.H - a.G) * a.dv) + d;
+  const TA* src = reinterpret_cast<const TA*>(a.proj) + (size_t)m.row0 * a.ld + c;
+  const uint4 zero4 = make_uint4(0, 0, 0, 0);
+  uint4* mine = raw + threadIdx.x;
+  auto at = [&](int r) -> uint4* { return mine + ((r + kCapSlots) & (kCapSlots - 1)) * blockDim.x; };      // row r of the run, r >= -R
+  auto fetch = [&](int r) {                            // (rows behind the run: zeros)
+    if (act && r < m.n)
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((unsigned)__cvta_generic_to_shared(at(r))),
+                   "l"(src + (int64_t)(m.q0 + r) * a.ld) : "memory");
+    else
+      *at(r) = zero4;
+  };
+  auto commit = [] { asm volatile("cp.async.commit_group;" ::: "memory"); };
+  if constexpr (R > 0)
+#pragma unroll
+  for (int b = 0; b < R; ++b) {                        // the rows before the run
+    const int q = m.q0 - 1 - b, p = m.ctx + q;
+    uint4 x = zero4;
+    if (act && q >= 0) {
+      x = *reinterpret_cast<const uint4*>(src + (int64_t)q * a.ld);
+    } else if (act && p >= 0 && m.slot >= 0) {
+      const float* rp = a.ring + ((size_t)m.slot * R + p % RR) * C + c;
+      TA* xv = reinterpret_cast<TA*>(&x);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ca_store(xv + i, rp[i]);
+    }
+    *at(-1 - b) = x;
+  }
+  fetch(0);
+  fetch(1);
+  commit();
+  fetch(2);
+  fetch(3);
+  commit();
+  float w[TAPS][V];
+  uint4 nraw = zero4;                                  // norm weights, bf16 (V of them)
+  if (act) {
+    conv_weights<TAPS, V>(w, a.conv_w, c, C);
+    conv_ring_put<TA, TAPS>(m, src, a.ld, a.ring, c, C);
+    if (norm && qk) {
+      const bf16* nv = (is_q ? a.qnorm_w : a.knorm_w) + (a.joint ? (is_q ? hs : hs - a.H) * a.dk : 0) + d;
+      bf16* nr = reinterpret_cast<bf16*>(&nraw);
+#pragma unroll
+      for (int i = 0; i < V; ++i) nr[i] = nv[i];
+    }
+  }
+  const bool turn = act && qk && d < a.dims;            // (dims is a whole number of pieces)
+  const int partner = (turn && a.half_layout) ? (d < half ? lane + half / V : lane - half / V) : lane;
   const int g = is_k ? hs - a.H : hs - a.H - a.G;
-  const float2* table = a.cs + (size_t)(m.row0 + m.q0) * half;
-  for (int i = threadIdx.x; i < m.n * half; i += blockDim.x) cs[i] = table[i];
-  {
-    const int C = (a.H + a.G) * a.dk + a.G * a.dv;
-    const int c = (qk ? hs * a.dk : (a.H + a.G) * a.dk + (hs - a.H - a.G) * a.dv) + d;
-    const TA* src = reinterpret_cast<const TA*>(a.proj) + (size_t)m.row0 * a.ld + c;
-    uint4 win[R + NB];
-    float w[TAPS][V];
+  const int row0 = m.row0 + m.q0;
+  const float2* table = a.cs + (size_t)row0 * half + (a.half_layout ? (d < half ? d : d - half) : d / 2);
+  const bool warp_q = (threadIdx.x >> 5) * per_warp < a.H;                                   // the warp holds query heads
+  const bool warp_k = ((threadIdx.x >> 5) + 1) * per_warp > a.H && (threadIdx.x >> 5) * per_warp < a.H + a.G;
+  const float inv_q = 1.0f / (float)(a.H * a.dk), inv_k = 1.0f / (float)(a.G * a.dk), inv_dk = 1.0f / (float)a.dk;
+  const float sgn = d < half ? -1.0f : 1.0f;
+  TA* q_dst = reinterpret_cast<TA*>(a.q_out) + ((size_t)row0 * a.H + hs) * a.wk + d;
+  TA* const kv_dst = reinterpret_cast<TA*>(is_k ? a.k_cache : a.v_cache) + d;
+  for (int r0 = 0; r0 < m.n; r0 += 2) {
+    asm volatile("cp.async.wait_group 1;" ::: "memory");       // (a thread reads only what it fetched itself)
+    float y[2][V], f[2] = {1.0f, 1.0f};
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+#pragma unroll
+      for (int i = 0; i < V; ++i) y[r][i] = 0.f;
     if (act) {
-      conv_window<TA, TAPS, NB>(win, m, src, a.ld, a.ring, c, C);
-      conv_weights<TAPS, V>(w, a.conv_w, c, C);
-      conv_ring_put<TA, TAPS>(m, src, a.ld, a.ring, c, C);
-    }
 #pragma unroll
-    for (int r = 0; r < NB; ++r) {
-      if (r >= m.n) break;
-      float y[V], ss = 0.f;
-#pragma unroll
-      for (int i = 0; i < V; ++i) y[i] = 0.f;
-      if (act) conv_row<TA, TAPS, NB>(win, r, w, y);
-      if (qk) {
-#pragma unroll
-        for (int i = 0; i < V; ++i) ss = fmaf(y[i], y[i], ss);
-#pragma unroll
-        for (int i = 0; i < V; i += 4)
-          *reinterpret_cast<float4*>(ys + (((size_t)r * cta_heads + in_cta) * (V / 4) + i / 4) * lph * 4 + li * 4) =
-              make_float4(y[i], y[i + 1], y[i + 2], y[i + 3]);
-      } else if (act || pad) {
-        const int slot = slots[r];
-        uint4 outv;
-        TA* ov = reinterpret_cast<TA*>(&outv);
-#pragma unroll
-        for (int i = 0; i < V; ++i) ca_store(ov + i, y[i]);     // (zeros behind the head's own columns)
-        if (slot >= 0)
-          *reinterpret_cast<uint4*>(reinterpret_cast<TA*>(a.v_cache) + cap_cache_row(a, slot, g) * wide + d) = outv;
-      }
-      if (norm) {
-        for (int o = lph >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);    // all lanes take part
-        if (li == 0) head_ss[in_cta][r] = ss;
-      }
-    }
-  }
-  __syncthreads();
-  if (a.joint && norm) {
-    if (threadIdx.x < 2 * NB) {
-      const int p = threadIdx.x / NB, r = threadIdx.x % NB;
-      const int lo = p == 0 ? 0 : a.H, hi = p == 0 ? a.H : a.H + a.G, first = blockIdx.y * cta_heads;
-      float v = 0.f;
-      if (r < m.n)
-        for (int h = max(lo, first); h < min(hi, first + cta_heads); ++h) v += head_ss[h - first][r];
-      part[p][r] = v;
-    }
-    cg::cluster_group cluster = cg::this_cluster();
-    cluster.sync();
-    if (threadIdx.x < 2 * NB) {
-      const int p = threadIdx.x / NB, r = threadIdx.x % NB;
-      float v = 0.f;
-      for (unsigned k = 0; k < gridDim.y; ++k) v += cluster.map_shared_rank(&part[0][0], k)[p * NB + r];
-      mul[p][r] = 1.0f / sqrtf(v / (float)((p == 0 ? a.H : a.G) * a.dk) + a.eps);
-    }
-    __syncthreads();
-  }
-  if (qk && (act || pad)) {
-    float nw[V];
-    const bf16* nv = is_q ? a.qnorm_w : a.knorm_w;
-#pragma unroll
-    for (int i = 0; i < V; ++i)
-      nw[i] = act && norm ? __bfloat162float(nv[(a.joint ? (is_q ? hs : hs - a.H) * a.dk : 0) + d + i]) : 1.0f;
-    const bool turn = act && d < a.dims;                // (dims is a whole number of pieces)
-    const int other = (turn && a.half_layout) ? (d < half ? li + half / V : li - half / V) : li;
-    float ow[V];                                         // the partner's norm weights
-#pragma unroll
-    for (int i = 0; i < V; ++i)
-      ow[i] = turn && norm ? __bfloat162float(nv[(a.joint ? (is_q ? hs : hs - a.H) * a.dk : 0) + other * V + i]) : 1.0f;
-#pragma unroll
-    for (int r = 0; r < NB; ++r) {
-      if (r >= m.n) break;
-      float f = 1.0f;
-      if (norm) f = a.joint ? mul[is_q ? 0 : 1][r] : 1.0f / sqrtf(head_ss[in_cta][r] / (float)a.dk + a.eps);
-      float y[V], o[V];
-      const float* row = ys + ((size_t)r * cta_heads + in_cta) * V * lph;
-#pragma unroll
-      for (int i = 0; i < V; i += 4) {
-        const float4 t = *reinterpret_cast<const float4*>(row + (i / 4) * lph * 4 + li * 4);
-        y[i] = t.x * f * nw[i]; y[i + 1] = t.y * f * nw[i + 1]; y[i + 2] = t.z * f * nw[i + 2]; y[i + 3] = t.w * f * nw[i + 3];
-      }
-      if (turn && a.half_layout) {
-        const float2* t = cs + r * half + (d < half ? d : d - half);
-#pragma unroll
-        for (int i = 0; i < V; i += 4) {
-          const float4 t4 = *reinterpret_cast<const float4*>(row + (i / 4) * lph * 4 + other * 4);
-          o[i] = t4.x; o[i + 1] = t4.y; o[i + 2] = t4.z; o[i + 3] = t4.w;
-        }
+      for (int k = -R; k < 2; ++k) {                           // input row r0 + k serves rows r0 + k .. r0 + k + R
+        const uint4 xr = *at(r0 + k);
+        const TA* x = reinterpret_cast<const TA*>(&xr);
 #pragma unroll
         for (int i = 0; i < V; ++i) {
-          const float p = o[i] * f * ow[i];
-          y[i] = d < half ? y[i] * t[i].x - p * t[i].y : y[i] * t[i].x + p * t[i].y;
-        }
-      } else if (turn) {
-        const float2* t = cs + r * half + d / 2;
+          const float v = ca_f32(x[i]);
 #pragma unroll
-        for (int i = 0; i < V; i += 2) {
-          const float u = y[i], v = y[i + 1];
-          y[i] = u * t[i / 2].x - v * t[i / 2].y;
-          y[i + 1] = v * t[i / 2].x + u * t[i / 2].y;
+          for (int r = 0; r < 2; ++r)
+            if (r - k >= 0 && r - k <= R) y[r][i] = fmaf(w[r - k >= 0 && r - k <= R ? r - k : 0][i], v, y[r][i]);
         }
       }
+    }
+    fetch(r0 + 4);
+    fetch(r0 + 5);
+    commit();
+    if (norm) {
+      float (*hss)[kCapJointWarps * 32] = head_ss[(r0 >> 1) & 1];
+      float ss[2];
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        ss[r] = 0.f;
+#pragma unroll
+        for (int i = 0; i < V; ++i) ss[r] = fmaf(y[r][i], y[r][i], ss[r]);
+      }
+      if (lph == 16) {                                         // (128-wide heads; all lanes take part)
+#pragma unroll
+        for (int o = 8; o > 0; o >>= 1)
+#pragma unroll
+          for (int r = 0; r < 2; ++r) ss[r] += __shfl_xor_sync(0xffffffffu, ss[r], o);
+      } else {
+        for (int o = lph >> 1; o > 0; o >>= 1)
+#pragma unroll
+          for (int r = 0; r < 2; ++r) ss[r] += __shfl_xor_sync(0xffffffffu, ss[r], o);
+      }
+      if (a.joint && li == 0) {
+        hss[0][hs] = ss[0];
+        hss[1][hs] = ss[1];
+      }
+      if (a.joint) {
+        __syncthreads();                                       // (the other parity's sums may still be read)
+        // half a warp sums one row: a fixed order, the same in every warp
+        const int hr = lane >> 4, hl = lane & 15;
+        float sq = 0.f, sk = 0.f;
+        if (warp_q) {
+          for (int h = hl; h < a.H; h += 16) sq += hss[hr][h];
+#pragma unroll
+          for (int o = 8; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+        }
+        if (warp_k) {
+          for (int h = a.H + hl; h < a.H + a.G; h += 16) sk += hss[hr][h];
+#pragma unroll
+          for (int o = 8; o > 0; o >>= 1) sk += __shfl_xor_sync(0xffffffffu, sk, o);
+        }
+        const float fq = rsqrtf(fmaf(sq, inv_q, a.eps)), fk = rsqrtf(fmaf(sk, inv_k, a.eps));
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const float bq = __shfl_sync(0xffffffffu, fq, 16 * r), bk = __shfl_sync(0xffffffffu, fk, 16 * r);
+          if (qk) f[r] = is_q ? bq : bk;
+        }
+      } else if (qk) {
+#pragma unroll
+        for (int r = 0; r < 2; ++r) f[r] = rsqrtf(fmaf(ss[r], inv_dk, a.eps));
+      }
+      if (qk) {
+        const bf16* nr = reinterpret_cast<const bf16*>(&nraw);
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+#pragma unroll
+          for (int i = 0; i < V; ++i) y[r][i] *= f[r] * __bfloat162float(nr[i]);
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      if (r0 + r >= m.n) break;
+      if (a.half_layout && a.dims > 0) {
+#pragma unroll
+        for (int i = 0; i < V; i += 2) {
+          const float o0 = __shfl_sync(0xffffffffu, y[r][i], partner), o1 = __shfl_sync(0xffffffffu, y[r][i + 1], partner);
+          if (turn) {
+            const float4 t = *reinterpret_cast<const float4*>(table + (size_t)(r0 + r) * half + i);
+            y[r][i] = fmaf(o0, sgn * t.y, y[r][i] * t.x);
+            y[r][i + 1] = fmaf(o1, sgn * t.w, y[r][i + 1] * t.z);
+          }
+        }
+      } else if (turn) {
+#pragma unroll
+        for (int i = 0; i < V; i += 2) {
+          const float2 t = table[(size_t)(r0 + r) * half + i / 2];
+          const float u = y[r][i], v = y[r][i + 1];
+          y[r][i] = u * t.x - v * t.y;
+          y[r][i + 1] = v * t.x + u * t.y;
+        }
+      }
+      if (!act && !pad) continue;
       uint4 outv;
       TA* ov = reinterpret_cast<TA*>(&outv);
 #pragma unroll
-      for (int i = 0; i < V; ++i) ca_store(ov + i, y[i]);       // (zeros behind the head's own columns)
+      for (int i = 0; i < V; ++i) ca_store(ov + i, y[r][i]);    // (zeros behind the head's own columns)
       if (is_q) {
-        *reinterpret_cast<uint4*>(reinterpret_cast<TA*>(a.q_out) + ((size_t)(m.row0 + m.q0 + r) * a.H + hs) * a.wk + d) = outv;
+        *reinterpret_cast<uint4*>(q_dst + (size_t)((r0 + r) * a.H) * a.wk) = outv;
       } else {
-        const int slot = slots[r];
-        if (slot >= 0) *reinterpret_cast<uint4*>(reinterpret_cast<TA*>(a.k_cache) + cap_cache_row(a, slot, g) * wide + d) = outv;
+        const int slot = a.slots[row0 + r0 + r];
+        if (slot >= 0)
+          *reinterpret_cast<uint4*>(kv_dst + cap_cache_row(a, slot, g) * wide) = outv;
       }
     }
   }
-  if (a.joint && norm) cg::this_cluster().sync();       // nobody leaves while another CTA may still read its sums
 }
 
 // Any width, any number of taps: warps take the head slots in turn, lanes the columns; a head is staged in shared memory
@@ -504,7 +551,7 @@ extern "C" int b200_conv_attn_prep_ex(const void* proj, int f32, int64_t ld, con
   if (n_x == 0) return B200_OK;
   int shift = 0;
   while ((1 << shift) < page) ++shift;
-  const CapArgs a{proj, ld, conv_w, (const bf16*)qnorm_w, (const bf16*)knorm_w, taps > 1 ? ring : nullptr, cu_seq, ctx_lens,
+  CapArgs a{proj, ld, conv_w, (const bf16*)qnorm_w, (const bf16*)knorm_w, taps > 1 ? ring : nullptr, cu_seq, ctx_lens,
                   state_slots, tile_seq, tile_q0, n_tiles * per_tile, per_tile, n_prompt, slots, q_out, k_cache, v_cache, H, G,
                   dk, dv, wk, wv, page, (1 << shift) == page ? shift : -1, taps, eps, joint_norm, rot_dims, half_layout, (const float2*)cos_sin};
   cudaStream_t s = (cudaStream_t)stream;
@@ -516,32 +563,26 @@ extern "C" int b200_conv_attn_prep_ex(const void* proj, int f32, int64_t ld, con
     const int piece = half_layout ? 2 * vec : vec;      // the rotated entries in whole pieces (and their partners too)
     int lph = 1;
     while (lph < wmax / vec) lph <<= 1;
-    // a power of two of CTAs (one cluster) that covers all head slots, in CTAs of equal size
-    const int all_warps = lph <= 32 ? (n_heads + 32 / lph - 1) / (32 / lph) : 1 << 20;
-    int ny = 1;
-    while (ny < 8 && ny * kCapJointWarps < all_warps) ny <<= 1;
-    const int warps_v = (all_warps + ny - 1) / ny;
-    const size_t smem_v = sizeof(float) * kCapRows * ((size_t)rot_dims + (size_t)warps_v * 32 * vec);
+    const int warps = lph <= 32 ? (n_heads + 32 / lph - 1) / (32 / lph) : 1 << 20;       // all head slots in one CTA
+    const size_t smem_v = sizeof(uint4) * kCapSlots * 32 * (size_t)warps;
     if (al && taps <= 4 && dk % vec == 0 && dv % vec == 0 && wk % vec == 0 && wv % vec == 0 && ld % vec == 0 && C % 4 == 0 &&
-        ny * kCapJointWarps >= all_warps && rot_dims % piece == 0 && smem_v <= 100 * 1024) {
-      cudaLaunchConfig_t cfg = {};
-      cudaLaunchAttribute at[1];
-      at[0].id = cudaLaunchAttributeClusterDimension;
-      at[0].val.clusterDim.x = 1;
-      at[0].val.clusterDim.y = ny;
-      at[0].val.clusterDim.z = 1;
-      cfg.gridDim = dim3(n_x, ny);
-      cfg.blockDim = dim3(warps_v * 32);
-      cfg.dynamicSmemBytes = smem_v;
-      cfg.stream = s;
-      cfg.attrs = at;
-      cfg.numAttrs = 1;
-      cudaError_t e = cudaSuccess;
-#define B200_CAJ(TA, N)                                                                                                           \
-  do {                                                                                                                            \
-    if (smem_v > 40 * 1024)                                                                                                       \
-      e = cudaFuncSetAttribute(conv_attn_prep_joint_vec_kernel<TA, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);  \
-    if (e == cudaSuccess) e = cudaLaunchKernelEx(&cfg, conv_attn_prep_joint_vec_kernel<TA, N>, a, lph);                           \
+        warps <= kCapJointWarps && rot_dims % piece == 0 && (n_tiles == 0 || tile_rows % kCapRun == 0) &&
+        (reinterpret_cast<uintptr_t>(cos_sin) & 15) == 0) {
+      a.per_tile = n_tiles > 0 ? tile_rows / kCapRun : 1;
+      a.n_pieces = n_tiles * a.per_tile;
+      const int n_run = a.n_pieces + n_single;
+#define B200_CAJ(TA, N)                                                                                                       \
+  do {                                                                                                                        \
+    if (smem_v > 32 * 1024) {                                                                                                 \
+      const cudaError_t e = cudaFuncSetAttribute(conv_attn_prep_joint_vec_kernel<TA, N>,                                      \
+                                                 cudaFuncAttributeMaxDynamicSharedMemorySize,                                 \
+                                                 (int)(sizeof(uint4) * kCapSlots * 32 * kCapJointWarps));                     \
+      if (e != cudaSuccess) {                                                                                                 \
+        b200_set_error("conv_attn_prep(joint): %s", cudaGetErrorString(e));                                                   \
+        return B200_ERR_CUDA;                                                                                                 \
+      }                                                                                                                       \
+    }                                                                                                                         \
+    conv_attn_prep_joint_vec_kernel<TA, N><<<n_run, warps * 32, smem_v, s>>>(a, lph);                                         \
   } while (0)
 #define B200_CAJT(TA)                        \
   switch (taps) {                            \
@@ -553,10 +594,6 @@ extern "C" int b200_conv_attn_prep_ex(const void* proj, int f32, int64_t ld, con
       if (f32) { B200_CAJT(float) } else { B200_CAJT(bf16) }
 #undef B200_CAJT
 #undef B200_CAJ
-      if (e != cudaSuccess) {
-        b200_set_error("conv_attn_prep(joint): %s", cudaGetErrorString(e));
-        return B200_ERR_CUDA;
-      }
       return b200_check_launch("b200_conv_attn_prep(joint)");
     }
     const size_t smem = sizeof(float) * kCapWarps * (dk > dv ? dk : dv);
