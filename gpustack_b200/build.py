@@ -130,7 +130,6 @@ PRE_NORM_SOURCES = [
     "conv_attn_prep.cu",
     "conv_rec_prep.cu",
     "gated_scan.cu",
-    "linear_attn.cu",
     "attention_sink.cu",
 ]
 

@@ -324,7 +324,7 @@ gated_scan_kernel(GatedScanArgs a) {
 
 // Single rows (a decode step): the state, the token's rows and its gates are in flight together; no staging, no barrier.
 template <int L, int R4, bool DELTA>
-__global__ void __launch_bounds__(kGsWarps * 32, 1)
+__global__ void __launch_bounds__(kGsWarps * 32, 4)
 gated_step_kernel(GatedScanArgs a) {
   constexpr int R2 = 2 * R4, CPW = 32 / L, COLS = kGsWarps * CPW;
   const int s = blockIdx.x, h = blockIdx.y, z = blockIdx.z;
@@ -392,6 +392,11 @@ int gated_scan_form(const GatedScanArgs& a, int n_seqs, int max_len, cudaStream_
     gated_step_kernel<L, R4, DELTA><<<dim3(n_seqs, a.H, (a.dv + COLS - 1) / COLS), kGsWarps * 32, 0, s>>>(a);
     return b200_check_launch("b200_gated_scan(step)");
   }
+  // too few CTAs to fill the GPU: the widest spread of a column over lanes, the shortest walk per token
+  if constexpr (PL == 16 && PR4 == 2) {
+    constexpr int COLS = kGsWarps * 2 * (32 / PL);
+    if (n_seqs * a.H * ((a.dv + COLS - 1) / COLS) < 148) return gated_scan_launch<32, 1, 2, DELTA>(a, n_seqs, s);
+  }
   return gated_scan_launch<PL, PR4, 2, DELTA>(a, n_seqs, s);
 }
 
@@ -406,8 +411,9 @@ int gated_scan_pick(const GatedScanArgs& a, int n_seqs, int max_len, cudaStream_
 }
 
 // ------------------------------------------------------------------------------------------- out
-// out = RMSnorm over `parts` equal pieces of (y * silu(z)), times w: the gate comes BEFORE the norm.  One CTA per row; the
-// gated row is staged in shared memory between the statistic and the product.
+// out = RMSnorm over `parts` equal pieces of (y * silu(z)), times w[channel] -- the gate BEFORE the norm -- or, with the gate
+// AFTER it, RMSnorm of the pieces of y times w[place in the piece] (one weight vector for all pieces) times silu(z).  One CTA
+// per row; the row is staged in shared memory between the statistic and the product.
 template <typename TA>
 __device__ __forceinline__ float4 gs_ld4(const TA* p);
 template <>
@@ -427,7 +433,7 @@ __device__ __forceinline__ float gs_silu(float z) { return z / (1.0f + expf(-z))
 
 constexpr int kGnThreads = 256;
 
-template <typename TA, bool VEC>
+template <typename TA, bool VEC, bool AFTER>
 __global__ void __launch_bounds__(kGnThreads)
 gate_norm_kernel(const float* __restrict__ y, const TA* __restrict__ proj, int64_t ld, int z_col, const bf16* __restrict__ w,
                  TA* out, int64_t ldo, int C, int parts, float eps) {
@@ -448,12 +454,14 @@ gate_norm_kernel(const float* __restrict__ y, const TA* __restrict__ proj, int64
         const int c = p * W + i;
         if (VEC) {
           float4 v = *reinterpret_cast<const float4*>(yr + c);
-          const float4 g = gs_ld4<TA>(zr + c);
-          v.x *= gs_silu(g.x); v.y *= gs_silu(g.y); v.z *= gs_silu(g.z); v.w *= gs_silu(g.w);
+          if (!AFTER) {
+            const float4 g = gs_ld4<TA>(zr + c);
+            v.x *= gs_silu(g.x); v.y *= gs_silu(g.y); v.z *= gs_silu(g.z); v.w *= gs_silu(g.w);
+          }
           *reinterpret_cast<float4*>(row + c) = v;
           ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
         } else {
-          const float v = yr[c] * gs_silu(gs_ld1(zr + c));
+          const float v = AFTER ? yr[c] : yr[c] * gs_silu(gs_ld1(zr + c));
           row[c] = v;
           ss = fmaf(v, v, ss);
         }
@@ -473,12 +481,56 @@ gate_norm_kernel(const float* __restrict__ y, const TA* __restrict__ proj, int64
       const int c = p * W + i;
       if (VEC) {
         float4 v = *reinterpret_cast<const float4*>(row + c);
-        const float4 g = gs_ld4<bf16>(w + c);
+        const float4 g = gs_ld4<bf16>(w + (AFTER ? i : c));
+        if (AFTER) {
+          const float4 t = gs_ld4<TA>(zr + c);
+          v.x *= gs_silu(t.x); v.y *= gs_silu(t.y); v.z *= gs_silu(t.z); v.w *= gs_silu(t.w);
+        }
         gs_st4(o + c, make_float4(v.x * rstd * g.x, v.y * rstd * g.y, v.z * rstd * g.z, v.w * rstd * g.w));
       } else {
-        gs_st1(o + c, row[c] * rstd * gs_ld1(w + c));
+        gs_st1(o + c, row[c] * rstd * gs_ld1(w + (AFTER ? i : c)) * (AFTER ? gs_silu(gs_ld1(zr + c)) : 1.0f));
       }
     }
+  }
+}
+
+// Pieces of up to 128 channels (a head): W / 4 neighbouring lanes share one, a thread holds up to 8 of its row's 16-byte
+// groups in registers and all their loads are in flight together.
+template <typename TA, bool AFTER>
+__global__ void __launch_bounds__(kGnThreads)
+gate_norm_heads_kernel(const float* __restrict__ y, const TA* __restrict__ proj, int64_t ld, int z_col, const bf16* __restrict__ w, TA* out,
+                       int64_t ldo, int C, int W, float eps) {
+  constexpr int N = 8;
+  const int t = blockIdx.x, i0 = threadIdx.x * 4, step = kGnThreads * 4, lanes = W >> 2;
+  const float* yr = y + (size_t)t * C;
+  const TA* zr = proj + (size_t)t * ld + z_col;
+  TA* o = out + (size_t)t * ldo;
+  float4 v[N], g[N];
+#pragma unroll
+  for (int n = 0; n < N; ++n) {
+    const int i = i0 + n * step;
+    if (n * step >= C) break;
+    v[n] = g[n] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < C) {
+      v[n] = *reinterpret_cast<const float4*>(yr + i);
+      g[n] = gs_ld4<TA>(zr + i);
+    }
+  }
+#pragma unroll
+  for (int n = 0; n < N; ++n) {
+    const int i = i0 + n * step;
+    if (n * step >= C) break;
+    g[n] = make_float4(gs_silu(g[n].x), gs_silu(g[n].y), gs_silu(g[n].z), gs_silu(g[n].w));
+    float4 x = v[n];
+    if (!AFTER) { x.x *= g[n].x; x.y *= g[n].y; x.z *= g[n].z; x.w *= g[n].w; }
+    float ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w)));
+    for (int w_ = lanes >> 1; w_ > 0; w_ >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, w_);
+    if (i >= C) continue;
+    const float rstd = 1.0f / sqrtf(ss / (float)W + eps);
+    const float4 c = gs_ld4<bf16>(w + (AFTER ? i % W : i));
+    x = make_float4(x.x * rstd * c.x, x.y * rstd * c.y, x.z * rstd * c.z, x.w * rstd * c.w);
+    if (AFTER) { x.x *= g[n].x; x.y *= g[n].y; x.z *= g[n].z; x.w *= g[n].w; }
+    gs_st4(o + i, x);
   }
 }
 
@@ -502,19 +554,33 @@ extern "C" int b200_gated_scan(const float* x, int64_t ld, int q_col, int k_col,
 }
 
 extern "C" int b200_gate_norm(const float* y, const void* proj, int f32, int64_t ld, int z_col, const void* w, void* out,
-                              int64_t ldo, int T, int C, int parts, float eps, void* stream) {
+                              int64_t ldo, int T, int C, int parts, int gate_after, float eps, void* stream) {
   B200_REQUIRE(T >= 0 && C > 0 && parts > 0 && C % parts == 0, "gate_norm: %d channels in %d parts", C, parts);
   if (T == 0) return B200_OK;
   const size_t smem = sizeof(float) * (size_t)C;
-  B200_REQUIRE(smem <= 48 * 1024, "gate_norm: %d channels exceed the staged row (12288)", C);
   cudaStream_t s = (cudaStream_t)stream;
   auto al = [](const void* p, int n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; };
   const int n = f32 ? 16 : 8;
   const bool vec = (C / parts) % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 && z_col % 4 == 0 && al(y, 16) && al(proj, n) && al(out, n) && al(w, 8);
-#define B200_GN(TA, V) \
-  gate_norm_kernel<TA, V><<<T, kGnThreads, smem, s>>>(y, (const TA*)proj, ld, z_col, (const bf16*)w, (TA*)out, ldo, C, parts, eps)
-  if (f32) { if (vec) B200_GN(float, true); else B200_GN(float, false); }
-  else { if (vec) B200_GN(bf16, true); else B200_GN(bf16, false); }
+  const int W = C / parts, lanes = W / 4;
+  if (vec && lanes <= 32 && (lanes & (lanes - 1)) == 0 && C <= kGnThreads * 4 * 8) {
+#define B200_GNH(TA, A) gate_norm_heads_kernel<TA, A><<<T, kGnThreads, 0, s>>>(y, (const TA*)proj, ld, z_col, (const bf16*)w, (TA*)out, ldo, C, W, eps)
+    if (f32) { if (gate_after) B200_GNH(float, true); else B200_GNH(float, false); }
+    else { if (gate_after) B200_GNH(bf16, true); else B200_GNH(bf16, false); }
+#undef B200_GNH
+    return b200_check_launch("b200_gate_norm");
+  }
+  B200_REQUIRE(smem <= 48 * 1024, "gate_norm: %d channels exceed the staged row (12288)", C);
+#define B200_GN(TA, V, A) \
+  gate_norm_kernel<TA, V, A><<<T, kGnThreads, smem, s>>>(y, (const TA*)proj, ld, z_col, (const bf16*)w, (TA*)out, ldo, C, parts, eps)
+#define B200_GN2(TA)                                                                                     \
+  do {                                                                                                   \
+    if (gate_after) { if (vec) B200_GN(TA, true, true); else B200_GN(TA, false, true); }                 \
+    else { if (vec) B200_GN(TA, true, false); else B200_GN(TA, false, false); }                          \
+  } while (0)
+  if (f32) B200_GN2(float);
+  else B200_GN2(bf16);
+#undef B200_GN2
 #undef B200_GN
   return b200_check_launch("b200_gate_norm");
 }

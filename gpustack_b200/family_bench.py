@@ -1193,6 +1193,8 @@ def _kernel_numbers_bovitar(size, T, B, ctx, log):
         t_new = _time(lambda: ops.gate_norm(o_raw[:n], pz[:n], Ci, nw, mo[:n], sg, 1e-5), flush)
         t_like = _time(lambda: ops.linattn_out(o_raw[:n], pz[:n], Ci, nw[:sw], mo[:n], sh, sw, 1e-5, False, "silu"), flush)
         put("gate_norm" + tag, t_new, n * Ci * 8.0, "linattn_out" + tag, t_like, n * Ci * 8.0, "bytes")
+        t_new = _time(lambda: ops.gate_norm(o_raw[:n], pz[:n], Ci, nw[:dw], mo[:n], Ci // dw, 1e-5, gate_after=True), flush)
+        put("gate_norm, gate after" + tag, t_new, n * Ci * 8.0, "linattn_out" + tag, t_like, n * Ci * 8.0, "bytes")
 
     # ---- routed SiLU experts chosen inside groups vs Danipel's clamped gated experts (both with their sum)
     xin = rnd(T, D)

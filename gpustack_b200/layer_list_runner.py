@@ -637,7 +637,7 @@ class LayerListRunner(ModelRunner):
         kc = G * S.shape[3]
         ops.gated_scan(x32, 0, kc, 2 * kc, gates, lw.decay_rate, lw.dt_bias, None, cu_all, ctx_all, slots_all, S, o_raw, H, G, dk, dv,
                        True, max_len=Tp if Tp else 1)
-        ops.linattn_out(o_raw, proj, m.conv_width, lw.out_norm, out, H, dv, self.mcfg.norm_eps, False, "silu")
+        ops.gate_norm(o_raw, proj, m.conv_width, lw.out_norm, out, H, self.mcfg.norm_eps, gate_after=True)
         ops.linear(out, lw.o, self.y[:T])
         self._pending = {"y": self.y[:T]}
         self.stats["kernel_launches"] += 6

@@ -184,7 +184,7 @@ SIGNATURES = {
                                   _vp, _vp, _i64, _f32, _vp]),
     "b200_gated_scan": (_i32, [_vp, _i64, _i32, _i32, _i32, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32,
                                _i32, _i32, _i32, _vp]),
-    "b200_gate_norm": (_i32, [_vp, _vp, _i32, _i64, _i32, _vp, _vp, _i64, _i32, _i32, _i32, _f32, _vp]),
+    "b200_gate_norm": (_i32, [_vp, _vp, _i32, _i64, _i32, _vp, _vp, _i64, _i32, _i32, _i32, _i32, _f32, _vp]),
     "b200_prenorm_join": (_i32, [_vp, _vp, _vp, _vp, _vp, _f32, _f32, _vp, _vp, _i32, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _f32,
                                  _f32, _vp]),
     "b200_moe_route_grouped": (_i32, [_vp, _i64, _vp, _vp, _vp, _i32, _i32, _i32, _f32, _i32, _i32, _i32, _i32, _vp]),

@@ -912,12 +912,15 @@ def gated_scan(x, q_col: int, k_col: int, v_col: int, gates, rate, dt_bias, skip
                                  1 if delta else 0, int(max_len), _stream()), "gated_scan")
 
 
-def gate_norm(y, proj, z_col: int, norm_w, out, parts: int, eps: float):
-    """out = RMS norm over `parts` equal pieces of (y * silu(z)) * w; z: columns z_col .. of proj; y fp32 contiguous rows."""
+def gate_norm(y, proj, z_col: int, norm_w, out, parts: int, eps: float, gate_after: bool = False):
+    """out = RMS norm over `parts` equal pieces of (y * silu(z)) * w; z: columns z_col .. of proj; y fp32 contiguous rows.
+    gate_after: RMS norm of the pieces of y, times one weight vector of a piece's width, times silu(z)."""
     _cuda(y, proj, norm_w, out)
     _req(y, torch.float32, "y")
+    if norm_w.numel() != (y.shape[1] // parts if gate_after else y.shape[1]):
+        raise B200Error("gate_norm: one weight per channel, or with gate_after one per place in a piece")
     check(load().b200_gate_norm(_p(y), _p(proj), _is_f32(proj), proj.stride(0), z_col, _p(norm_w), _p(out), out.stride(0), y.shape[0],
-                                y.shape[1], parts, eps, _stream()), "gate_norm")
+                                y.shape[1], parts, 1 if gate_after else 0, eps, _stream()), "gate_norm")
 
 
 def prenorm_join(x_in, w, eps: float, y=None, pair=None, routed=None, x_out=None, h_out=None, rows=None, out_scale: float = 1.0):

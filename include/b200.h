@@ -585,9 +585,10 @@ int b200_gated_scan(const float* x, int64_t ld, int q_col, int k_col, int v_col,
                     const float* rate, const float* dt_bias, const float* skip, const int32_t* cu_seq, const int32_t* ctx_lens,
                     const int32_t* state_slots, float* S, float* o_raw, int n_seqs, int H, int G, int dk, int dv, int delta,
                     int max_len, void* stream);
-/* out = RMSnorm over `parts` equal pieces of (y * silu(z)) * w (the gate comes before the norm). */
+/* out = RMSnorm over `parts` equal pieces of (y * silu(z)) * w (the gate comes before the norm, one weight per channel), or
+ * with gate_after RMSnorm of the pieces of y * w * silu(z) (one weight vector of a piece's width for all pieces). */
 int b200_gate_norm(const float* y, const void* proj, int f32, int64_t ld, int z_col, const void* w, void* out, int64_t ldo,
-                   int T, int C, int parts, float eps, void* stream);
+                   int T, int C, int parts, int gate_after, float eps, void* stream);
 /* z = x_in + c; x_out = z; h_out = z / rms(z) * w * out_scale.  c: y (NULL: nothing); or with y2 the normed pair
  * ya * y / rms(y) * wy + yb * y2 / rms(y2) * wy2; or with yp a routed feed-forward, sum_j yp[pair_row[t top_k + j]] (+ shared[t]).
  * rows != NULL: gather, h_out only. */

@@ -140,12 +140,12 @@ def test_library_subset_of_a_pre_norm_model():
 
     c = LayerListConfig.from_dict(_cfg())
     tag, srcs = build.layer_list_sources(c)
-    assert tag == "pre_norm_routed_tc" and {"prenorm.cu", "conv_attn_prep.cu", "conv_rec_prep.cu", "gated_scan.cu", "linear_attn.cu",
+    assert tag == "pre_norm_routed_tc" and {"prenorm.cu", "conv_attn_prep.cu", "conv_rec_prep.cu", "gated_scan.cu",
                                             "attention_sink.cu", "attention.cu", "attention_prefill_tc.cu", "moe.cu"} <= set(srcs)
     assert not {"mlstm.cu", "sandwich.cu", "allreduce.cu", "norm.cu", "postnorm.cu", "latent.cu"} & set(srcs)
     h = ctypes.CDLL(str(build.build(sources=srcs, tag=tag)))
     for n in ("b200_embed_streams", "b200_prenorm_join", "b200_conv_attn_prep_ex", "b200_rot_table", "b200_conv_rec_prep", "b200_gated_scan",
-              "b200_gate_norm", "b200_linattn_out", "b200_attn_sink_prefill_cap", "b200_attn_sink_decode_cap", "b200_paged_attn_prefill_cap",
+              "b200_gate_norm", "b200_attn_sink_prefill_cap", "b200_attn_sink_decode_cap", "b200_paged_attn_prefill_cap",
               "b200_paged_attn_decode_cap", "b200_moe_route_grouped", "b200_moe_align", "b200_moe_gather_scaled", "b200_moe_grouped_gemm_ex",
               "b200_linear_simt_grouped_ex", "b200_gemm_bf16_silu_mul", "b200_linear_simt", "b200_sample_softcap_f32", "b200_last_error"):
         assert hasattr(h, n), n

@@ -397,9 +397,9 @@ def test_one_early_write_is_still_read_a_thousand_tokens_later(delta):
             assert _rel(torch.cat(outs), want.view(T, dv)) < 1e-5 + T * 2.0 ** -25, (gone, len(cuts))
 
 
-@pytest.mark.parametrize("C,parts", [(48, 1), (48, 3), (35, 5), (512, 2), (640, 10), (1024, 64), (4096, 1)])
+@pytest.mark.parametrize("C,parts", [(48, 1), (48, 3), (35, 5), (512, 2), (640, 10), (1024, 64), (4096, 1), (8192, 64), (5000, 1250)])
 @pytest.mark.parametrize("dtype", [torch.float32, BF])
-def test_gate_before_the_grouped_norm(C, parts, dtype):
+def test_gate_before_and_after_the_grouped_norm(C, parts, dtype):
     from gpustack_b200 import ops
 
     T, z_col = 5, 12
@@ -408,7 +408,13 @@ def test_gate_before_the_grouped_norm(C, parts, dtype):
     out = torch.zeros(T, C, dtype=dtype, device="cuda")
     ops.gate_norm(y.cuda(), z.cuda(), z_col, w.cuda(), out, parts, 1e-5)
     want = O.grouped_rms(y.to(F64) * O.silu(z[:, z_col:z_col + C].to(F64)), parts, 1e-5) * w.to(F64)
-    assert _rel(out, want) < (3e-6 if dtype == torch.float32 else 8e-3)
+    tol = 3e-6 if dtype == torch.float32 else 8e-3
+    assert _rel(out, want) < tol
+    # ... and the norm of every piece, one weight vector for all of them, before the gate
+    shared = w[:C // parts].contiguous()
+    ops.gate_norm(y.cuda(), z.cuda(), z_col, shared.cuda(), out, parts, 1e-5, gate_after=True)
+    want = O.grouped_rms(y.to(F64), parts, 1e-5) * shared.to(F64).repeat(parts) * O.silu(z[:, z_col:z_col + C].to(F64))
+    assert _rel(out, want) < tol
 
 
 @pytest.mark.parametrize("D", [37, 64, 300, 5000])
